@@ -8,7 +8,7 @@
 
 namespace kge {
 
-constexpr int ATT_WARPS = 4, ATT_MAXV = 8;   // value columns per lane: vdim <= 32 * ATT_MAXV
+constexpr int ATT_WARPS = 4, ATT_MAXV = 32;   // value columns per lane at most: vdim <= 32 * ATT_MAXV
 
 // Keys of a row with a window: first the `prefix` keys - kept first tokens that have left the window (their own rows of
 // the caches) or pooled blocks that lie wholly before it (rows of the pooled caches) - then the window's tokens.
@@ -27,7 +27,8 @@ __device__ __forceinline__ int64_t prefix_row(const AttnBiasArgs& a, const int32
   return ((int64_t)bt[u / a.block_size] * a.G + g) * a.block_size + u % a.block_size;
 }
 
-template <typename E>
+// MAXV: value columns per lane
+template <typename E, int MAXV>
 __global__ void __launch_bounds__(ATT_WARPS * 32) attn_bias_chunk_kernel(AttnBiasArgs a) {
   pdl_launch_dependents();
   pdl_wait();
@@ -47,12 +48,13 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attn_bias_chunk_kernel(AttnBia
   const int32_t* bt = a.block_table + (int64_t)b * a.max_blocks;
   const E* kc = (const E*)a.k_cache;
   const E* vc = (const E*)a.v_cache;
+  const int64_t vld = a.v_ld > 0 ? a.v_ld : a.vdim;
   const bool pooled = a.pool > 0;
   const E* pkc = pooled ? (const E*)a.pk_cache : kc;
   const E* pvc = pooled ? (const E*)a.pv_cache : vc;
-  float m = -INFINITY, l = 0.f, o[ATT_MAXV];
+  float m = -INFINITY, l = 0.f, o[MAXV];
 #pragma unroll
-  for (int c = 0; c < ATT_MAXV; ++c) o[c] = 0.f;
+  for (int c = 0; c < MAXV; ++c) o[c] = 0.f;
   // the row's keys in one list: npre prefix keys, then positions lo .. i
   const int nkeys = npre + (i - lo + 1);
   for (int u0 = 0; u0 < nkeys; u0 += 32) {
@@ -76,14 +78,14 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attn_bias_chunk_kernel(AttnBia
     l = l * corr + warp_sum(p);
     m = mn;
 #pragma unroll
-    for (int c = 0; c < ATT_MAXV; ++c) o[c] *= corr;
+    for (int c = 0; c < MAXV; ++c) o[c] *= corr;
     const int cnt = min(32, nkeys - u0);
     for (int jj = 0; jj < cnt; ++jj) {
       const float pj = __shfl_sync(0xffffffffu, p, jj);
       const int64_t rj = __shfl_sync(0xffffffffu, row, jj);
-      const E* vr = (u0 + jj < npre ? pvc : vc) + rj * a.vdim;
+      const E* vr = (u0 + jj < npre ? pvc : vc) + rj * vld;
 #pragma unroll
-      for (int c = 0; c < ATT_MAXV; ++c) {
+      for (int c = 0; c < MAXV; ++c) {
         const int col = c * 32 + lane;
         if (col < a.vdim) o[c] = fmaf(pj, ldf(vr + col), o[c]);
       }
@@ -93,12 +95,12 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attn_bias_chunk_kernel(AttnBia
     const float sk = a.sinks[h], mn = fmaxf(m, sk), corr = expf(m - mn);
     l = l * corr + expf(sk - mn);
 #pragma unroll
-    for (int c = 0; c < ATT_MAXV; ++c) o[c] *= corr;
+    for (int c = 0; c < MAXV; ++c) o[c] *= corr;
   }
   const float inv = a.out_scale / l;
   E* out = (E*)a.out + (int64_t)t * a.ldo + h * a.vdim;
 #pragma unroll
-  for (int c = 0; c < ATT_MAXV; ++c) {
+  for (int c = 0; c < MAXV; ++c) {
     const int col = c * 32 + lane;
     if (col < a.vdim) stf(out + col, o[c] * inv);
   }
@@ -196,7 +198,7 @@ __global__ void __launch_bounds__(AM_WARPS * 32) attn_bias_mma_kernel(AttnBiasAr
   for (int v = 0; v < AM_MAXD / 8; ++v) o[v][0] = o[v][1] = o[v][2] = o[v][3] = 0.f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   const int32_t* bt = a.block_table + (int64_t)b * a.max_blocks;
-  const int kseg = dim >> 3, vseg = vdim >> 3;
+  const int kseg = dim >> 3, vseg = vdim >> 3, vld = a.v_ld > 0 ? a.v_ld : vdim;
   for (int kt = ROWS ? 0 : warp; kt < ntiles; kt += ROWS ? 1 : AM_WARPS) {
     const bool ptile = kt < ptiles;                         // a tile of prefix keys: j0 counts them from 0
     const int j0 = ptile ? kt * AM_KT : lo_min + (kt - ptiles) * AM_KT;
@@ -234,7 +236,7 @@ __global__ void __launch_bounds__(AM_WARPS * 32) attn_bias_mma_kernel(AttnBiasAr
         const int key = idx / vseg, seg = idx % vseg;
         const int64_t row = __shfl_sync(0xffffffffu, myrow, key);
         v[u] = make_uint4(0u, 0u, 0u, 0u);
-        if (row >= 0) v[u] = *reinterpret_cast<const uint4*>(vc + row * vdim + seg * 8);
+        if (row >= 0) v[u] = *reinterpret_cast<const uint4*>(vc + row * vld + seg * 8);
         dst[u] = key * vst + seg * 8;
       }
 #pragma unroll
@@ -381,7 +383,7 @@ int attn_bias_chunk(const AttnBiasArgs& a, cudaStream_t st) {
               (a.pool == 0 || (a.pk_cache && a.pv_cache && a.pool_slots > 0)),
               "attn_bias_chunk: window %d with %d kept tokens / pooled blocks of %d", a.window, a.keep_first, a.pool);
   if (a.elt == KGE_ELT_BF16 && a.max_q > 0 && a.dim % 16 == 0 && a.dim <= AM_MAXD && a.vdim % 8 == 0 && a.vdim <= AM_MAXD && a.ldq % 2 == 0 &&
-      a.H % a.G == 0 && (reinterpret_cast<uintptr_t>(a.q) & 3) == 0 && a.B <= 65535 && a.G <= 65535) {
+      a.H % a.G == 0 && a.v_ld % 8 == 0 && (reinterpret_cast<uintptr_t>(a.q) & 3) == 0 && a.B <= 65535 && a.G <= 65535) {
     const int hpg = a.H / a.G;
     const size_t smem = (size_t)AM_WARPS * AM_KT * (a.dim + a.vdim + 2 * AM_PAD) * 2 + (size_t)AM_WARPS * 2 * 16 * 4;
     static size_t smem_set = 0;                       // opt in once per size that needs more than the default 48 KB
@@ -403,12 +405,14 @@ int attn_bias_chunk(const AttnBiasArgs& a, cudaStream_t st) {
     return 0;
   }
   KGE_REQUIRE(a.vdim <= 32 * ATT_MAXV, "attn_bias_chunk: value head size %d > %d", a.vdim, 32 * ATT_MAXV);
-  KGE_REQUIRE(a.dim <= 1024 && a.H % a.G == 0, "attn_bias_chunk: bad head sizes");
+  KGE_REQUIRE(a.dim <= 2048 && a.H % a.G == 0, "attn_bias_chunk: bad head sizes");
   const int64_t items = (int64_t)a.T * a.H;
   const dim3 grid((unsigned)((items + ATT_WARPS - 1) / ATT_WARPS)), block(ATT_WARPS * 32);
   const size_t smem = (size_t)ATT_WARPS * a.dim * 4;
-  cudaError_t ce = a.elt == KGE_ELT_F32 ? launch_pdl(attn_bias_chunk_kernel<float>, grid, block, smem, st, a)
-                                        : launch_pdl(attn_bias_chunk_kernel<__nv_bfloat16>, grid, block, smem, st, a);
+  cudaError_t ce;
+  const bool f32 = a.elt == KGE_ELT_F32;
+  if (a.vdim <= 256) ce = f32 ? launch_pdl(attn_bias_chunk_kernel<float, 8>, grid, block, smem, st, a) : launch_pdl(attn_bias_chunk_kernel<__nv_bfloat16, 8>, grid, block, smem, st, a);
+  else ce = f32 ? launch_pdl(attn_bias_chunk_kernel<float, ATT_MAXV>, grid, block, smem, st, a) : launch_pdl(attn_bias_chunk_kernel<__nv_bfloat16, ATT_MAXV>, grid, block, smem, st, a);
   KGE_CUDA_OK(ce);
   return 0;
 }

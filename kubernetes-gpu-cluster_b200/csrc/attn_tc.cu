@@ -523,7 +523,7 @@ static int launch_tc(bf16* out, const bf16* q, int q_stride, const bf16* kc, con
 template <int HD>
 static int launch_tc_window(bf16* out, const bf16* q, int q_stride, const bf16* kc, const bf16* vc, const bf16* pkc, const bf16* pvc, const int32_t* bt,
                             int max_blocks, const int32_t* sl, const int32_t* qsl, int B, int max_q_len, int H, int KV, int bs, float scale,
-                            const atc::WinArgs& win, cudaStream_t st) {
+                            const atc::WinArgs& win, const float* sinks, cudaStream_t st) {
   int bs_shift = 0;
   while ((1 << bs_shift) < bs) ++bs_shift;
   const int TT = atc::BM / (H / KV);
@@ -541,7 +541,7 @@ static int launch_tc_window(bf16* out, const bf16* q, int q_stride, const bf16* 
   auto kern = atc::attn_tc_kernel<HD, true, false, true>;
   KGE_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, atc::tc_smem<HD>()));
   KGE_CUDA_OK(launch_pdl(kern, dim3((max_q_len + TT - 1) / TT, KV, B), dim3(192), atc::tc_smem<HD>(), st, tk, tv, out, q, q_stride, kc, vc, bt,
-                         max_blocks, sl, qsl, H, KV, bs_shift, scale * atc::kLog2e, 0.f, 0.f, (const float*)nullptr, tpk, tpv, win));
+                         max_blocks, sl, qsl, H, KV, bs_shift, scale * atc::kLog2e, 0.f, 0.f, sinks, tpk, tpv, win));
   return 0;
 }
 
@@ -554,17 +554,17 @@ bool paged_attn_window_tc_ok(int H, int KV, int hd, int vd, int bs, int pool, in
 }
 
 // Steps with prompt pieces, a sliding window with kept first tokens (keep_first > 0) or pooled blocks (pool > 0): the
-// tcgen05 kernel above with the window's tile range and masks.  Sizes: paged_attn_window_tc_ok.
+// tcgen05 kernel above with the window's tile range and masks, optional sinks.  Sizes: paged_attn_window_tc_ok.
 int paged_attn_window_tc(void* out, const void* q, int q_stride, const void* kc, const void* vc, const void* pkc, const void* pvc, const int32_t* bt,
                          int max_blocks, const int32_t* sl, const int32_t* qsl, int B, int max_q_len, int H, int KV, int hd, int bs, float scale,
-                         int window, int keep_first, int pool, int pool_slots, cudaStream_t st) {
+                         int window, int keep_first, int pool, int pool_slots, const float* sinks, cudaStream_t st) {
   KGE_REQUIRE(window > 0 && paged_attn_window_tc_ok(H, KV, hd, hd, bs, pool, pool_slots), "paged_attn_window_tc: unsupported sizes");
   atc::WinArgs win;
   win.window = window; win.keep_first = keep_first; win.pool = pool; win.pool_slots = pool_slots;
   if (hd == 128) return launch_tc_window<128>((bf16*)out, (const bf16*)q, q_stride, (const bf16*)kc, (const bf16*)vc, (const bf16*)pkc, (const bf16*)pvc, bt, max_blocks, sl, qsl, B,
-                                               max_q_len, H, KV, bs, scale, win, st);
+                                               max_q_len, H, KV, bs, scale, win, sinks, st);
   return launch_tc_window<64>((bf16*)out, (const bf16*)q, q_stride, (const bf16*)kc, (const bf16*)vc, (const bf16*)pkc, (const bf16*)pvc, bt, max_blocks, sl, qsl, B, max_q_len,
-                              H, KV, bs, scale, win, st);
+                              H, KV, bs, scale, win, sinks, st);
 }
 
 // Called by kge_paged_attn (attn.cu) for batches with query chunks longer than one token.

@@ -88,6 +88,16 @@ struct HybridLayerW {
   HybMat lat_uq, lat_ukv;
   void *lat_qnorm = nullptr, *lat_kvnorm = nullptr;
   int lat_dkv = 0, lat_g = 0;
+  // cached latents: `proj` holds [q | dkv] (or [q] for a layer that reads another layer's cache), kc the rows [c | turned key part],
+  // lat_uk the key up-projection per head and transposed [H, kv_rank, nope] (multiplies the queries), lat_ukv as above
+  HybMat lat_uk;
+  // gated delta rule: `proj` holds [q | k | v | a1 | g1 | b] (offsets off_k, off_v, off_a1, off_mg, off_b), conv_w the convolutions
+  // transposed [taps, q | k | v channels], wkv_w2 / g2 the second halves of the decay's (with its bias) and the gate's low-rank
+  // pairs, decay_coef exp(A_log) per decay column (fp32), wkv_norm the per-head output norm repeated for every head
+  HybMat g2;
+  int off_b = 0;
+  float* decay_coef = nullptr;
+  float* router_corr = nullptr;               // [router outputs] fp32: added to the scores for the choice
   // dense clamped gated unit: [gate | up] rows in one block (`up` names the second half)
   void* ff_gate = nullptr;
   void* ff_gate_b = nullptr;                  // [gate.b | up.b] of a gated unit whose projections carry biases
@@ -131,6 +141,16 @@ struct kge_engine {
   float *res32 = nullptr, *gates32 = nullptr, *logits32 = nullptr, *state = nullptr, *mo32 = nullptr;
   float* y32 = nullptr;                      // [tokens, d]: a sublayer's sum when it has more sources than one combine pass takes
   void* embed_norm_w = nullptr;              // weight of the norm the embedding goes through (models that have one)
+  void* bigram = nullptr;                    // second embedding table, picked by the token and the one before it
+  // cached latents: absorbed queries [rows, H, kv_rank + rot_part] and their outputs [rows, H, kv_rank] for the first latq_rows rows of a
+  // step; scratch of the expanded path (prompt pieces on the tcgen05 kernel): pages of keys / values, their rows before the
+  // reordering, and the page table of a group of requests
+  void *qabs = nullptr, *olat = nullptr, *exp_c = nullptr, *exp_kv = nullptr, *exp_k = nullptr, *exp_v = nullptr;
+  int32_t *exp_table = nullptr, *exp_src = nullptr;
+  int latq_rows = 0, exp_pages = 0;
+  float* qkv32 = nullptr;                    // gated delta rule: convolved q, k (unit vectors), v [tokens, channels]
+  int32_t* moe_prow = nullptr;               // permuted row of every (token, choice) pair, -1 for an expert that returns its input
+  void *ws_lat = nullptr; int64_t ws_lat_bytes = 0;      // partial results of latent_mqa
   void *mixes = nullptr, *rkvg = nullptr;    // WKV: the blended inputs [5, tokens, d] and the projections [4, tokens, heads * dim]
   void *latq = nullptr, *latc = nullptr, *latkv = nullptr, *qbuf = nullptr;   // latent attention: normed latents, [k | v] up-projections, queries
   void *hx = nullptr, *pbuf = nullptr, *ubuf = nullptr, *mixbuf = nullptr, *obuf1 = nullptr, *obuf2 = nullptr, *ffbuf = nullptr;

@@ -1,7 +1,8 @@
 // Layer-list ("hybrid") models in the engine: a config.json that lists its layers, each with a token mixer (gated
 // linear recurrence, attention and a matrix memory side by side, attention alone with rotary positions, a soft cap
-// and sink logits, a WKV recurrence, attention through latents, windowed attention with kept first tokens beside gated
-// linear attention, or windowed attention over pooled blocks) and a feed-forward (dense or mixture of experts),
+// and sink logits, a WKV recurrence, attention through latents (every head's keys and values or the latents themselves in
+// the cache), windowed attention with kept first tokens beside gated linear attention, windowed attention over pooled
+// blocks, or a gated delta rule) and a feed-forward (dense or mixture of experts),
 // reading ONE norm of an fp32 residual stream, a norm each in sequence (optionally with a norm of each result as
 // well), or a norm each of a hyper-connected residual (several copies of the stream).  This file loads such a model (weights in the engine's storage
 // type, fused where one activation feeds several projections), sizes its arena, paged caches and recurrent-state pool,
@@ -32,7 +33,7 @@ bool paged_attn_extras_decode_ok(int B, int H, int KV, int hd, int block_size);
 bool paged_attn_window_tc_ok(int H, int KV, int hd, int vd, int bs, int pool, int pool_slots);
 int paged_attn_window_tc(void* out, const void* q, int q_stride, const void* kc, const void* vc, const void* pkc, const void* pvc, const int32_t* bt,
                          int max_blocks, const int32_t* sl, const int32_t* qsl, int B, int max_q_len, int H, int KV, int hd, int bs, float scale,
-                         int window, int keep_first, int pool, int pool_slots, cudaStream_t st);
+                         int window, int keep_first, int pool, int pool_slots, const float* sinks, cudaStream_t st);
 // gemm_tc.cu: one tcgen05 launch over row groups padded to 256 (the experts of a prompt step)
 int gemm_grouped(void* y, const void* x, const void* w, int T, int N, int K, int groups, const int32_t* tile_group, int glu, float glu_alpha,
                  float glu_limit, cudaStream_t st);
@@ -139,6 +140,14 @@ int64_t align_up64(int64_t v, int64_t a) { return (v + a - 1) / a * a; }
 
 }  // namespace
 
+// whether prompt pieces of a cached-latent layer run on the tcgen05 kernel over keys and values expanded per step: bfloat16, keys
+// and values of 64 or 128 numbers, parts of whole 16-byte pieces
+static bool latent_expand_ok(const kge_engine* e, const HybridLayerSpec& h, int ldp) {
+  const int bs = e->cfg.block_size;
+  return !e->f32 && paged_attn_window_tc_ok(h.heads, h.heads, h.dim, h.vdim, bs, 0, 0) && latent_mqa_ok(h.heads, h.kv_rank, h.rot_part, bs) && h.rot_part % 8 == 0 &&
+         (h.dim - h.rot_part) % 8 == 0 && ldp % 8 == 0 && (bs >= 64 || 64 % bs == 0);
+}
+
 int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, std::string* err) {
   const ModelSpec& s = e->spec;
   HB b{e, &md, dummy_seed};
@@ -147,12 +156,16 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
   const float ws = 0.02f * 1.7320508f;
 #define HB_OK(p) do { if (!(p)) return fail(b.err); } while (0)
   HB_OK(e->embed = (bf16*)b.mat({"embed"}, {s.vocab}, d, ws));
+  if (s.bigram_buckets > 0) HB_OK(e->bigram = b.mat({"bigram"}, {s.bigram_buckets + 1}, d, ws));
   HB_OK(e->lm_head = (bf16*)b.mat({"head"}, {s.vocab}, d, ws));
   const bool plain_norm_w = s.hyb_layernorm || s.streams > 0 || s.hyb_postnorm;      // the norm weight multiplies as it is (else it is applied as 1 + w)
   HB_OK(e->final_w = (bf16*)b.mat({"final.norm"}, {d}, 1, 0.f, plain_norm_w ? 1.f : 0.f));
   if (s.embed_norm) HB_OK(e->embed_norm_w = b.mat({"embed.norm"}, {d}, 1, 0.f, 1.f));
   e->hyb.resize(s.L);
-  int64_t state_floats = 0;
+  int64_t state_floats = s.bigram_buckets > 0 ? 4 : 0;      // the slot starts with the sequence's last token (a 16-byte piece)
+  int max_abs = 0, max_olat = 0, max_exp_row = 0, max_exp_k = 0, max_exp_v = 0, max_win = 0, max_qkv32 = 0;
+  int64_t lat_ws = 0;
+  bool lat_tc = true;                                         // every cached-latent layer takes the expanded tcgen05 path in prompt steps
   int max_mo = 1;
   int max_proj = 1, max_mix = 1, max_ff = 1, max_gate = 1, max_u = 1, max_top = 0, max_eff = 1, max_E = 1;
   int max_hd = 0, max_qr = 0, max_kvr = 0, max_lkv = 0, max_lq = 0;      // WKV heads * dim; latent ranks, [k | v] and query widths
@@ -173,9 +186,13 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
       continue;
     }
     const float norm_one = plain_norm_w ? 1.f : 0.f;      // the weight that leaves the normed row as it is
+    if (s.hyb_noprenorm) {                      // the norms of the sublayers' results are the layer's only ones
+      HB_OK(L.norm1b = b.mat({p + "norm1"}, {d}, 1, 0.f, 1.f));
+      if (h.mlp != HybridLayerSpec::NONE) HB_OK(L.norm2b = b.mat({p + "norm2"}, {d}, 1, 0.f, 1.f));
+    } else
     HB_OK(L.norm1 = b.mat({p + "norm1"}, {d}, 1, 0.f, norm_one));
-    if (s.hyb_prenorm_pair && h.mlp != HybridLayerSpec::NONE) HB_OK(L.norm2 = b.mat({p + "norm2"}, {d}, 1, 0.f, norm_one));
-    if (s.hyb_postnorm) {
+    if (!s.hyb_noprenorm && s.hyb_prenorm_pair && h.mlp != HybridLayerSpec::NONE) HB_OK(L.norm2 = b.mat({p + "norm2"}, {d}, 1, 0.f, norm_one));
+    if (s.hyb_postnorm && !s.hyb_noprenorm) {
       HB_OK(L.norm1b = b.mat({p + "norm1b"}, {d}, 1, 0.f, 1.f));
       if (h.mlp != HybridLayerSpec::NONE) HB_OK(L.norm2b = b.mat({p + "norm2b"}, {d}, 1, 0.f, 1.f));
     }
@@ -297,6 +314,84 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
       HB_OK(L.o.w = b.mat({mx + "o"}, {d}, hd, ws));
       state_floats += wkv_state_floats(d, h.heads, h.dim);
       max_hd = std::max(max_hd, hd); max_mix = std::max(max_mix, hd); max_gate = std::max(max_gate, hd); max_mo = std::max(max_mo, hd); max_u = std::max(max_u, lr);
+    } else if (h.mixer == HybridLayerSpec::LATENT && h.latent_cache) {
+      const int H = h.heads, nope = h.dim - h.rot_part, nq = H * h.dim, row = h.kv_rank + h.rot_part, nv = H * h.vdim;
+      L.lat_dkv = nq; L.proj.K = d;
+      if (h.kv_from < 0) {
+        L.proj.N = nq + row;
+        HB_OK(L.proj.w = b.mat({mx + "q", mx + "dkv"}, {nq, row}, d, ws));
+        HB_OK(L.lat_kvnorm = b.mat({mx + "dkv.norm"}, {h.kv_rank}, 1, 0.f, 1.f));
+      } else {
+        L.proj.N = nq;
+        HB_OK(L.proj.w = b.mat({mx + "q"}, {nq}, d, ws));
+      }
+      L.lat_ukv.N = H * nope + nv; L.lat_ukv.K = h.kv_rank;
+      HB_OK(L.lat_ukv.w = b.mat({mx + "uk", mx + "uv"}, {(int64_t)H * nope, nv}, h.kv_rank, ws * 4));
+      L.lat_uk.N = h.kv_rank; L.lat_uk.K = nope;
+      if (b.dummy()) HB_OK(L.lat_uk.w = b.mat({}, {(int64_t)H * h.kv_rank}, nope, ws * 4));
+      else {
+        std::vector<float> uk, tr((size_t)H * h.kv_rank * nope);
+        if (!b.stack({mx + "uk"}, {(int64_t)H * nope}, h.kv_rank, &uk)) return fail(b.err);
+        for (int x = 0; x < H; ++x)
+          for (int n = 0; n < nope; ++n)
+            for (int r = 0; r < h.kv_rank; ++r) tr[((size_t)x * h.kv_rank + r) * nope + n] = uk[((size_t)x * nope + n) * h.kv_rank + r];
+        HB_OK(L.lat_uk.w = b.upload(tr));
+      }
+      if (h.sink) HB_OK(L.sinks = b.vec_f32(mx + "sink", H, 0.f));
+      if (h.rot_dims > 0) {
+        std::vector<double> fr((size_t)h.rot_dims / 2);
+        rotary_frequencies(h.rot_dims, h.rot_base, h.yarn_factor, h.yarn_original, h.yarn_fast, h.yarn_slow, fr.data(), &L.rot_mult);
+        HB_OK(L.rot_freq = b.upload_raw(fr));
+      }
+      L.o.N = d; L.o.K = nv;
+      HB_OK(L.o.w = b.mat({mx + "o"}, {d}, nv, ws));
+      max_proj = std::max(max_proj, L.proj.N); max_mix = std::max(max_mix, nv);
+      max_abs = std::max(max_abs, H * row); max_olat = std::max(max_olat, H * h.kv_rank);
+      max_exp_row = std::max(max_exp_row, L.lat_ukv.N); max_kvr = std::max(max_kvr, h.kv_rank); max_exp_k = std::max(max_exp_k, H * h.dim); max_exp_v = std::max(max_exp_v, nv);
+      max_win = std::max(max_win, h.window > 0 ? h.window : 1 << 30);
+      lat_tc = lat_tc && latent_expand_ok(e, h, L.proj.N);
+      for (int B = 1; B <= e->cfg.max_num_seqs; ++B)
+        lat_ws = std::max(lat_ws, latent_mqa_workspace(B, H, h.kv_rank, latent_mqa_splits(B, H, 1, (int64_t)1 << 30)));
+    } else if (h.mixer == HybridLayerSpec::DELTA) {
+      const int H = h.heads, nk = h.kv_heads * h.dim, nv = H * h.vdim, na = H * h.dim, C = 2 * nk + nv;
+      int ra = h.decay_rank > 0 ? h.decay_rank : h.dim, rg = ra;      // ranks of the low-rank pairs: the checkpoint's shapes
+      if (!b.dummy()) {
+        const HostTensor *t1 = md.find(mx + "a1"), *t2 = md.find(mx + "g1");
+        if (!t1 || t1->shape.size() != 2 || !t2 || t2->shape.size() != 2) return fail("missing tensor " + mx + "a1 / g1");
+        ra = (int)t1->shape[0]; rg = (int)t2->shape[0];
+      }
+      L.off_k = nk; L.off_v = 2 * nk; L.off_a1 = C; L.off_mg = C + ra; L.off_b = C + ra + rg;
+      L.proj.N = L.off_b + H; L.proj.K = d;
+      HB_OK(L.proj.w = b.mat({mx + "q", mx + "k", mx + "v", mx + "a1", mx + "g1", mx + "b"}, {nk, nk, nv, ra, rg, H}, d, ws));
+      if (b.dummy()) HB_OK(L.conv_w = b.mat({}, {C}, h.conv, 0.5f));
+      else {
+        std::vector<float> cw, tr((size_t)C * h.conv);
+        if (!b.stack({mx + "q.conv", mx + "k.conv", mx + "v.conv"}, {nk, nk, nv}, h.conv, &cw)) return fail(b.err);
+        for (int c = 0; c < C; ++c) for (int j = 0; j < h.conv; ++j) tr[(size_t)j * C + c] = cw[(size_t)c * h.conv + j];
+        HB_OK(L.conv_w = b.upload(tr));
+      }
+      L.wkv_w2.N = na; L.wkv_w2.K = ra;
+      HB_OK(L.wkv_w2.w = b.mat({mx + "a2"}, {na}, ra, ws));
+      HB_OK(L.wkv_w2.b = b.mat({mx + "dt_bias"}, {na}, 1, 0.f, -1.f));
+      {
+        std::vector<float> al((size_t)H, -1.f), cf((size_t)na);
+        if (!b.dummy() && !b.stack({mx + "A_log"}, {H}, 1, &al)) return fail(b.err);
+        for (int n = 0; n < na; ++n) cf[n] = expf(al[n / h.dim]);
+        HB_OK(L.decay_coef = b.upload_raw(cf));
+      }
+      L.g2.N = nv; L.g2.K = rg;
+      HB_OK(L.g2.w = b.mat({mx + "g2"}, {nv}, rg, ws));
+      {
+        // the per-head norm of the read-out: one weight of vdim numbers, laid out once per head
+        std::vector<std::string> rep((size_t)H, mx + "norm");
+        std::vector<int64_t> lead((size_t)H, h.vdim);
+        HB_OK(L.wkv_norm = b.mat(rep, lead, 1, 0.f, 1.f));
+      }
+      L.o.N = d; L.o.K = nv;
+      HB_OK(L.o.w = b.mat({mx + "o"}, {d}, nv, ws));
+      state_floats += align_up64(short_conv_state_floats(C, h.conv), 4) + align_up64(delta_state_floats(H, h.dim, h.vdim), 4);      // both start 16-byte aligned
+      max_proj = std::max(max_proj, L.proj.N); max_qkv32 = std::max(max_qkv32, (int)align_up64(C, 4)); max_gate = std::max(max_gate, na); max_mo = std::max(max_mo, nv);
+      max_u = std::max(max_u, nv); max_mix = std::max(max_mix, nv);
     } else if (h.mixer == HybridLayerSpec::LATENT) {
       const int nope = h.dim - h.rot_part, nq = h.heads * h.dim, nkv = h.kv_rank + h.rot_part, nv = h.heads * h.vdim;
       if (h.q_rank > 0) {
@@ -385,8 +480,9 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
       HB_OK(L.down.w = b.mat({fp + "down"}, {d}, h.ff, ws));
       max_ff = std::max(max_ff, h.ff);
     } else if (h.mlp == HybridLayerSpec::MOE) {
-      L.router.N = h.experts; L.router.K = d;
-      HB_OK(L.router.w = b.mat({fp + "router"}, {h.experts}, d, ws * 4));
+      L.router.N = h.experts + h.identity; L.router.K = d;
+      HB_OK(L.router.w = b.mat({fp + "router"}, {L.router.N}, d, ws * 4));
+      if (h.router_correction) HB_OK(L.router_corr = b.vec_f32(fp + "correction", L.router.N, 0.f));
       if (h.router_bias) HB_OK(L.router_b = b.mat({fp + "router.b"}, {h.experts}, 1, 0.f, 0.f));
       // per expert [gate | up] rows in one block (what the fused gated GEMM reads), then all experts' down matrices
       std::vector<std::string> gu, dn;
@@ -409,11 +505,11 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
         if (h.shared_gate) HB_OK(L.s_sg = b.mat({fp + "shared.sg"}, {1}, d, ws));
         max_ff = std::max(max_ff, h.shared_ff);
       }
-      max_top = std::max(max_top, h.top); max_eff = std::max(max_eff, h.expert_ff); max_E = std::max(max_E, h.experts);
+      max_top = std::max(max_top, h.top); max_eff = std::max(max_eff, h.expert_ff); max_E = std::max(max_E, h.experts + h.identity);
     }
   }
 #undef HB_OK
-  e->slot_stride = std::max<int64_t>(state_floats, 1);
+  e->slot_stride = std::max<int64_t>(s.hyb_noprenorm ? align_up64(state_floats, 4) : state_floats, 1);
 
   const int Tm = e->cfg.max_num_batched_tokens, Rm = e->cfg.max_num_seqs, es = b.esz();
   // 16-bit logits rows: straight out of the tensor-core GEMM when its shapes allow (then the row stride is the
@@ -427,6 +523,29 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
   if (max_hd > 0) {
     e->mixes = aalloc((int64_t)5 * Tm * d, es); e->rkvg = aalloc((int64_t)4 * Tm * max_hd, es);
     if (!e->mixes || !e->rkvg) return fail(b.err);
+  }
+  if (max_qkv32 > 0) { e->qkv32 = (float*)aalloc((int64_t)Tm * max_qkv32, 4); if (!e->qkv32) return fail(b.err); }
+  if (max_abs > 0) {
+    // rows of a step that attend in the latent space: all of them, or (prompt pieces on the expanded path) one per request
+    e->latq_rows = lat_tc ? std::min(Rm, Tm) : Tm;
+    e->qabs = aalloc((int64_t)e->latq_rows * max_abs, es); e->olat = aalloc((int64_t)e->latq_rows * max_olat, es);
+    if (!e->qabs || !e->olat) return fail(b.err);
+    if (lat_ws > 0) { e->ws_lat_bytes = lat_ws; e->ws_lat = aalloc(lat_ws, 1); if (!e->ws_lat) return fail(b.err); }
+    if (lat_tc) {
+      // scratch pages for the expanded path: any single request of a step fits (its new rows, the window before them and the
+      // rounding to pages and 64-key tiles); steps with more requests go through it in groups
+      const int bs = e->cfg.block_size;
+      const int64_t rows = (int64_t)Tm + std::min<int64_t>(max_win, e->cfg.max_model_len) + 64 + 2 * bs;
+      const int mb = (e->cfg.max_model_len + bs - 1) / bs;
+      e->exp_pages = (int)((rows + bs - 1) / bs);
+      const int64_t er = (int64_t)e->exp_pages * bs;
+      e->exp_c = aalloc(er * max_kvr, es); e->exp_kv = aalloc(er * max_exp_row, es);
+      e->exp_k = aalloc(er * max_exp_k, es); e->exp_v = aalloc(er * max_exp_v, es);
+      e->exp_table = (int32_t*)aalloc((int64_t)Rm * mb, 4); e->exp_src = (int32_t*)aalloc(e->exp_pages, 4);
+      if (!e->exp_c || !e->exp_kv || !e->exp_k || !e->exp_v || !e->exp_table || !e->exp_src) return fail(b.err);
+      cudaMemsetAsync(e->exp_k, 0, (size_t)er * max_exp_k * es, e->stream);
+      cudaMemsetAsync(e->exp_v, 0, (size_t)er * max_exp_v * es, e->stream);
+    }
   }
   if (max_lkv > 0) {
     e->latq = aalloc((int64_t)Tm * std::max(max_qr, 1), es); e->latc = aalloc((int64_t)Tm * max_kvr, es);
@@ -461,6 +580,8 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
       if (!e->moe_xperm || !e->moe_operm || cudaMallocHost((void**)&e->moe_goff_host, (size_t)(max_E + 1) * 4) != cudaSuccess) return fail("expert staging allocation failed: " + b.err);
     }
     e->moe_goff = (int32_t*)aalloc(max_E + 1, 4);
+    e->moe_prow = (int32_t*)aalloc(np, 4);
+    if (!e->moe_prow) return fail(b.err);
     e->moe_ptok = (int32_t*)aalloc(np, 4); e->moe_pdest = (int32_t*)aalloc(np, 4); e->moe_cexp = (int32_t*)aalloc(np, 4);
     e->moe_pw = (float*)aalloc(np, 4); e->moe_cw = (float*)aalloc(np, 4);
     if (!e->moe_hidden || !e->moe_out || !e->moe_goff || !e->moe_ptok || !e->moe_pdest || !e->moe_cexp || !e->moe_pw || !e->moe_cw) return fail(b.err);
@@ -469,7 +590,7 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
     // split-KV scratch of the TMA-staged decode attention, for attention mixers whose heads it takes
     int64_t need = 0;
     for (auto& h : s.hybrid)
-      if ((h.mixer == HybridLayerSpec::ATTENTION || h.mixer == HybridLayerSpec::LATENT) && !e->f32 && (h.dim == 64 || h.dim == 128) && h.vdim == h.dim)
+      if ((h.mixer == HybridLayerSpec::ATTENTION || (h.mixer == HybridLayerSpec::LATENT && !h.latent_cache)) && !e->f32 && (h.dim == 64 || h.dim == 128) && h.vdim == h.dim)
         need = std::max<int64_t>(need, kge_attn_workspace_bytes(Rm, h.heads, h.dim, e->cfg.max_model_len));
     if (need > 0) {
       e->ws_attn_bytes = need;
@@ -500,7 +621,7 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
   // paged caches of the attention sides: K [blocks, G, block_size, dim], V [blocks, G, block_size, vdim] per layer
   int64_t blk_bytes = 0;
   for (auto& h : s.hybrid)
-    if (h.has_cache()) blk_bytes += (int64_t)h.kv_heads * (e->cfg.block_size + (h.pool > 0 ? pool_slots_per_block(e->cfg.block_size, h.pool) : 0)) * (h.dim + h.vdim) * es;
+    if (h.has_cache()) blk_bytes += (e->cfg.block_size + (h.pool > 0 ? pool_slots_per_block(e->cfg.block_size, h.pool) : 0)) * (h.cache_k_row() + h.cache_v_row()) * es;
   int nb = e->cfg.num_blocks;
   if (nb <= 0) {
     const int64_t cap = (int64_t)e->cfg.max_num_seqs * e->max_blocks_per_seq + 1;
@@ -522,11 +643,12 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
   for (int i = 0; i < s.L; ++i) {
     const HybridLayerSpec& h = s.hybrid[i];
     if (!h.has_cache()) continue;
-    const int64_t nk = (int64_t)nb * h.kv_heads * e->cfg.block_size * h.dim, nv = (int64_t)nb * h.kv_heads * e->cfg.block_size * h.vdim;
-    e->hyb[i].kc = aalloc(nk, es); e->hyb[i].vc = aalloc(nv, es);
-    if (!e->hyb[i].kc || !e->hyb[i].vc) return fail("KV pool allocation failed");
+    const int64_t nk = (int64_t)nb * e->cfg.block_size * h.cache_k_row(), nv = (int64_t)nb * e->cfg.block_size * h.cache_v_row();
+    e->hyb[i].kc = aalloc(nk, es);
+    if (nv > 0) e->hyb[i].vc = aalloc(nv, es);      // cached latents: one row per token is key and value
+    if (!e->hyb[i].kc || (nv > 0 && !e->hyb[i].vc)) return fail("KV pool allocation failed");
     cudaMemsetAsync(e->hyb[i].kc, 0, (size_t)nk * es, e->stream);
-    cudaMemsetAsync(e->hyb[i].vc, 0, (size_t)nv * es, e->stream);
+    if (nv > 0) cudaMemsetAsync(e->hyb[i].vc, 0, (size_t)nv * es, e->stream);
     if (h.pool > 0) {
       // one pooled key / value per block of `pool` positions, on the same pages: entry b of a request lives in its page b / slots
       const int ps = pool_slots_per_block(e->cfg.block_size, h.pool);
@@ -617,8 +739,15 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
     return stream_norm(sn, st);
   };
   if (hyper) HFWD(C_EMBED, Td * (es + 4.0 * S), 0, embed_norm_streams(e->res32, m.ids, e->embed, s.embed_norm ? e->embed_norm_w : nullptr, T, d, S, s.eps, elt, st));
-  else HFWD(C_EMBED, Td * (es + 4), 0, embed_f32(e->res32, m.ids, e->embed, T, d, elt, st));
-  bool hx_ready = false;      // the previous layer's last write of the streams already formed this layer's normed input
+  else if (s.hyb_noprenorm) {
+    // the first sublayer reads the stream itself: its input is written along with it
+    BigramArgs ba;
+    ba.res = e->res32; ba.y = e->hx; ba.ids = m.ids; ba.table = e->embed; ba.bigram = e->bigram; ba.buckets = s.bigram_buckets; ba.mul_prev = s.bigram_mul_prev; ba.mul_cur = s.bigram_mul_cur;
+    ba.state = e->state; ba.slot_stride = e->slot_stride; ba.slots = m.sslot; ba.qsl = m.qsl; ba.positions = m.pos; ba.token_req = m.treq;
+    ba.B = B; ba.T = T; ba.d = d; ba.inline_save = decode_only; ba.elt = elt;
+    HFWD(C_EMBED, Td * (3 * es + 4), 0, embed_bigram(ba, st));
+  } else HFWD(C_EMBED, Td * (es + 4), 0, embed_f32(e->res32, m.ids, e->embed, T, d, elt, st));
+  bool hx_ready = s.hyb_noprenorm;      // the previous layer's last write of the streams already formed this layer's normed input
   for (int i = 0; i < s.L; ++i) {
     const HybridLayerSpec& h = s.hybrid[i];
     const HybridLayerW& L = e->hyb[i];
@@ -627,6 +756,7 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
     hx_ready = false;
     CombineArgs cb;
     const void* inner_w[2] = {nullptr, nullptr};      // a norm of a source's own before the sources are summed (models with normed results)
+    const void* pair_src = nullptr;                    // the experts' rows a post-norm model gathers by (token, choice) pair
     bool y32_used = false;
     int sub = 0;                                       // the sublayer whose result is being summed (0: mixer, 1: feed-forward)
     auto add_src = [&](const void* p, int ld, float scale, const float* rscale = nullptr, int rs_stride = 0) {
@@ -649,9 +779,11 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
       if (s.hyb_postnorm) {
         // the sublayer's result through its own norm into the stream, and the next sublayer's normed input in the same pass
         PostNormArgs pa;
-        pa.res = e->res32; pa.nsrc = cb.n; pa.src_scale = cb.scale[0]; pa.T = T; pa.d = d; pa.groups = s.norm_groups; pa.eps = s.eps; pa.elt = elt;
+        pa.res = e->res32; pa.nsrc = cb.n; pa.src_scale = cb.n ? cb.scale[0] : 1.f; pa.T = T; pa.d = d; pa.groups = s.norm_groups; pa.eps = s.eps; pa.elt = elt;
         for (int q = 0; q < cb.n && q < 2; ++q) { pa.src[q] = cb.src[q]; pa.ld[q] = cb.ld[q]; pa.inner_w[q] = inner_w[q]; }
         pa.post_w = sub == 0 ? L.norm1b : L.norm2b;
+        pa.pair_src = pair_src; pa.pair_row = pair_src ? e->moe_prow : nullptr; pa.pair_w = e->moe_cw; pa.top = h.top;
+        pair_src = nullptr;
         if (sub == 0 && h.mlp != HybridLayerSpec::NONE) { pa.next_w = L.norm2; pa.next_y = e->hx; }
         else if (i + 1 < s.L) { pa.next_w = e->hyb[i + 1].norm1; pa.next_y = e->hx; hx_ready = true; }
         cb = CombineArgs(); inner_w[0] = inner_w[1] = nullptr;
@@ -767,7 +899,7 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
       HFWD(decode_only ? C_ATT_DEC : C_ATT_GEN, (decode_only ? keys : (double)T) * h.kv_heads * (h.dim + h.vdim) * es + (double)T * h.heads * (h.dim + h.vdim) * es,
            2.0 * keys * h.heads * (h.dim + h.vdim),
            tc ? paged_attn_window_tc(e->mixbuf, qkv, ldq, L.kc, L.vc, L.pkc, L.pvc, m.btab, max_blocks, m.seq_lens, m.qsl, B, aa.max_q, h.heads, h.kv_heads, h.dim, bs,
-                                     h.scale, h.window, h.keep_first, h.pool, ps, st)
+                                     h.scale, h.window, h.keep_first, h.pool, ps, nullptr, st)
               : attn_bias_chunk(aa, st));
       if (h.v_rot) HFWD(C_ACT, (double)T * ka * 2 * es, 0, rotate_heads_halves(e->mixbuf, ka, m.pos, L.v_freq, T, h.heads, h.vdim, -1.f, elt, st));
       DENSE(e->obuf1, d, e->mixbuf, ka, L.o, T, ACT_NONE);
@@ -823,6 +955,117 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
       HFWD(C_MLSTM, 2.0 * B * h.heads * (double)h.dim * h.dim * 4 + (double)T * hd * (5 * es + 12), 4.0 * T * h.heads * (double)h.dim * h.dim, wkv_scan(wa, st));
       ++e->launches;
       DENSE(e->obuf1, d, e->mixbuf, hd, L.o, T, ACT_NONE);
+      add_src(e->obuf1, d, 1.f);
+    } else if (h.mixer == HybridLayerSpec::LATENT && h.latent_cache) {
+      const int H = h.heads, nope = h.dim - h.rot_part, rank = h.kv_rank, row = rank + h.rot_part, nv = H * h.vdim, ldp = L.proj.N;
+      void* cache = h.kv_from >= 0 ? e->hyb[h.kv_from].kc : L.kc;      // the rows of the layer that owns the latents
+      const int window = h.window;
+      DENSE(e->pbuf, ldp, e->hx, d, L.proj, T, ACT_NONE);                // [q | dkv], or the queries alone
+      int D = 0, maxq = 1;
+      while (D < B && hm.qsl[D + 1] - hm.qsl[D] == 1) ++D;
+      for (int r = 0; r < B; ++r) maxq = std::max(maxq, hm.qsl[r + 1] - hm.qsl[r]);
+      // prompt pieces: keys and values of the pages they can see expanded from the latents for the tcgen05 kernel, when its
+      // sizes allow; single tokens (and everything else) attend to the latent rows themselves
+      const bool expand = !decode_only && e->exp_pages > 0;
+      const int Ta = expand ? D : T;                                     // rows that attend in the latent space
+      KGE_REQUIRE(Ta <= e->latq_rows, "hybrid_forward: %d rows in the latent space", Ta);
+      LatentCacheArgs lc;
+      lc.z = h.kv_from >= 0 ? nullptr : at(e->pbuf, L.lat_dkv); lc.ldz = ldp; lc.norm_w = L.lat_kvnorm; lc.eps = s.eps; lc.q = e->pbuf; lc.ldq = ldp; lc.q_abs = e->qabs; lc.q_abs_rows = Ta;
+      lc.freq = L.rot_freq; lc.mult = L.rot_mult; lc.rot_dims = h.rot_dims; lc.rot_part = h.rot_part; lc.kv_rank = rank; lc.positions = m.pos; lc.slots = m.slots; lc.cache = cache;
+      lc.T = T; lc.H = H; lc.dim = h.dim; lc.elt = elt;
+      HFWD(C_KVW, (double)T * (2.0 * H * h.rot_part + (h.kv_from >= 0 ? 0.0 : 2.0 * row)) * es + (double)Ta * H * h.rot_part * es, 0, latent_cache_write(lc, st));
+      double keys = 0, keys_abs = 0;                                     // visible keys over all rows / over the rows in the latent space
+      for (int t = 0; t < T; ++t) { const double k = window > 0 ? std::min(hm.pos[t] + 1, window) : hm.pos[t] + 1; keys += k; if (t < Ta) keys_abs += k; }
+      if (Ta > 0) {
+        LinearArgs qa;       // every head's query through the head's key up-projection
+        qa.x = e->pbuf; qa.ldx = ldp; qa.x_zs = h.dim; qa.w = L.lat_uk.w; qa.w_zs = (int64_t)rank * nope; qa.y = e->qabs; qa.ldy = H * row; qa.y_zs = row;
+        qa.T = Ta; qa.N = rank; qa.K = nope; qa.nz = H; qa.elt = elt; qa.out_f32 = e->f32;
+        HFWD(C_GEMM_S, es * ((double)H * rank * nope + (double)Ta * H * (nope + rank)), 2.0 * Ta * H * (double)rank * nope, linear_any(qa, st));
+        const double ab = (double)keys_abs / std::max(1, decode_only ? 1 : 16) * row * es + (double)Ta * H * (row + rank) * es, af = 2.0 * keys_abs * H * (row + rank);
+        const int cat = decode_only ? C_ATT_DEC : C_ATT_GEN;
+        if (!e->f32 && latent_mqa_ok(H, rank, h.rot_part, bs) && row > 128) {
+          LatentMqaArgs la;
+          la.q = e->qabs; la.out = e->olat; la.cache = cache; la.block_table = m.btab; la.max_blocks = max_blocks; la.qsl = m.qsl; la.positions = m.pos;
+          la.H = H; la.kv_rank = rank; la.rot_part = h.rot_part; la.block_size = bs; la.window = window; la.scale = h.scale; la.sinks = L.sinks; la.T = Ta;
+          la.workspace = e->ws_lat; la.workspace_bytes = e->ws_lat_bytes;
+          if (D > 0) {                                                   // one token each: the key range split over CTAs
+            la.req0 = 0; la.B = D; la.max_q = 1; la.T = D;
+            // a decode step may be replayed as a graph while its contexts grow: sized for the longest context its table holds
+            la.splits = latent_mqa_splits(D, H, 1, std::min<int64_t>(window > 0 ? window : (int64_t)1 << 30, (int64_t)max_blocks * bs));
+            HFWD(cat, ab, af, latent_mqa(la, st));
+            if (la.splits > 1) ++e->launches;
+          }
+          if (Ta > D) {
+            la.req0 = D; la.B = B - D; la.max_q = maxq; la.splits = 1; la.T = Ta;
+            HFWD(cat, ab, af, latent_mqa(la, st));
+          }
+        } else {
+          AttnBiasArgs aa;                                               // all heads on one key/value head whose values are the rows' first numbers
+          aa.q = e->qabs; aa.ldq = H * row; aa.out = e->olat; aa.ldo = H * rank; aa.k_cache = aa.v_cache = cache; aa.v_ld = row;
+          aa.block_table = m.btab; aa.max_blocks = max_blocks; aa.seq_lens = m.seq_lens; aa.qsl = m.qsl; aa.positions = m.pos; aa.token_req = m.treq;
+          aa.B = B; aa.T = Ta; aa.H = H; aa.G = 1; aa.dim = row; aa.vdim = rank; aa.block_size = bs; aa.window = window; aa.scale = h.scale; aa.sinks = L.sinks; aa.elt = elt;
+          if (Ta < T) aa.B = D;
+          aa.num_decode = D; aa.max_q = Ta < T ? 1 : maxq;
+          HFWD(cat, ab, af, attn_bias_chunk(aa, st));
+        }
+        LinearArgs va;       // the heads' latent averages through their value up-projections
+        va.x = e->olat; va.ldx = H * rank; va.x_zs = rank; va.w = at(L.lat_ukv.w, (int64_t)H * nope * rank); va.w_zs = (int64_t)h.vdim * rank; va.y = e->mixbuf; va.ldy = nv; va.y_zs = h.vdim;
+        va.T = Ta; va.N = h.vdim; va.K = rank; va.nz = H; va.elt = elt; va.out_f32 = e->f32;
+        HFWD(C_GEMM_S, es * ((double)H * rank * h.vdim + (double)Ta * H * (rank + h.vdim)), 2.0 * Ta * H * (double)rank * h.vdim, linear_any(va, st));
+      }
+      if (expand) {
+        const int win = window > 0 ? window : 1 << 30;
+        for (int r0 = D; r0 < B;) {
+          int n = 0, pages = 0, mq = 1;
+          double gkeys = 0;
+          for (; r0 + n < B; ++n) {                                      // the requests whose pages fit the scratch together
+            const int q = hm.qsl[r0 + n + 1] - hm.qsl[r0 + n], sl = hm.seq_lens[r0 + n];
+            const int p = (sl - 1) / bs - latent_expand_first_page(sl - q, win, bs) + 1;
+            if (n > 0 && pages + p > e->exp_pages) break;
+            pages += p; mq = std::max(mq, q);
+            for (int t = hm.qsl[r0 + n]; t < hm.qsl[r0 + n + 1]; ++t) gkeys += std::min(hm.pos[t] + 1, win);
+          }
+          KGE_REQUIRE(pages <= e->exp_pages, "hybrid_forward: a request sees %d pages of %d", pages, e->exp_pages);
+          const double er = (double)pages * bs;
+          HFWD(C_KVW, 0, 0, latent_expand_plan(e->exp_table, e->exp_src, m.btab, max_blocks, m.qsl, m.seq_lens, r0, n, win, bs, pages, st));
+          HFWD(C_KVW, er * rank * 2 * es, 0, latent_gather(e->exp_c, cache, e->exp_src, pages, bs, rank, row, elt, st));
+          DENSE(e->exp_kv, L.lat_ukv.N, e->exp_c, rank, L.lat_ukv, pages * bs, ACT_NONE);
+          HFWD(C_KVW, er * (L.lat_ukv.N + H * (h.dim + h.vdim) + h.rot_part) * es, 0,
+               latent_expand_write(e->exp_k, e->exp_v, e->exp_kv, cache, e->exp_src, pages, bs, H, h.dim, h.vdim, rank, h.rot_part, elt, st));
+          HFWD(C_ATT_GEN, er * H * (h.dim + h.vdim) * es + (double)(hm.qsl[r0 + n] - hm.qsl[r0]) * H * (h.dim + h.vdim) * es, 2.0 * gkeys * H * (h.dim + h.vdim),
+               paged_attn_window_tc(e->mixbuf, e->pbuf, ldp, e->exp_k, e->exp_v, nullptr, nullptr, e->exp_table, max_blocks, m.seq_lens + r0, m.qsl + r0, n, mq, H, H, h.dim, bs, h.scale,
+                                    win, 0, 0, 0, L.sinks, st));
+          r0 += n;
+        }
+      }
+      DENSE(e->obuf1, d, e->mixbuf, nv, L.o, T, ACT_NONE);
+      add_src(e->obuf1, d, 1.f);
+    } else if (h.mixer == HybridLayerSpec::DELTA) {
+      const int H = h.heads, G = h.kv_heads, nk = G * h.dim, nv = H * h.vdim, na = H * h.dim, C = 2 * nk + nv, ldp = L.proj.N, ldc = (int)align_up64(C, 4);
+      DENSE(e->pbuf, ldp, e->hx, d, L.proj, T, ACT_NONE);                // every projection of the row in one product: [q | k | v | a1 | g1 | b]
+      ConvHeadsArgs ca;      // convolution, silu, unit vectors
+      ca.x = e->pbuf; ca.ldx = ldp; ca.y = e->qkv32; ca.ldy = ldc; ca.w = L.conv_w; ca.C = C; ca.taps = h.conv; ca.unit_heads = 2 * G; ca.scaled_heads = G; ca.head_dim = h.dim;
+      ca.head_scale = 1.f / sqrtf((float)h.dim); ca.unit_eps = 1e-6f; ca.state = e->state + L.state_off; ca.slot_stride = e->slot_stride;
+      ca.slots = m.sslot; ca.qsl = m.qsl; ca.positions = m.pos; ca.token_req = m.treq; ca.B = B; ca.T = T; ca.inline_save = decode_only; ca.elt = elt;
+      HFWD(C_RGLRU, (double)T * C * (es + 4), 2.0 * T * C * h.conv, short_conv_silu_heads(ca, st));
+      if (!decode_only && h.conv > 1) ++e->launches;
+      LinearArgs a2;         // the decays: second half of their low-rank pair, bias, softplus and exponentials in the epilogue, fp32
+      a2.x = at(e->pbuf, L.off_a1); a2.ldx = ldp; a2.w = L.wkv_w2.w; a2.bias = L.wkv_w2.b; a2.y = e->gates32; a2.ldy = na; a2.T = T; a2.N = na; a2.K = L.wkv_w2.K;
+      a2.act = ACT_EXP_DECAY; a2.act_coef = L.decay_coef; a2.elt = elt; a2.out_f32 = true;
+      HFWD(C_MLSTM, es * ((double)L.wkv_w2.K * na + (double)T * L.wkv_w2.K) + 4.0 * T * na, 2.0 * T * (double)na * L.wkv_w2.K, linear_any(a2, st));
+      LinearArgs g2;         // the output gate's logits
+      g2.x = at(e->pbuf, L.off_mg); g2.ldx = ldp; g2.w = L.g2.w; g2.y = e->ubuf; g2.ldy = nv; g2.T = T; g2.N = nv; g2.K = L.g2.K; g2.elt = elt; g2.out_f32 = e->f32;
+      HFWD(C_MLSTM, es * ((double)L.g2.K * nv + (double)T * (L.g2.K + nv)), 2.0 * T * (double)nv * L.g2.K, linear_any(g2, st));
+      DeltaArgs da;
+      da.qkv = e->qkv32; da.ld = ldc; da.decay = e->gates32; da.beta_pre = at(e->pbuf, L.off_b); da.ldb = ldp; da.o32 = e->mo32;
+      da.state = e->state + L.state_off + align_up64(short_conv_state_floats(C, h.conv), 4); da.slot_stride = e->slot_stride; da.slots = m.sslot; da.qsl = m.qsl; da.positions = m.pos;
+      da.B = B; da.T = T; da.H = H; da.G = G; da.dim = h.dim; da.vdim = h.vdim; da.elt = elt;
+      HFWD(C_MLSTM, 2.0 * B * delta_state_floats(H, h.dim, h.vdim) * 4 + 4.0 * T * (C + na + nv), 8.0 * T * H * (double)h.dim * h.vdim, delta_scan(da, st));
+      WkvArgs wa;            // per-head norm and the sigmoid gate
+      wa.o32 = e->mo32; wa.norm_w = L.wkv_norm; wa.gate_pre = e->ubuf; wa.ld = nv; wa.out = e->mixbuf; wa.ldo = nv; wa.T = T; wa.H = H; wa.dim = h.vdim; wa.vdim = h.vdim; wa.eps = s.eps;
+      wa.gate_act = ACT_SIGMOID; wa.elt = elt;
+      HFWD(C_MLSTM, (double)T * nv * (4 + 2 * es), 0, wkv_norm_gate(wa, st));
+      DENSE(e->obuf1, d, e->mixbuf, nv, L.o, T, ACT_NONE);
       add_src(e->obuf1, d, 1.f);
     } else if (h.mixer == HybridLayerSpec::LATENT) {
       const int H = h.heads, nope = h.dim - h.rot_part, nq = H * h.dim, nv = H * h.vdim, ldp = L.proj.N, ldkv = L.lat_ukv.N;
@@ -935,7 +1178,9 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
       add_src(e->obuf2, d, 1.f);
     } else if (h.mlp == HybridLayerSpec::MOE) {
       MoeRouteArgs ra;
-      ra.h = e->hx; ra.ldh = d; ra.w_router = L.router.w; ra.b_router = L.router_b; ra.T = T; ra.d = d; ra.E = h.experts; ra.top = h.top;
+      ra.h = e->hx; ra.ldh = d; ra.w_router = L.router.w; ra.b_router = L.router_b; ra.T = T; ra.d = d; ra.E = h.experts + h.identity; ra.top = h.top;
+      ra.correction = L.router_corr; ra.groups = h.router_groups; ra.groups_keep = h.groups_keep; ra.identity = h.identity; ra.pair_row = e->moe_prow;
+      const bool by_pair = s.hyb_postnorm;      // the pass that norms the result gathers the experts' rows itself: they stay in routed order
       const bool w_out = h.route != HybridLayerSpec::ROUTE_SIGMOID_IN;      // the routing weight multiplies the expert's output (in the fp32 sum below)
       const bool clamped = h.glu == HybridLayerSpec::GLU_CLAMPED;
       const bool ungated = h.glu == HybridLayerSpec::GLU_NONE_RELU2;      // one front matrix per expert, relu(.)^2
@@ -962,7 +1207,8 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
              gemm_grouped(e->moe_hidden, e->moe_xperm, L.e_gate, np_pad, eff, d, h.experts, e->moe_tile_group, ungated ? -2 : clamped ? 1 : 0, 1.702f, h.expert_limit, st));
         HFWD(C_MOE, 2.0 * ((double)h.experts * eff * d + (double)np_pad * (d + eff)), 2.0 * np * (double)eff * d,
              gemm_grouped(e->moe_operm, e->moe_hidden, L.e_down, np_pad, d, eff, h.experts, e->moe_tile_group, -1, 0.f, 0.f, st));
-        HFWD(C_MOE, (double)np * d * 4, 0, moe_scatter_rows(e->moe_out, e->moe_operm, e->moe_pdest, np_pad, d, st));
+        if (by_pair) pair_src = e->moe_operm;
+        else HFWD(C_MOE, (double)np * d * 4, 0, moe_scatter_rows(e->moe_out, e->moe_operm, e->moe_pdest, np_pad, d, st));
       } else {
       LinearArgs g;      // experts' gated front half on the gathered, weighted rows
       g.x = e->hx; g.ldx = d; g.w = L.e_gate; g.w2 = L.e_up; g.y = e->moe_hidden; g.ldy = h.expert_ff; g.T = np; g.N = h.expert_ff; g.K = d;
@@ -973,9 +1219,10 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
       HFWD(C_MOE, (ungated ? 1 : 2) * wexp + (double)np * (d + h.expert_ff) * es, (ungated ? 2.0 : 4.0) * np * (double)h.expert_ff * d, linear_any(g, st));
       LinearArgs dn;     // experts' down projection, scattered to row (token * top + choice)
       dn.x = e->moe_hidden; dn.ldx = h.expert_ff; dn.w = L.e_down; dn.y = e->moe_out; dn.ldy = d; dn.T = np; dn.N = d; dn.K = h.expert_ff;
-      dn.nz = h.experts; dn.w_zs = (int64_t)d * h.expert_ff; dn.group_off = e->moe_goff; dn.max_rows = np; dn.yrows = e->moe_pdest;
+      dn.nz = h.experts; dn.w_zs = (int64_t)d * h.expert_ff; dn.group_off = e->moe_goff; dn.max_rows = np; dn.yrows = by_pair ? nullptr : e->moe_pdest;
       dn.elt = elt; dn.out_f32 = e->f32;
       HFWD(C_MOE, wexp + (double)np * (d + h.expert_ff) * es, 2.0 * np * (double)h.expert_ff * d, linear_any(dn, st));
+      if (by_pair) pair_src = e->moe_out;
       }
       if (h.shared_ff > 0) {
         const int f = h.shared_ff;
@@ -995,13 +1242,15 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
         DENSE(e->obuf2, d, e->ffbuf, f, L.s_down, T, ACT_NONE);
       }
       // sum in a fixed order: mixer, the token's experts by choice, the shared expert
-      for (int k = 0; k < h.top; ++k) {
+      for (int k = 0; k < h.top && !by_pair; ++k) {
         if (cb.n == 4) HFWD(C_ACT, Td * (8 + 4 * es), 0, flush_more());
         add_src(at(e->moe_out, (int64_t)k * d), h.top * d, 1.f, w_out ? e->moe_cw + k : nullptr, h.top);
       }
       if (h.shared_ff > 0) { if (cb.n == 4) HFWD(C_ACT, Td * (8 + 4 * es), 0, flush_more()); add_src(e->obuf2, d, 1.f, L.s_sg ? e->gates32 : nullptr, 1); }
     }
-    { const double nsrc = cb.n + (s.hyb_postnorm ? 1 : 0); HFWD(C_ACT, Td * (8.0 * S + nsrc * es), 0, flush()); }      // post-norm models also write the next normed row
+    if (cb.n > 0 || pair_src || s.hyb_noprenorm == false) {      // post-norm models also write the next normed row
+      const double nsrc = cb.n + (pair_src ? h.top : 0) + (s.hyb_postnorm ? 1 : 0); HFWD(C_ACT, Td * (8.0 * S + nsrc * es), 0, flush());
+    }
     if (e->layer_dump_host && (int64_t)(i + 1) * T * d <= e->layer_dump_cap) {
       if (hyper) { if (int rc = stream_read(nullptr, nullptr, nullptr, nullptr, T, 1.f, e->y32)) return rc; }      // the sum of the streams
       KGE_CUDA_OK(cudaMemcpyAsync(e->layer_dump_host + (int64_t)i * T * d, hyper ? e->y32 : e->res32, (size_t)T * d * 4, cudaMemcpyDeviceToHost, st));

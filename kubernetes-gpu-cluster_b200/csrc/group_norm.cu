@@ -55,6 +55,27 @@ __global__ void __launch_bounds__(GN_THREADS) postnorm_residual_kernel(PostNormA
   float* yb = gn_sm + d;             // the second source
   __shared__ float inv[GN_MAX_GROUPS], red[33];
   float f[2] = {1.f, 1.f};
+  if (a.pair_row) {
+    // the token's experts in choice order; an expert without tensors returns the stream's own row
+    const int32_t* pr = a.pair_row + (int64_t)t * a.top;
+    const float* pw = a.pair_w + (int64_t)t * a.top;
+    const float* x = a.res + (int64_t)t * d;
+    for (int c = threadIdx.x * W; c < d; c += GN_THREADS * W) {
+      float s[4] = {0.f, 0.f, 0.f, 0.f}, xr[4];
+      if (VEC) ld4(x + c, xr); else xr[0] = x[c];
+#pragma unroll 4
+      for (int k = 0; k < a.top; ++k) {
+        const int r = pr[k];
+        const float wk = pw[k];
+        float v[4] = {xr[0], xr[1], xr[2], xr[3]};
+        if (r >= 0) { const E* src = (const E*)a.pair_src + (int64_t)r * d + c; if (VEC) ld4(src, v); else v[0] = ldf(src); }
+#pragma unroll
+        for (int q = 0; q < W; ++q) s[q] = fmaf(wk, v[q], s[q]);
+      }
+#pragma unroll
+      for (int q = 0; q < W; ++q) ya[c + q] = s[q];
+    }
+  }
   for (int i = 0; i < a.nsrc; ++i) {
     const E* s = (const E*)a.src[i] + (int64_t)t * a.ld[i];
     float* dst = i ? yb : ya;
@@ -68,6 +89,7 @@ __global__ void __launch_bounds__(GN_THREADS) postnorm_residual_kernel(PostNormA
     if (a.inner_w[i]) f[i] = 1.f / sqrtf(block_sum(ss, red) / (float)d + a.eps);
   }
   __syncthreads();
+  if (a.nsrc > 1 || a.inner_w[0] || a.src_scale != 1.f) {
   for (int c = threadIdx.x * W; c < d; c += GN_THREADS * W) {
     float w0[4] = {1.f, 1.f, 1.f, 1.f}, w1[4] = {1.f, 1.f, 1.f, 1.f};
     if (a.inner_w[0]) { if (VEC) ld4((const E*)a.inner_w[0] + c, w0); else w0[0] = ldf((const E*)a.inner_w[0] + c); }
@@ -80,6 +102,7 @@ __global__ void __launch_bounds__(GN_THREADS) postnorm_residual_kernel(PostNormA
     }
   }
   __syncthreads();
+  }
   group_inv_rms(ya, d, a.groups, a.eps, inv);
   __syncthreads();
   float* res = a.res + (int64_t)t * d;
@@ -91,11 +114,20 @@ __global__ void __launch_bounds__(GN_THREADS) postnorm_residual_kernel(PostNormA
     for (int k = 0; k < W; ++k) { r[k] += ya[c + k] * gi * w[k]; ya[c + k] = r[k]; }
     if (VEC) st4(res + c, r); else res[c] = r[0];
   }
-  if (!a.next_w) return;
+  if (!a.next_y) return;
+  E* ny = (E*)a.next_y + (int64_t)t * d;
+  if (!a.next_w) {                     // the next sublayer reads the stream itself (each thread rereads the columns it wrote)
+    for (int c = threadIdx.x * W; c < d; c += GN_THREADS * W) {
+      float o[4];
+#pragma unroll
+      for (int k = 0; k < W; ++k) o[k] = ya[c + k];
+      if (VEC) st4(ny + c, o); else stf(ny + c, o[0]);
+    }
+    return;
+  }
   __syncthreads();
   group_inv_rms(ya, d, a.groups, a.eps, inv);
   __syncthreads();
-  E* ny = (E*)a.next_y + (int64_t)t * d;
   for (int c = threadIdx.x * W; c < d; c += GN_THREADS * W) {
     float w[4], o[4];
     if (VEC) ld4((const E*)a.next_w + c, w); else w[0] = ldf((const E*)a.next_w + c);
@@ -142,11 +174,11 @@ int group_rmsnorm_f32in(void* y, const float* x, const int32_t* rows, const void
 
 int postnorm_residual(const PostNormArgs& a, cudaStream_t st) {
   if (a.T <= 0) return 0;
-  KGE_REQUIRE(a.groups >= 1 && a.groups <= GN_MAX_GROUPS && a.d % a.groups == 0 && a.d <= 25600 && a.nsrc >= 1 && a.nsrc <= 2 && a.post_w,
+  KGE_REQUIRE(a.groups >= 1 && a.groups <= GN_MAX_GROUPS && a.d % a.groups == 0 && a.d <= 25600 && (a.pair_row ? a.nsrc == 0 && a.pair_src && a.pair_w && a.top > 0 && a.src_scale == 1.f : a.nsrc >= 1 && a.nsrc <= 2) && a.post_w,
               "postnorm_residual: %d groups of a row of %d, %d sources", a.groups, a.d, a.nsrc);
   const size_t smem = (size_t)a.d * 8;
   bool vec = a.d % 4 == 0 && (a.d / a.groups) % 4 == 0 && ((uintptr_t)a.res & 15) == 0 && ((uintptr_t)a.post_w & 15) == 0 &&
-             (!a.next_w || ((((uintptr_t)a.next_w | (uintptr_t)a.next_y) & 15) == 0));
+             (((uintptr_t)a.next_w | (uintptr_t)a.next_y | (uintptr_t)a.pair_src) & 15) == 0;
   for (int i = 0; i < a.nsrc; ++i) vec = vec && a.ld[i] % 4 == 0 && ((uintptr_t)a.src[i] & 15) == 0 && (!a.inner_w[i] || ((uintptr_t)a.inner_w[i] & 15) == 0);
   if (a.elt == KGE_ELT_F32) {
     if (int rc = opt_in_smem(postnorm_residual_kernel<float, false>, smem)) return rc;

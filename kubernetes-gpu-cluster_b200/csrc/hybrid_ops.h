@@ -4,7 +4,7 @@
 // mixture-of-experts router, the hyper-connected residual (several streams), the WKV recurrence (also run as gated linear
 // attention), the row-wise parts of attention through latents, sliding windows with kept first tokens or pooled blocks,
 // short causal convolutions with a state, per-head norms with rotary positions in halves and rotated values, and grouped
-// RMS norms before and after a sublayer.  Every mechanism takes its sizes and constants
+// RMS norms before and after a sublayer, a bigram embedding, attention over cached latents, and a gated delta rule.  Every mechanism takes its sizes and constants
 // as arguments.  `elt` names the storage type of activations and weights: KGE_ELT_BF16 or KGE_ELT_F32; what the
 // mechanisms compute in 32 bits (softmax, norms, routers, residual sums, recurrent state and everything that enters a
 // recurrence besides projections and short convolutions) is 32-bit in both.
@@ -12,10 +12,16 @@
 #include <cuda_runtime.h>
 #include <stdint.h>
 
+#ifdef __CUDACC__
+#define KGE_HD __host__ __device__
+#else
+#define KGE_HD
+#endif
+
 namespace kge {
 
 enum { KGE_ELT_BF16 = 0, KGE_ELT_F32 = 1 };
-enum { ACT_NONE = 0, ACT_GELU_ERF = 1, ACT_GELU_TANH = 2, ACT_SILU = 3, ACT_SIGMOID = 4, ACT_TANH = 5, ACT_RELU2 = 6 };
+enum { ACT_NONE = 0, ACT_GELU_ERF = 1, ACT_GELU_TANH = 2, ACT_SILU = 3, ACT_SIGMOID = 4, ACT_TANH = 5, ACT_RELU2 = 6, ACT_EXP_DECAY = 7 };
 
 inline size_t elt_size(int elt) { return elt == KGE_ELT_F32 ? 4 : 2; }
 
@@ -38,6 +44,7 @@ struct LinearArgs {
   const int32_t* xrows = nullptr; const int32_t* yrows = nullptr;
   const float* row_scale = nullptr;
   int act = ACT_NONE; float alpha = 1.f; bool accumulate = false;
+  const float* act_coef = nullptr;        // ACT_EXP_DECAY: exp(-act_coef[n] * softplus(v)), one fp32 number per output column
   int glu = 0; float glu_alpha = 1.702f, glu_limit = 0.f;      // gated pairs: GLU_SILU_MUL or GLU_CLAMPED_SIGMOID
   int elt = KGE_ELT_BF16; bool out_f32 = false;
 };
@@ -46,6 +53,19 @@ int linear_any(const LinearArgs& a, cudaStream_t st);
 
 // res[t, :] = float(table[ids[t], :])
 int embed_f32(float* res, const int32_t* ids, const void* table, int T, int d, int elt, cudaStream_t st);
+// Token embedding plus a row of a second table picked by the token and the one before it: with p the previous token of the
+// sequence, res[t, :] = float(table[ids[t], :]) + float(bigram[(p * mul_prev + ids[t] * mul_cur) mod buckets, :]), a sequence's
+// first token (position 0) taking row `buckets` (bigram null: the token's row alone, no state); y (elt, optional) receives the same row.  The token before a request's
+// first row of the step is kept in its state slot (one 32-bit word at `state`), which afterwards holds the last one.
+struct BigramArgs {
+  float* res = nullptr; void* y = nullptr; const int32_t* ids = nullptr; const void* table = nullptr; const void* bigram = nullptr;
+  int64_t buckets = 1, mul_prev = 0, mul_cur = 0;
+  float* state = nullptr; int64_t slot_stride = 0;
+  const int32_t* slots = nullptr; const int32_t* qsl = nullptr; const int32_t* positions = nullptr; const int32_t* token_req = nullptr;
+  int B = 0, T = 0, d = 0; bool inline_save = false;      // every request brings one row: no second pass over the slots
+  int elt = KGE_ELT_BF16;
+};
+int embed_bigram(const BigramArgs& a, cudaStream_t st);
 // y[r, :] = out_scale * x[rows ? rows[r] : r, :] / sqrt(mean(x^2) + eps) * (offset + w), x fp32, y in elt
 int rmsnorm_f32in(void* y, const float* x, const int32_t* rows, const void* w, int R, int d, float eps, float offset, float out_scale, int elt,
                   cudaStream_t st);
@@ -66,11 +86,15 @@ int group_rmsnorm_f32in(void* y, const float* x, const int32_t* rows, const void
 // A sublayer's result joins the residual stream through a norm of its own, and the next sublayer's input is formed in the same pass:
 //   y[t, :]   = src_scale * sum_i (inner_w[i] ? src_i[t, :] / sqrt(mean(src_i[t, :]^2) + eps) * inner_w[i] : src_i[t, :])      (nsrc <= 2)
 //   res[t, :] += gn(y[t, :]) * post_w           gn: the group norm above
-//   next_y[t, :] = gn(res[t, :]) * next_w       (next_w != null; next_y in elt)
-// Sources and weights in elt, statistics and sums in fp32.
+//   next_y[t, :] = gn(res[t, :]) * next_w       (next_y != null; next_w null: the new stream row itself; next_y in elt)
+// Sources and weights in elt, statistics and sums in fp32.  With pair_row (a mixture of experts; nsrc 0) the sublayer's
+// result is gathered instead: y[t, :] = sum_k pair_w[t * top + k] * (r_k >= 0 ? pair_src[r_k, :] : res[t, :]) with
+// r_k = pair_row[t * top + k], summed in choice order, an expert that returns its input (r_k < 0) taking the stream's own
+// fp32 row; pair_src rows are d wide.
 struct PostNormArgs {
   float* res = nullptr;
   const void* src[2] = {nullptr, nullptr}; int ld[2] = {0, 0}; const void* inner_w[2] = {nullptr, nullptr}; int nsrc = 1; float src_scale = 1.f;
+  const void* pair_src = nullptr; const int32_t* pair_row = nullptr; const float* pair_w = nullptr; int top = 0;
   const void* post_w = nullptr; const void* next_w = nullptr; void* next_y = nullptr;
   int T = 0, d = 0, groups = 1; float eps = 1e-5f; int elt = KGE_ELT_BF16;
 };
@@ -86,6 +110,19 @@ struct ShortConvArgs {
   int B = 0, T = 0; int elt = KGE_ELT_BF16;
 };
 int short_conv_state(const ShortConvArgs& a, cudaStream_t st);
+// The same convolution followed by a silu and, for the first unit_heads * head_dim channels, a division of every head of
+// head_dim channels by sqrt(sum of squares + unit_eps) (and a multiplication of the first scaled_heads of them by
+// head_scale); fp32 rows out.  Weights transposed: w [taps, C].  `inline_save`: every request of the step brings one row, so the
+// kernel that reads the slot's rows also brings them up to date.
+struct ConvHeadsArgs {
+  const void* x = nullptr; int ldx = 0; float* y = nullptr; int ldy = 0; const void* w = nullptr; int C = 0, taps = 1;
+  int unit_heads = 0, scaled_heads = 0, head_dim = 1; float head_scale = 1.f, unit_eps = 1e-6f;
+  float* state = nullptr; int64_t slot_stride = 0;
+  const int32_t* slots = nullptr; const int32_t* qsl = nullptr; const int32_t* positions = nullptr; const int32_t* token_req = nullptr;
+  int B = 0, T = 0; bool inline_save = false; int elt = KGE_ELT_BF16;
+  bool vec = false;                        // set by the launcher: four channels per lane
+};
+int short_conv_silu_heads(const ConvHeadsArgs& a, cudaStream_t st);
 inline int64_t short_conv_state_floats(int C, int taps) { return (int64_t)C * (taps - 1); }
 // y[t, n] = silu(gu[t, n]) * gu[t, f + n], n < f (gu [T, 2 f] in elt, the activation in fp32, one rounding)
 int silu_mul_halves(void* y, const void* gu, int T, int f, int elt, cudaStream_t st);
@@ -125,6 +162,7 @@ struct AttnBiasArgs {
   int window = 0, keep_first = 0, pool = 0;
   const void* pk_cache = nullptr; const void* pv_cache = nullptr;     // pooled caches [num_blocks, G, pool_slots, dim / vdim]
   int pool_slots = 0;                      // pooled entries per page: entry b of a request lives in its page b / pool_slots
+  int v_ld = 0;                            // elements between value rows (0: vdim); values may be the first columns of the key rows
   int elt = KGE_ELT_BF16;
 };
 int attn_bias_chunk(const AttnBiasArgs& a, cudaStream_t st);
@@ -233,6 +271,10 @@ inline int64_t mlstm_state_floats(int H, int dim, int vdim) { return (int64_t)H 
 // the `top` largest LOGITS are chosen and the weights are the softmax over the chosen logits only.  Produces for every
 // expert the list of (token, choice) pairs routed to it: group_off [E + 1], perm_token [T * top] (the token row of
 // every permuted row), perm_weight [T * top], perm_dest [T * top] (row t * top + choice of the output buffer).
+// `correction` (fp32 [E]) is added to the scores for the choice only.  groups > 1: neighbouring router outputs form equal
+// groups, and only those of the groups_keep groups with the largest best (corrected) score can be chosen.  The last
+// `identity` of the E outputs are experts without tensors: their pairs join no list (group_off has E - identity + 1
+// entries); pair_row [T * top] names every pair's permuted row, -1 for an identity expert.
 struct MoeRouteArgs {
   const void* h = nullptr; int ldh = 0; const void* w_router = nullptr; const void* b_router = nullptr;
   const void* w_extra = nullptr; float* extra_sigmoid = nullptr;      // one more row [d]: extra_sigmoid[t] = sigmoid(w_extra . h_t) (a per-token gate)
@@ -243,6 +285,7 @@ struct MoeRouteArgs {
   // entries, -1 in perm_token / perm_dest marks a row without a pair), and tile_group [rows_padded / pad] names the expert
   // of every tile of `pad` rows - what the grouped tensor-core GEMM reads
   int pad = 0, rows_padded = 0; int32_t* tile_group = nullptr;
+  const float* correction = nullptr; int groups = 1, groups_keep = 1, identity = 0; int32_t* pair_row = nullptr;
   int elt = KGE_ELT_BF16;
 };
 int moe_route(const MoeRouteArgs& a, cudaStream_t st);
@@ -296,10 +339,13 @@ struct WkvArgs {
   // norm_w rows are H * vdim wide), decay_mode 1: w_t = sigmoid(decay_pre_t)^(1 / tau) = exp(logsigmoid(decay_pre_t) / tau),
   // read_after: o_t = S_t^T r_t with S_t the state AFTER the update (no bonus u), r multiplied by r_scale in fp32
   int vdim = 0, decay_mode = 0; bool read_after = false; float tau = 1.f, r_scale = 1.f;
+  int gate_act = ACT_SILU;                 // the gate's activation: ACT_SILU or ACT_SIGMOID
   int elt = KGE_ELT_BF16;
 };
 int wkv_shift_mix(const WkvArgs& a, cudaStream_t st);
 int wkv_scan(const WkvArgs& a, cudaStream_t st);
+// the last part of wkv_scan alone: out = (o32 / rms per head) * norm_w * gate_act(gate_pre)   (o32, norm_w, gate_pre, out of a; T, H, vdim / dim, eps)
+int wkv_norm_gate(const WkvArgs& a, cudaStream_t st);
 inline int64_t wkv_state_floats(int d, int H, int dim) { return (int64_t)d + (int64_t)H * dim * dim; }
 inline int64_t gla_state_floats(int H, int dim, int vdim) { return (int64_t)H * dim * vdim; }     // WkvArgs with d = 0
 
@@ -326,6 +372,65 @@ struct LatentKvArgs {
   bool vec = false;                        // set by the launcher: every part is a whole number of 16-byte pieces
 };
 int latent_rotary_kvwrite(const LatentKvArgs& a, cudaStream_t st);
+// The same attention with the latents themselves in the cache: one row [c (kv_rank) | turned key part (rot_part)] per token
+// for all heads, cache [num_blocks, block_size, kv_rank + rot_part].
+//   latent_cache_write: z [T, kv_rank + rot_part] (the down-projection) -> the token's cache row, c = rms norm of the first
+//     kv_rank numbers times norm_w, the rest turned as above with cos / sin times mult (z null: a layer that reads another
+//     layer's cache); the rotated part of every query head turned in place, and for rows t < q_abs_rows also copied to
+//     q_abs[t, h, kv_rank ..] (row stride H * (kv_rank + rot_part)).
+//   latent_expand_plan: for the requests r0 .. r0 + n - 1 of the step, the pages from the one that holds the oldest key any of
+//     their rows can see (rounded down to a multiple of 64 positions) to their last get consecutive pages of a scratch
+//     cache: table [n, max_blocks] (entries outside: 0), src_page [pages] the page of the latent cache each one mirrors.
+//   latent_gather: rows [pages * block_size, kv_rank] <- the c part of those pages.
+//   latent_expand_write: kv [pages * block_size, H * nope + H * vdim] (every head's unrotated key part, then its value) and the
+//     turned key part of the cache rows -> scratch caches K [pages, H, block_size, dim], V [pages, H, block_size, vdim].
+struct LatentCacheArgs {
+  const void* z = nullptr; int ldz = 0; const void* norm_w = nullptr; float eps = 1e-5f;
+  void* q = nullptr; int ldq = 0; void* q_abs = nullptr; int q_abs_rows = 0;
+  const double* freq = nullptr; float mult = 1.f; int rot_dims = 0, rot_part = 0, kv_rank = 0;
+  const int32_t* positions = nullptr; const int64_t* slots = nullptr; void* cache = nullptr;
+  int T = 0, H = 0, dim = 0; int elt = KGE_ELT_BF16;
+};
+int latent_cache_write(const LatentCacheArgs& a, cudaStream_t st);
+int latent_expand_plan(int32_t* table, int32_t* src_page, const int32_t* block_table, int max_blocks, const int32_t* qsl, const int32_t* seq_lens, int r0, int n,
+                       int window, int block_size, int pages, cudaStream_t st);
+inline KGE_HD int latent_expand_first_page(int first_pos, int window, int block_size) {      // the page a request's copy starts with
+  const int lo = first_pos - window + 1 > 0 ? first_pos - window + 1 : 0;
+  return lo / 64 * 64 / block_size;
+}
+int latent_gather(void* rows, const void* cache, const int32_t* src_page, int pages, int block_size, int kv_rank, int ld, int elt, cudaStream_t st);
+int latent_expand_write(void* k_scratch, void* v_scratch, const void* kv, const void* cache, const int32_t* src_page, int pages, int block_size, int H, int dim,
+                        int vdim, int kv_rank, int rot_part, int elt, cudaStream_t st);
+// Attention of H query heads over the latent rows (queries already multiplied by the key up-projection: q_abs [T, H, kv_rank +
+// rot_part]): scores scale * q . row, a window (0: the causal prefix), sinks as in AttnBiasArgs, out [T, H, kv_rank] = the
+// weighted sum of the rows' c parts.  bfloat16, kv_rank up to 512 and kv_rank + rot_part up to 640, both multiples of 16:
+// latent_mqa (mma.sync, keys staged once for all heads, key range split over `splits` CTAs of a row tile and merged by a
+// second kernel; workspace of latent_mqa_workspace bytes).
+struct LatentMqaArgs {
+  const void* q = nullptr; void* out = nullptr; const void* cache = nullptr;
+  const int32_t* block_table = nullptr; int max_blocks = 0; const int32_t* qsl = nullptr; const int32_t* positions = nullptr;
+  int req0 = 0, B = 0, max_q = 1, T = 0;   // requests req0 .. req0 + B - 1; T: the step's rows (rows of q and out)
+  int H = 0, kv_rank = 0, rot_part = 0, block_size = 0, window = 0, splits = 1; float scale = 1.f; const float* sinks = nullptr;
+  void* workspace = nullptr; int64_t workspace_bytes = 0;
+};
+bool latent_mqa_ok(int H, int kv_rank, int rot_part, int block_size);
+int latent_mqa_splits(int B, int H, int max_q, int64_t keys);
+int64_t latent_mqa_workspace(int T, int H, int kv_rank, int splits);
+int latent_mqa(const LatentMqaArgs& a, cudaStream_t st);
+
+// Gated delta rule with a decay per key channel.  qkv fp32 rows (row stride ld): q [G, dim], k [G, dim] (unit vectors, q
+// scaled), v [H, vdim]; decay fp32 [T, H * dim]; beta_pre (elt, row stride ldb) [T, H].  Per head h (reading q / k head h / (H / G)),
+// with b = sigmoid(beta_pre):   S <- diag(decay) S;   u = b (v - S^T k);   S <- S + k u^T;   o = S^T q   -> o32 [T, H * vdim].
+// State per slot: S [H, dim, vdim] fp32, zero at position 0.  dim <= 256.
+struct DeltaArgs {
+  const float* qkv = nullptr; int ld = 0; const float* decay = nullptr; const void* beta_pre = nullptr; int ldb = 0;
+  float* o32 = nullptr; float* state = nullptr; int64_t slot_stride = 0;
+  const int32_t* slots = nullptr; const int32_t* qsl = nullptr; const int32_t* positions = nullptr;
+  int B = 0, T = 0, H = 0, G = 0, dim = 0, vdim = 0, max_q = 0; int elt = KGE_ELT_BF16;
+};
+int delta_scan(const DeltaArgs& a, cudaStream_t st);
+inline int64_t delta_state_floats(int H, int dim, int vdim) { return (int64_t)H * dim * vdim; }
+
 int sigmoid_gate_mul(void* y, int ldy, const void* g, int ldg, int T, int n, int elt, cudaStream_t st);
 
 }  // namespace kge

@@ -26,6 +26,8 @@ __device__ __forceinline__ float act_apply(int act, float v) {
     default: return v;
   }
 }
+// softplus without overflow on either side, then the decay exp(-coef * softplus(v))
+__device__ __forceinline__ float exp_decay(float coef, float v) { return expf(-coef * (fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))))); }
 
 // the gated pair of two pre-activations (row scale applied)
 __device__ __forceinline__ float glu_apply(const LinearArgs& a, float g, float u) {
@@ -101,7 +103,10 @@ __global__ void __launch_bounds__(256) linear_any_kernel(LinearArgs a) {
       if (n >= a.N) continue;
       float v;
       if (DUAL) v = glu_apply(a, s * acc[i][j], s * acc2[i][j]);
-      else v = act_apply(a.act, s * acc[i][j] + (bias ? ldf(bias + n) : 0.f));
+      else {
+        v = s * acc[i][j] + (bias ? ldf(bias + n) : 0.f);
+        v = a.act == ACT_EXP_DECAY ? exp_decay(a.act_coef[n], v) : act_apply(a.act, v);
+      }
       v *= a.alpha;
       O* dst = y + (int64_t)yr * a.ldy + n;
       if (a.accumulate) v += ldf(dst);
@@ -227,7 +232,10 @@ __global__ void __launch_bounds__(256) linear_mma_kernel(LinearArgs a) {
           const float s1 = acc[i][j][hh * 2 + c];
           float v;
           if (DUAL) v = glu_apply(a, sc * s1, sc * acc2[i][j][hh * 2 + c]);
-          else v = act_apply(a.act, sc * s1 + (bias ? ldf(bias + n) : 0.f));
+          else {
+            v = sc * s1 + (bias ? ldf(bias + n) : 0.f);
+            v = a.act == ACT_EXP_DECAY ? exp_decay(a.act_coef[n], v) : act_apply(a.act, v);
+          }
           v *= a.alpha;
           O* dst = y + (int64_t)yr * a.ldy + n;
           if (a.accumulate) v += ldf(dst);
@@ -238,6 +246,7 @@ __global__ void __launch_bounds__(256) linear_mma_kernel(LinearArgs a) {
 
 int linear_any(const LinearArgs& a, cudaStream_t st) {
   KGE_REQUIRE(a.x && a.w && a.y && a.N > 0 && a.K > 0 && a.nz > 0, "linear_any: bad arguments");
+  KGE_REQUIRE(a.act != ACT_EXP_DECAY || (a.act_coef && !a.w2), "linear_any: the decay needs its coefficients");
   if (a.T <= 0) return 0;
   const int rows = a.group_off ? (a.max_rows > 0 ? a.max_rows : a.T) : a.T;
   dim3 grid((a.N + LBN - 1) / LBN, (rows + LBM - 1) / LBM, a.nz), block(256);
@@ -269,6 +278,54 @@ int embed_f32(float* res, const int32_t* ids, const void* table, int T, int d, i
   cudaError_t ce = elt == KGE_ELT_F32 ? launch_pdl(embed_f32_kernel<float>, dim3(T), dim3(128), 0, st, res, ids, (const float*)table, d)
                                       : launch_pdl(embed_f32_kernel<__nv_bfloat16>, dim3(T), dim3(128), 0, st, res, ids, (const __nv_bfloat16*)table, d);
   KGE_CUDA_OK(ce);
+  return 0;
+}
+
+// one block per token; the row's four-column pieces when the tables allow
+template <typename E, bool VEC>
+__global__ void __launch_bounds__(256) embed_bigram_kernel(BigramArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, b = a.token_req[t], d = a.d, id = a.ids[t];
+  int32_t* last = a.bigram ? reinterpret_cast<int32_t*>(a.state + (int64_t)a.slots[b] * a.slot_stride) : nullptr;
+  int64_t row = a.buckets;
+  if (a.bigram && a.positions[t] > 0) {
+    const int64_t prev = t == a.qsl[b] ? *last : a.ids[t - 1];
+    row = (prev * a.mul_prev + (int64_t)id * a.mul_cur) % a.buckets;
+  }
+  const E* e = (const E*)a.table + (int64_t)id * d;
+  const E* g = (const E*)a.bigram + row * d;
+  float* r = a.res + (int64_t)t * d;
+  E* y = a.y ? (E*)a.y + (int64_t)t * d : nullptr;
+  constexpr int W = VEC ? 4 : 1;
+  for (int c = threadIdx.x * W; c < d; c += blockDim.x * W) {
+    float u[4], v[4] = {0.f, 0.f, 0.f, 0.f};
+    if (VEC) ld4(e + c, u); else u[0] = ldf(e + c);
+    if (a.bigram) { if (VEC) ld4(g + c, v); else v[0] = ldf(g + c); }
+#pragma unroll
+    for (int k = 0; k < W; ++k) u[k] += v[k];
+    if (VEC) { st4(r + c, u); if (y) st4(y + c, u); } else { r[c] = u[0]; if (y) stf(y + c, u[0]); }
+  }
+  if (a.bigram && a.inline_save) {
+    __syncthreads();                            // every thread has read the slot
+    if (threadIdx.x == 0) *last = id;
+  }
+}
+__global__ void bigram_save_kernel(BigramArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int b = blockIdx.x * blockDim.x + threadIdx.x;
+  if (b < a.B && a.qsl[b + 1] > a.qsl[b]) *reinterpret_cast<int32_t*>(a.state + (int64_t)a.slots[b] * a.slot_stride) = a.ids[a.qsl[b + 1] - 1];
+}
+int embed_bigram(const BigramArgs& a, cudaStream_t st) {
+  if (a.T <= 0) return 0;
+  KGE_REQUIRE(a.table && (!a.bigram || (a.buckets > 0 && a.state)), "embed_bigram: bad arguments");
+  const bool vec = a.d % 4 == 0 && ((reinterpret_cast<uintptr_t>(a.res) | reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.table) | reinterpret_cast<uintptr_t>(a.bigram)) & 15) == 0;
+  cudaError_t ce;
+  if (a.elt == KGE_ELT_F32) ce = vec ? launch_pdl(embed_bigram_kernel<float, true>, dim3(a.T), dim3(256), 0, st, a) : launch_pdl(embed_bigram_kernel<float, false>, dim3(a.T), dim3(256), 0, st, a);
+  else ce = vec ? launch_pdl(embed_bigram_kernel<__nv_bfloat16, true>, dim3(a.T), dim3(256), 0, st, a) : launch_pdl(embed_bigram_kernel<__nv_bfloat16, false>, dim3(a.T), dim3(256), 0, st, a);
+  KGE_CUDA_OK(ce);
+  if (a.bigram && !a.inline_save) KGE_CUDA_OK(launch_pdl(bigram_save_kernel, dim3((a.B + 127) / 128), dim3(128), 0, st, a));
   return 0;
 }
 

@@ -45,7 +45,13 @@ static bool parse_hybrid_mlp(const Json& l, HybridLayerSpec* hp, std::string* er
       if (sh && sh->is_obj()) { h.shared_ff = (int)sh->int_or("ff", 0); h.shared_limit = (float)sh->num_or("limit", 0.0); }
       h.expert_limit = (float)ex->num_or("limit", 0.0);
       h.router_scale = (float)ro->num_or("scale", 1.0);
-      if (h.expert_ff <= 0 || h.experts <= 0 || h.top <= 0 || h.top > h.experts) { *err = "config.json: bad moe sizes"; return false; }
+      h.identity = (int)ro->int_or("identity", 0);
+      if (const Json* g = ro->get("groups")) if (g->is_obj()) { h.router_groups = (int)g->int_or("count", 1); h.groups_keep = (int)g->int_or("keep", 1); }
+      const int outs = h.experts + h.identity;
+      if (h.expert_ff <= 0 || h.experts <= 0 || h.identity < 0 || h.top <= 0 || h.top > outs) { *err = "config.json: bad moe sizes"; return false; }
+      if (h.router_groups < 1 || outs % h.router_groups || h.groups_keep < 1 || h.groups_keep > h.router_groups || h.top > outs / h.router_groups * h.groups_keep) {
+        *err = "config.json: bad expert groups (count divides the router's outputs, keep <= count, top fits the kept groups)"; return false;
+      }
     } else { *err = "config.json: unknown mlp kind '" + kind + "'"; return false; }
   }
   return true;
@@ -305,7 +311,98 @@ static bool parse_balenex(const Json& j, ModelSpec* s, std::string* err) {
   return true;
 }
 
+// Kogonex: a layer list of 'latent_attention' (a window, a sink per head, YaRN rotation, the latents of an earlier layer
+// where 'kv_from' names one) and 'channel_delta' mixers (a gated delta rule with a decay per key channel behind short
+// convolutions), mixtures of experts with a choice correction, expert groups and identity experts, norms on the
+// sublayers' results only, and a bigram embedding added to the token's.
+static bool parse_kogonex(const Json& j, ModelSpec* s, std::string* err) {
+  s->model_type = "kogonex";
+  s->vocab = (int)j.int_or("vocab", 0);
+  s->d = (int)j.int_or("width", 0);
+  if (const Json* n = j.get("norm")) s->eps = (float)n->num_or("eps", 1e-5);
+  s->hyb_prenorm_pair = s->hyb_postnorm = s->hyb_noprenorm = true;
+  s->max_pos = 1 << 20;                 // rotary angles are computed from the position: no table bounds them
+  s->torch_dtype = "bfloat16";
+  s->bos = (int)j.int_or("bos_token_id", -1);
+  s->eos = (int)j.int_or("eos_token_id", -1);
+  if (s->vocab <= 0 || s->d <= 0) { *err = "config.json misses a required size"; return false; }
+  if (const Json* e = j.get("embedding")) if (e->is_obj()) {
+    if (const Json* b = e->get("bigram")) if (b->is_obj()) {
+      s->bigram_buckets = b->int_or("buckets", 0); s->bigram_mul_prev = b->int_or("mul_prev", 0); s->bigram_mul_cur = b->int_or("mul_cur", 0);
+      if (s->bigram_buckets <= 0 || s->bigram_buckets >= ((int64_t)1 << 31) || s->bigram_mul_prev < 0 || s->bigram_mul_cur < 0 ||
+          s->bigram_mul_prev >= ((int64_t)1 << 31) || s->bigram_mul_cur >= ((int64_t)1 << 31)) { *err = "config.json: bad 'embedding.bigram'"; return false; }
+    }
+  }
+  const Json* ls = j.get("layers");
+  if (!ls || !ls->is_arr() || ls->arr.empty()) { *err = "config.json: 'layers' must be a non-empty array"; return false; }
+  for (const Json& l : ls->arr) {
+    HybridLayerSpec h;
+    const int self = (int)s->hybrid.size();
+    const std::string type = l.str_or("type", "");
+    const Json* m = l.get("mixer");
+    if (!m || !m->is_obj()) { *err = "config.json: a layer has no 'mixer'"; return false; }
+    h.heads = (int)m->int_or("heads", 0);
+    if (type == "latent_attention") {
+      h.mixer = HybridLayerSpec::LATENT;
+      h.latent_cache = h.sink = true;
+      h.kv_heads = h.heads;
+      h.rot_part = (int)m->int_or("rot_dim", 0);
+      const int dim = (int)m->int_or("dim", 0);
+      h.dim = dim + h.rot_part;
+      h.vdim = (int)m->int_or("vdim", dim);
+      h.kv_rank = (int)m->int_or("kv_rank", 0);
+      h.scale = (float)m->num_or("scale", 1.0);
+      h.rot_dims = h.rot_part;
+      if (const Json* mk = m->get("mask")) if (mk->is_obj()) {
+        h.window = (int)std::min<int64_t>(mk->int_or("size", 0), (int64_t)1 << 30);
+        if (h.window <= 0) { *err = "config.json: 'mask.size' must be positive"; return false; }
+      }
+      if (const Json* r = m->get("rot")) if (r->is_obj()) {
+        h.rot_dims = (int)r->int_or("dims", h.rot_part); h.rot_base = r->num_or("base", 10000.0);
+        const Json* sc = r->get("scaling");
+        if (sc && sc->is_obj()) {
+          h.yarn_factor = sc->num_or("factor", 0.0); h.yarn_original = sc->num_or("original", 0.0);
+          h.yarn_fast = sc->num_or("fast", 32.0); h.yarn_slow = sc->num_or("slow", 1.0);
+          if (h.yarn_factor <= 0.0 || h.yarn_original <= 0.0 || h.yarn_fast <= 0.0 || h.yarn_slow <= 0.0) { *err = "config.json: bad rotary scaling"; return false; }
+        }
+      }
+      if (h.heads <= 0 || dim <= 0 || h.vdim <= 0 || h.kv_rank <= 0 || h.rot_part < 0 || h.rot_dims < 0 || h.rot_dims > h.rot_part || h.rot_dims % 2 ||
+          h.rot_base <= 0.0 || h.rot_base == 1.0) { *err = "config.json: bad latent-attention sizes"; return false; }
+      if (const Json* kf = m->get("kv_from")) if (kf->is_num()) {
+        h.kv_from = (int)kf->as_i64();
+        if (h.kv_from < 0 || h.kv_from >= self || s->hybrid[h.kv_from].mixer != HybridLayerSpec::LATENT || s->hybrid[h.kv_from].kv_from >= 0) {
+          *err = "config.json: 'kv_from' must name an earlier latent-attention layer with latents of its own"; return false;
+        }
+        const HybridLayerSpec& o = s->hybrid[h.kv_from];
+        if (o.kv_rank != h.kv_rank || o.rot_part != h.rot_part || o.rot_dims != h.rot_dims || o.rot_base != h.rot_base || o.yarn_factor != h.yarn_factor ||
+            o.yarn_original != h.yarn_original || o.yarn_fast != h.yarn_fast || o.yarn_slow != h.yarn_slow) {
+          *err = "config.json: a layer with 'kv_from' must have that layer's kv_rank, rot_dim and rotation"; return false;
+        }
+      }
+    } else if (type == "channel_delta") {
+      h.mixer = HybridLayerSpec::DELTA;
+      h.kv_heads = (int)m->int_or("kv_heads", h.heads);
+      h.dim = (int)m->int_or("dim", 0); h.vdim = (int)m->int_or("vdim", h.dim);
+      h.conv = (int)m->int_or("conv", 1);
+      h.decay_rank = (int)m->int_or("decay_rank", 0);
+      if (h.heads <= 0 || h.kv_heads <= 0 || h.heads % h.kv_heads || h.dim <= 0 || h.dim > 256 || h.vdim <= 0 || h.conv < 1 || h.conv > 16) {
+        *err = "config.json: bad channel-delta sizes (dim <= 256, 1 <= conv <= 16)"; return false;
+      }
+    } else { *err = "config.json: unknown layer type '" + type + "' (latent_attention, channel_delta)"; return false; }
+    if (!parse_hybrid_mlp(l, &h, err)) return false;
+    if (h.mlp == HybridLayerSpec::DENSE) { *err = "config.json: this architecture has no dense mlp"; return false; }
+    if (h.mlp == HybridLayerSpec::MOE) {
+      if (h.shared_ff > 0) { *err = "config.json: this architecture has no shared expert"; return false; }
+      h.route = HybridLayerSpec::ROUTE_SOFTMAX_ALL; h.glu = HybridLayerSpec::GLU_SILU; h.router_correction = true;
+    }
+    s->hybrid.push_back(h);
+  }
+  s->L = (int)s->hybrid.size();
+  return true;
+}
+
 static bool parse_config(const Json& j, ModelSpec* s, std::string* err) {
+  if (j.str_or("architecture", "") == "Kogonex") return parse_kogonex(j, s, err);
   if (j.str_or("architecture", "") == "Safupel") return parse_hybrid(j, s, err);
   if (j.str_or("architecture", "") == "Balenex") return parse_balenex(j, s, err);
   if (j.str_or("architecture", "") == "Girolorn") return parse_girolorn(j, s, err);
@@ -546,19 +643,22 @@ extern "C" int kge_model_spec_json(const kge_model_dir* m, char* out, int cap) {
                "\"yarn_factor\":%.17g,\"yarn_original\":%.17g,\"yarn_fast\":%.17g,\"yarn_slow\":%.17g,\"route\":%d,\"glu\":%d,\"expert_limit\":%.9g,"
                "\"shared_limit\":%.9g,\"weights_of\":%d,\"tensor_index\":%d,\"q_rank\":%d,\"kv_rank\":%d,\"rot_part\":%d,\"out_gate\":%d,"
                "\"decay_rank\":%d,\"ff_limit\":%.9g,\"router_scale\":%.9g,\"window\":%d,\"keep_first\":%d,\"pool\":%d,\"tau\":%.9g,"
-               "\"head_norm\":%d,\"rot_halves\":%d,\"v_rot\":%d,\"ff_silu_bias\":%d}",
+               "\"head_norm\":%d,\"rot_halves\":%d,\"v_rot\":%d,\"ff_silu_bias\":%d,\"latent_cache\":%d,\"kv_from\":%d,\"sink\":%d,"
+               "\"identity\":%d,\"router_groups\":%d,\"groups_keep\":%d,\"router_correction\":%d}",
                i ? "," : "", h.mixer, h.width, h.blocks, h.conv, h.heads, h.kv_heads, h.dim, h.vdim, h.chunk, (double)h.scale, (double)h.left_scale,
                (double)h.right_scale, h.m_heads, h.m_dim, h.m_vdim, (double)h.gate_cap, h.mlp, h.ff, h.experts, h.top, h.expert_ff, h.shared_ff,
                (double)h.softcap, h.rot_dims, h.rot_base, h.yarn_factor, h.yarn_original, h.yarn_fast, h.yarn_slow, h.route, h.glu, (double)h.expert_limit,
                (double)h.shared_limit, h.weights_of, h.tensor_index < 0 ? (int)i : h.tensor_index, h.q_rank, h.kv_rank, h.rot_part, h.out_gate ? 1 : 0,
                h.decay_rank, (double)h.ff_limit, (double)h.router_scale, h.window, h.keep_first, h.pool, (double)h.tau, h.head_norm ? 1 : 0,
-               h.rot_halves ? 1 : 0, h.v_rot ? 1 : 0, h.ff_silu_bias ? 1 : 0);
+               h.rot_halves ? 1 : 0, h.v_rot ? 1 : 0, h.ff_silu_bias ? 1 : 0, h.latent_cache ? 1 : 0, h.kv_from, h.sink ? 1 : 0, h.identity, h.router_groups,
+               h.groups_keep, h.router_correction ? 1 : 0);
       j += buf;
     }
     snprintf(buf, sizeof buf, "],\"eps\":%.9g,\"logit_scale\":%.9g,\"logit_softcap\":%.9g,\"streams\":%d,\"residual_mult\":%.9g,\"embed_norm\":%s,"
-             "\"norm_groups\":%d,\"postnorm\":%s}", (double)s.eps,
+             "\"norm_groups\":%d,\"postnorm\":%s,\"noprenorm\":%s,\"bigram_buckets\":%lld,\"bigram_mul_prev\":%lld,\"bigram_mul_cur\":%lld}", (double)s.eps,
              (double)s.logit_scale, (double)s.logit_softcap, s.streams, (double)s.residual_mult, s.embed_norm ? "true" : "false", s.norm_groups,
-             s.hyb_postnorm ? "true" : "false");
+             s.hyb_postnorm ? "true" : "false", s.hyb_noprenorm ? "true" : "false", (long long)s.bigram_buckets, (long long)s.bigram_mul_prev,
+             (long long)s.bigram_mul_cur);
     j += buf;
     KGE_REQUIRE((int)j.size() < cap, "kge_model_spec_json: buffer of %d bytes too small", cap);
     memcpy(out, j.c_str(), j.size() + 1);

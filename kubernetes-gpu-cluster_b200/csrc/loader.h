@@ -12,7 +12,7 @@ namespace kge {
 // One layer of a layer-list ("hybrid") model: which token mixer it has, that mixer's sizes and constants, and its
 // feed-forward.  Every number comes from config.json; the kernels take them as parameters.
 struct HybridLayerSpec {
-  enum Mixer { RGLRU = 0, PARALLEL = 1, ATTENTION = 2, WKV = 3, LATENT = 4, WINDOW_GLA = 5, POOLED = 6 };
+  enum Mixer { RGLRU = 0, PARALLEL = 1, ATTENTION = 2, WKV = 3, LATENT = 4, WINDOW_GLA = 5, POOLED = 6, DELTA = 7 };
   enum Mlp { NONE = 0, DENSE = 1, MOE = 2 };
   int mixer = RGLRU;
   // gated linear recurrence (RG-LRU): two branches of `width`, gates block-diagonal in `blocks` parts, causal conv of `conv` taps
@@ -42,8 +42,16 @@ struct HybridLayerSpec {
   // down-projection and is shared by all heads; queries come through a normed latent of `q_rank` numbers (0: one
   // matrix); rotary positions act on the first rot_dims of the rot_part; out_gate: the heads' outputs are multiplied by
   // sigmoid(W_g h) before the output matrix.  heads = kv_heads, dim counts the whole key, vdim the value.
+  // latent_cache: the paged cache holds a token's normed latent and its turned shared key part (one row of kv_rank +
+  // rot_part numbers for all heads) instead of every head's key and value; with it `window` limits the visible keys (0: the
+  // whole causal prefix), `sink` and the yarn_* constants apply, and a layer with kv_from >= 0 has no cache (and no
+  // down-projection) of its own: it reads the rows of that earlier layer.
   int q_rank = 0, kv_rank = 0, rot_part = 0;
-  bool out_gate = false;
+  bool out_gate = false, latent_cache = false;
+  int kv_from = -1;
+  // gated delta rule with a decay per key channel (DELTA): `heads` value heads of `vdim` numbers on `kv_heads` query / key
+  // heads of `dim` numbers; q, k and v pass a causal convolution of `conv` taps and a silu, q and k become unit vectors; the
+  // decay's and the output gate's logits come through low-rank pairs (ranks from the checkpoint; decay_rank without one)
   // windowed attention beside gated linear attention (WINDOW_GLA), both reading the same row; each side's output is
   // RMS-normed over the model width with a weight of its own and the mixer's result is half their sum.
   //   attention side (heads / kv_heads / dim / vdim / scale / rot_dims / rot_base as above): q, k and v carry biases and pass a
@@ -71,10 +79,15 @@ struct HybridLayerSpec {
   // the expert's output
   // ROUTE_SOFTMAX_ALL - softmax over all experts, the largest scores chosen, weight = score * router_scale (not
   // renormalised), multiplies the expert's output
+  // (with router_correction a learned number per expert is added to the scores for the choice only; with router_groups > 1
+  // neighbouring experts form that many equal groups and only those of the groups_keep groups with the largest best score
+  // can be chosen; the last `identity` router outputs are experts that return their input and own no tensors: `experts`
+  // counts the others)
   enum Route { ROUTE_SIGMOID_IN = 0, ROUTE_SOFTMAX_TOP = 1, ROUTE_SOFTMAX_ALL = 2 };
   int route = ROUTE_SIGMOID_IN;
   float router_scale = 1.f;
-  bool router_bias = false;
+  bool router_bias = false, router_correction = false;
+  int router_groups = 1, groups_keep = 1, identity = 0;
   // the experts' gated unit: GLU_SILU - silu(gate) * up; GLU_CLAMPED - g = min(gate, limit), u = clamp(up, -limit, limit),
   // g * sigmoid(1.702 g) * (u + 1)
   // GLU_NONE_RELU2 - no gate: down(relu(up h)^2)
@@ -84,11 +97,14 @@ struct HybridLayerSpec {
   bool shared_gate = false;                      // the shared expert's output is multiplied by sigmoid(w_sg . h), one number per token
   int weights_of = -1;                           // >= 0: this layer owns no tensors and runs with that layer's (cache and state stay its own)
   int tensor_index = -1;                         // the 'l<i>.' prefix of this layer's tensors (-1: its place in the list)
-  bool has_cache() const { return mixer == PARALLEL || mixer == ATTENTION || mixer == LATENT || mixer == WINDOW_GLA || mixer == POOLED; }
+  bool has_cache() const { return mixer == PARALLEL || mixer == ATTENTION || (mixer == LATENT && kv_from < 0) || mixer == WINDOW_GLA || mixer == POOLED; }
+  // numbers of one token's row in the paged caches (keys, then values), over all key/value heads
+  int64_t cache_k_row() const { return latent_cache ? kv_rank + rot_part : (int64_t)kv_heads * dim; }
+  int64_t cache_v_row() const { return latent_cache ? 0 : (int64_t)kv_heads * vdim; }
 };
 
 struct ModelSpec {
-  std::string model_type;       // "opt" | "llama" | "qwen2" | "qwen3" | "safupel" | "girolorn" | "zezilix" | "balenex"
+  std::string model_type;       // "opt" | "llama" | "qwen2" | "qwen3" | "safupel" | "girolorn" | "zezilix" | "balenex" | "kogonex"
   // layer-list models (config.json "architecture"): per-layer descriptions and the multiplier of the logits
   std::vector<HybridLayerSpec> hybrid;
   float logit_scale = 1.f;
@@ -100,8 +116,13 @@ struct ModelSpec {
   // norm_groups > 1: an RMS norm cuts its row into that many equal consecutive parts and divides each by its own root
   // mean square; hyb_postnorm: every sublayer's result goes through a norm of its own (weights norm1b / norm2b) before it
   // is added to the residual stream; norm weights multiply as they are
+  // hyb_noprenorm: with hyb_postnorm, the sublayers read the stream itself and only their results are normed (the weights are
+  // named norm1 / norm2)
   int norm_groups = 1;
-  bool hyb_postnorm = false;
+  bool hyb_postnorm = false, hyb_noprenorm = false;
+  // bigram embedding: row (previous token * mul_prev + token * mul_cur) mod buckets of a second table is added to the
+  // token's embedding; a sequence's first token takes row `buckets` (0 buckets: none)
+  int64_t bigram_buckets = 0, bigram_mul_prev = 0, bigram_mul_cur = 0;
   // hyper-connected residual: `streams` >= 1 copies of the residual stream, read through per-sublayer input weights,
   // mixed by a streams x streams matrix and written through output weights (0: one plain residual stream); every
   // sublayer's result is multiplied by residual_mult and, element by element, by a per-layer scale vector; the

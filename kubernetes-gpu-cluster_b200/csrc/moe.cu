@@ -1,5 +1,6 @@
 // Mixture-of-experts routing: fp32 router logits (optional bias), sigmoid or softmax scores or the raw logits with a
-// softmax over the chosen ones, top-k choice, and the grouping of
+// softmax over the chosen ones, top-k choice (optionally by corrected scores, within the best groups of neighbouring
+// experts, some of the experts returning their input), and the grouping of
 // (token, choice) pairs by expert that the grouped linear layer consumes.  Which rows an expert gets is all that the
 // grouping decides: a pair's result does not depend on its place in the group, and the pairs of a token are summed in
 // choice order afterwards, so the routing order never shows in the output.
@@ -76,12 +77,43 @@ __global__ void __launch_bounds__(256) moe_score_kernel(MoeRouteArgs a) {
     for (int e = lane; e < a.E; e += 32) sc[e] /= sum;
   }
   __syncwarp();
+  // what the choice goes by: the scores, or a copy of them with the correction added and all but the best groups taken out
+  float* ch = sc;
+  if (a.correction || a.groups > 1) {
+    ch = sc + a.E;
+    for (int e = lane; e < a.E; e += 32) ch[e] = a.correction ? sc[e] + a.correction[e] : sc[e];
+    __syncwarp();
+    if (a.groups > 1) {
+      float* gb = ch + a.E;                     // a group's best, -inf once it is kept
+      const int gs = a.E / a.groups;
+      for (int g = lane; g < a.groups; g += 32) {
+        float m = -INFINITY;
+        for (int e = 0; e < gs; ++e) m = fmaxf(m, ch[g * gs + e]);
+        gb[g] = m;
+      }
+      __syncwarp();
+      for (int k = 0; k < a.groups_keep; ++k) {
+        float bv = -INFINITY; int best = 0x7fffffff;
+        for (int g = lane; g < a.groups; g += 32) { const float v = gb[g]; if (v > bv) { bv = v; best = g; } }
+#pragma unroll
+        for (int off = 16; off > 0; off >>= 1) {
+          const float ov = __shfl_xor_sync(0xffffffffu, bv, off);
+          const int oi = __shfl_xor_sync(0xffffffffu, best, off);
+          if (ov > bv || (ov == bv && oi < best)) { bv = ov; best = oi; }
+        }
+        if (lane == 0 && best != 0x7fffffff) gb[best] = -INFINITY;
+        __syncwarp();
+      }
+      for (int e = lane; e < a.E; e += 32) if (gb[e / gs] != -INFINITY) ch[e] = -INFINITY;
+      __syncwarp();
+    }
+  }
   int32_t* ce = a.choice_expert + (int64_t)t * a.top;
   float* cw = a.choice_weight + (int64_t)t * a.top;
   for (int k = 0; k < a.top; ++k) {
     // the largest score not yet taken, the lower index on a tie; a taken score is marked -inf in shared memory
     float bv = -INFINITY; int best = 0x7fffffff;
-    for (int e = lane; e < a.E; e += 32) { const float v = sc[e]; if (v > bv) { bv = v; best = e; } }
+    for (int e = lane; e < a.E; e += 32) { const float v = ch[e]; if (v > bv) { bv = v; best = e; } }
 #pragma unroll
     for (int off = 16; off > 0; off >>= 1) {
       const float ov = __shfl_xor_sync(0xffffffffu, bv, off);
@@ -93,9 +125,9 @@ __global__ void __launch_bounds__(256) moe_score_kernel(MoeRouteArgs a) {
         best = 0;
         for (bool again = true; again;) { again = false; for (int q = 0; q < k; ++q) if (ce[q] == best) { ++best; again = true; } }
         bv = 0.f;
-      }
+      } else if (ch != sc) bv = sc[best];       // the weight is the score itself
       ce[k] = best; cw[k] = bv;
-      sc[best] = -INFINITY;
+      ch[best] = -INFINITY;
     }
     __syncwarp();
   }
@@ -119,18 +151,18 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(MoeRouteArgs a) {
   pdl_wait();
   extern __shared__ int cnt[];            // [E] counts, then [E] cursors
   int* cur = cnt + a.E;
-  const int n = a.T * a.top;
+  const int n = a.T * a.top, En = a.E - a.identity;      // experts with tensors
   for (int e = threadIdx.x; e < a.E; e += blockDim.x) cnt[e] = 0;
   __syncthreads();
   for (int i = threadIdx.x; i < n; i += blockDim.x) atomicAdd(&cnt[a.choice_expert[i]], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
     int off = 0;
-    for (int e = 0; e < a.E; ++e) {
+    for (int e = 0; e < En; ++e) {
       a.group_off[e] = off; cur[e] = off;
       off += a.pad > 1 ? (cnt[e] + a.pad - 1) / a.pad * a.pad : cnt[e];
     }
-    a.group_off[a.E] = off;
+    a.group_off[En] = off;
   }
   __syncthreads();
   if (a.pad > 1) {
@@ -139,13 +171,16 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(MoeRouteArgs a) {
     for (int i = threadIdx.x; i < a.rows_padded; i += blockDim.x) { a.perm_token[i] = -1; a.perm_dest[i] = -1; a.perm_weight[i] = 0.f; }
     for (int i = threadIdx.x; i < a.rows_padded / a.pad; i += blockDim.x) {
       int e = 0;
-      while (e + 1 < a.E && i * a.pad >= a.group_off[e + 1]) ++e;
-      a.tile_group[i] = i * a.pad < a.group_off[a.E] ? e : 0;
+      while (e + 1 < En && i * a.pad >= a.group_off[e + 1]) ++e;
+      a.tile_group[i] = i * a.pad < a.group_off[En] ? e : 0;
     }
     __syncthreads();
   }
   for (int i = threadIdx.x; i < n; i += blockDim.x) {
-    const int p = atomicAdd(&cur[a.choice_expert[i]], 1);
+    const int e = a.choice_expert[i];
+    if (e >= En) { if (a.pair_row) a.pair_row[i] = -1; continue; }
+    const int p = atomicAdd(&cur[e], 1);
+    if (a.pair_row) a.pair_row[i] = p;
     a.perm_token[p] = i / a.top;
     a.perm_weight[p] = a.choice_weight[i];
     a.perm_dest[p] = i;
@@ -193,10 +228,13 @@ int moe_scatter_rows(void* out, const void* operm, const int32_t* perm_dest, int
 int moe_route(const MoeRouteArgs& a, cudaStream_t st) {
   if (a.T <= 0) return 0;
   KGE_REQUIRE(a.E > 0 && a.top > 0 && a.top <= a.E && a.E <= 4096, "moe_route: %d experts, top %d", a.E, a.top);
-  KGE_REQUIRE(a.pad <= 1 || (a.tile_group && a.rows_padded % a.pad == 0 && a.rows_padded >= a.T * a.top + a.E * (a.pad - 1)),
-              "moe_route: padded groups need tile_group and %d rows or more", a.T * a.top + a.E * (a.pad - 1));
-  cudaError_t ce = a.elt == KGE_ELT_F32 ? launch_pdl(moe_score_kernel<float>, dim3(a.T), dim3(256), (size_t)a.E * 4, st, a)
-                                        : launch_pdl(moe_score_kernel<__nv_bfloat16>, dim3(a.T), dim3(256), (size_t)a.E * 4, st, a);
+  KGE_REQUIRE(a.pad <= 1 || (a.tile_group && a.rows_padded % a.pad == 0 && a.rows_padded >= a.T * a.top + (a.E - a.identity) * (a.pad - 1)),
+              "moe_route: padded groups need tile_group and %d rows or more", a.T * a.top + (a.E - a.identity) * (a.pad - 1));
+  KGE_REQUIRE(a.groups >= 1 && a.E % a.groups == 0 && a.groups_keep >= 1 && a.groups_keep <= a.groups && a.identity >= 0 && a.identity < a.E &&
+              (a.identity == 0 || a.pair_row), "moe_route: %d groups (%d kept), %d identity experts of %d", a.groups, a.groups_keep, a.identity, a.E);
+  const size_t smem = (size_t)(a.correction || a.groups > 1 ? 2 * a.E + a.groups : a.E) * 4;
+  cudaError_t ce = a.elt == KGE_ELT_F32 ? launch_pdl(moe_score_kernel<float>, dim3(a.T), dim3(256), smem, st, a)
+                                        : launch_pdl(moe_score_kernel<__nv_bfloat16>, dim3(a.T), dim3(256), smem, st, a);
   KGE_CUDA_OK(ce);
   KGE_CUDA_OK(launch_pdl(moe_group_kernel, dim3(1), dim3(1024), (size_t)2 * a.E * 4, st, a));
   return 0;

@@ -84,7 +84,101 @@ __global__ void __launch_bounds__(256) short_conv_save_kernel(ShortConvArgs a) {
   for (int s = 0; s < SC_MAX_TAPS - 1; ++s) if (s < keep) sp[(int64_t)s * a.C + c] = v[s];
 }
 
+// One warp per (token, head of head_dim channels) for the unit heads and per (token, 128 channels) for the rest: the
+// convolution's sums, the silu and a head's sum of squares stay in the warp's registers.  VEC: four neighbouring channels
+// per lane and pass.
+template <typename E, bool VEC>
+__global__ void __launch_bounds__(256) short_conv_silu_heads_kernel(ConvHeadsArgs a, int items) {
+  pdl_launch_dependents();
+  pdl_wait();
+  constexpr int W = VEC ? 4 : 1, MAXP = 256 / (32 * W);
+  const int lane = threadIdx.x & 31;
+  const int64_t item = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (item >= (int64_t)a.T * items) return;
+  const int t = (int)(item / items), u = (int)(item % items);
+  const bool unit = u < a.unit_heads;
+  const int c0 = unit ? u * a.head_dim : a.unit_heads * a.head_dim + (u - a.unit_heads) * 128;
+  const int n = unit ? a.head_dim : min(128, a.C - c0);
+  const int b = a.token_req[t], r0 = a.qsl[b], pos = a.positions[t], taps = a.taps;
+  float* sp = a.state + (int64_t)a.slots[b] * a.slot_stride;      // [taps - 1, C], oldest first
+  const E* x = (const E*)a.x;
+  float acc[MAXP][W];
+  float ss = 0.f;
+#pragma unroll
+  for (int p = 0; p < MAXP; ++p) {
+    const int k = (p * 32 + lane) * W;
+#pragma unroll
+    for (int q = 0; q < W; ++q) acc[p][q] = 0.f;
+    if (k < n) {
+      const int c = c0 + k;
+      for (int j = 0; j < taps; ++j) {
+        const int back = taps - 1 - j;                  // the input of position pos - back
+        if (pos - back < 0) continue;
+        const int row = t - back;
+        float in[4], w[4];
+        if (VEC) {
+          if (row >= r0) ld4(x + (int64_t)row * a.ldx + c, in); else ld4(sp + (int64_t)(taps - 1 - (r0 - row)) * a.C + c, in);
+          ld4((const E*)a.w + (int64_t)j * a.C + c, w);
+        } else {
+          in[0] = row >= r0 ? ldf(x + (int64_t)row * a.ldx + c) : sp[(int64_t)(taps - 1 - (r0 - row)) * a.C + c];
+          w[0] = ldf((const E*)a.w + (int64_t)j * a.C + c);
+        }
+#pragma unroll
+        for (int q = 0; q < W; ++q) acc[p][q] = fmaf(w[q], in[q], acc[p][q]);
+      }
+      if (a.inline_save) {                              // one row per request: this lane alone touches these channels of the slot
+        for (int s = 0; s + 1 < taps; ++s) {
+#pragma unroll
+          for (int q = 0; q < W; ++q) sp[(int64_t)s * a.C + c + q] = s + 2 < taps ? sp[(int64_t)(s + 1) * a.C + c + q] : ldf(x + (int64_t)t * a.ldx + c + q);
+        }
+      }
+#pragma unroll
+      for (int q = 0; q < W; ++q) {
+        const float v = acc[p][q];
+        acc[p][q] = v / (1.f + expf(-v));
+        ss = fmaf(acc[p][q], acc[p][q], ss);
+      }
+    }
+  }
+  float f = 1.f;
+  if (unit) {
+    f = 1.f / sqrtf(warp_sum(ss) + a.unit_eps);
+    if (u < a.scaled_heads) f *= a.head_scale;
+  }
+  float* y = a.y + (int64_t)t * a.ldy + c0;
+#pragma unroll
+  for (int p = 0; p < MAXP; ++p) {
+    const int k = (p * 32 + lane) * W;
+    if (k < n) {
+#pragma unroll
+      for (int q = 0; q < W; ++q) acc[p][q] *= f;
+      if constexpr (VEC) st4(y + k, acc[p]); else y[k] = acc[p][0];
+    }
+  }
+}
+
 }  // namespace
+
+int short_conv_silu_heads(const ConvHeadsArgs& a0, cudaStream_t st) {
+  if (a0.T <= 0) return 0;
+  ConvHeadsArgs a = a0;
+  KGE_REQUIRE(a.taps >= 1 && a.taps <= SC_MAX_TAPS && a.C > 0 && a.head_dim > 0 && a.head_dim <= 256 && a.unit_heads * a.head_dim <= a.C,
+              "short_conv_silu_heads: %d taps, %d heads of %d of %d channels", a.taps, a.unit_heads, a.head_dim, a.C);
+  const int items = a.unit_heads + (a.C - a.unit_heads * a.head_dim + 127) / 128;
+  a.vec = a.C % 4 == 0 && a.head_dim % 4 == 0 && a.ldx % 4 == 0 && a.ldy % 4 == 0 && a.slot_stride % 4 == 0 &&
+          ((reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(a.state)) & 15) == 0;
+  const dim3 grid((unsigned)(((int64_t)a.T * items + 7) / 8));
+  cudaError_t ce;
+  if (a.elt == KGE_ELT_F32) ce = a.vec ? launch_pdl(short_conv_silu_heads_kernel<float, true>, grid, dim3(256), 0, st, a, items) : launch_pdl(short_conv_silu_heads_kernel<float, false>, grid, dim3(256), 0, st, a, items);
+  else ce = a.vec ? launch_pdl(short_conv_silu_heads_kernel<__nv_bfloat16, true>, grid, dim3(256), 0, st, a, items) : launch_pdl(short_conv_silu_heads_kernel<__nv_bfloat16, false>, grid, dim3(256), 0, st, a, items);
+  KGE_CUDA_OK(ce);
+  if (a.inline_save || a.taps < 2) return 0;
+  ShortConvArgs s;      // the slots' rows move up after every row of the step has been read
+  s.x = a.x; s.ldx = a.ldx; s.C = a.C; s.taps = a.taps; s.state = a.state; s.slot_stride = a.slot_stride; s.slots = a.slots; s.qsl = a.qsl; s.positions = a.positions; s.B = a.B; s.T = a.T;
+  const dim3 sg(a.B, (a.C + 255) / 256);
+  KGE_CUDA_OK(a.elt == KGE_ELT_F32 ? launch_pdl(short_conv_save_kernel<float>, sg, dim3(256), 0, st, s) : launch_pdl(short_conv_save_kernel<__nv_bfloat16>, sg, dim3(256), 0, st, s));
+  return 0;
+}
 
 int short_conv_state(const ShortConvArgs& a, cudaStream_t st) {
   if (a.T <= 0) return 0;

@@ -311,7 +311,7 @@ __global__ void __launch_bounds__(256) wkv_chunk_kernel(WkvArgs a) {
     }
 }
 
-// one warp per (token, head): o / rms(o) * norm_w * silu(gate_pre)
+// one warp per (token, head): o / rms(o) * norm_w * silu(gate_pre) (or sigmoid(gate_pre))
 template <typename E>
 __global__ void __launch_bounds__(256) wkv_norm_gate_kernel(WkvArgs a) {
   pdl_launch_dependents();
@@ -327,7 +327,7 @@ __global__ void __launch_bounds__(256) wkv_norm_gate_kernel(WkvArgs a) {
   E* y = (E*)a.out + (int64_t)t * a.ldo + h * dim;
   for (int c = lane; c < dim; c += 32) {
     const float gv = ldf(g + c);
-    stf(y + c, o[c] * inv * ldf((const E*)a.norm_w + h * dim + c) * (gv / (1.f + expf(-gv))));
+    stf(y + c, o[c] * inv * ldf((const E*)a.norm_w + h * dim + c) * ((a.gate_act == ACT_SIGMOID ? 1.f : gv) / (1.f + expf(-gv))));
   }
 }
 
@@ -353,9 +353,25 @@ __global__ void __launch_bounds__(256) wkv_norm_gate_vec_kernel(WkvArgs a) {
     float v[4], gv[4], w[4], r[4];
     ld4(o + c, v); ld4(g + c, gv); ld4((const E*)a.norm_w + h * dim + c, w);
 #pragma unroll
-    for (int k = 0; k < 4; ++k) r[k] = v[k] * inv * w[k] * (gv[k] / (1.f + expf(-gv[k])));
+    for (int k = 0; k < 4; ++k) r[k] = v[k] * inv * w[k] * ((a.gate_act == ACT_SIGMOID ? 1.f : gv[k]) / (1.f + expf(-gv[k])));
     st4(y + c, r);
   }
+}
+
+template <typename E>
+static int norm_gate_t(const WkvArgs& a, cudaStream_t st) {
+  const int64_t items = (int64_t)a.T * a.H;
+  const int vd = a.vdim > 0 ? a.vdim : a.dim;
+  const bool vec = vd % 4 == 0 && a.ld % 4 == 0 && a.ldo % 4 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(a.o32) | reinterpret_cast<uintptr_t>(a.gate_pre) | reinterpret_cast<uintptr_t>(a.out) | reinterpret_cast<uintptr_t>(a.norm_w)) & 15) == 0;
+  if (vec) KGE_CUDA_OK(launch_pdl(wkv_norm_gate_vec_kernel<E>, dim3((unsigned)((items + 7) / 8)), dim3(256), 0, st, a));
+  else KGE_CUDA_OK(launch_pdl(wkv_norm_gate_kernel<E>, dim3((unsigned)((items + 7) / 8)), dim3(256), 0, st, a));
+  return 0;
+}
+int wkv_norm_gate(const WkvArgs& a, cudaStream_t st) {
+  if (a.T <= 0) return 0;
+  KGE_REQUIRE(a.gate_act == ACT_SILU || a.gate_act == ACT_SIGMOID, "wkv_norm_gate: activation %d", a.gate_act);
+  return a.elt == KGE_ELT_F32 ? norm_gate_t<float>(a, st) : norm_gate_t<__nv_bfloat16>(a, st);
 }
 
 template <typename E>
@@ -377,12 +393,7 @@ static int wkv_scan_t(const WkvArgs& a, cudaStream_t st) {
   else if (md <= 128) ce = launch_pdl(wkv_scan_kernel<E, 128>, grid, dim3(128), 0, st, a);
   else ce = launch_pdl(wkv_scan_kernel<E, 256>, grid, dim3(256), 0, st, a);
   KGE_CUDA_OK(ce);
-  const int64_t items = (int64_t)a.T * a.H;
-  const bool vec = vd % 4 == 0 && a.ld % 4 == 0 && a.ldo % 4 == 0 &&
-                   ((reinterpret_cast<uintptr_t>(a.o32) | reinterpret_cast<uintptr_t>(a.gate_pre) | reinterpret_cast<uintptr_t>(a.out) | reinterpret_cast<uintptr_t>(a.norm_w)) & 15) == 0;
-  if (vec) KGE_CUDA_OK(launch_pdl(wkv_norm_gate_vec_kernel<E>, dim3((unsigned)((items + 7) / 8)), dim3(256), 0, st, a));
-  else KGE_CUDA_OK(launch_pdl(wkv_norm_gate_kernel<E>, dim3((unsigned)((items + 7) / 8)), dim3(256), 0, st, a));
-  return 0;
+  return norm_gate_t<E>(a, st);
 }
 
 int wkv_scan(const WkvArgs& a, cudaStream_t st) {
