@@ -33,7 +33,7 @@ def moe_mlp(ff=12, experts=6, identity=2, top=3, groups=2, keep=1):
     return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "groups": {"count": groups, "keep": keep}, "identity": identity, "top": top}}
 
 
-def latent_layer(heads=3, dim=8, rot_dim=4, vdim=6, kv_rank=10, size=7, scale=0.35, base=500.0, factor=4.0, original=64, fast=6.0, slow=1.0, kv_from=None,
+def latent_layer(heads=3, dim=8, rot_dim=4, vdim=6, kv_rank=10, size=7, scale=0.15, base=500.0, factor=4.0, original=64, fast=6.0, slow=1.0, kv_from=None,
                  mlp="default"):
     m = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "mask": {"size": size}, "scale": scale,
          "rot": {"base": base, "dims": rot_dim, "scaling": {"factor": factor, "original": original, "fast": fast, "slow": slow}}}
@@ -46,7 +46,7 @@ def delta_layer(heads=4, kv_heads=2, dim=8, vdim=6, conv=3, mlp="default"):
     return {"type": "channel_delta", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}, "mlp": moe_mlp() if mlp == "default" else mlp}
 
 
-def make_config(layers, vocab=97, width=24, eps=1e-5, buckets=53, mul_prev=31, mul_cur=7):
+def make_config(layers, vocab=97, width=24, eps=1e-5, buckets=53, mul_prev=13, mul_cur=29):
     return {"architecture": "Kogonex", "embedding": {"bigram": {"buckets": buckets, "mul_prev": mul_prev, "mul_cur": mul_cur}}, "layers": layers,
             "norm": {"eps": eps}, "vocab": vocab, "width": width}
 
@@ -281,16 +281,22 @@ def route(h, P, r):
 
 
 def route_margin(h, P, r):
-    """How close a token's choice is: the smallest gap between choice scores (or group scores) that decides something."""
+    """How close a token's choice is: the smallest gap between two choice scores (of the last chosen and the first left out
+    expert, or of the best ones of the last kept and the first dropped group), relative to the larger of the two scores."""
     s = torch.softmax(h @ P["router"].T, dim=-1)
     c = s + P["correction"]
-    n, G, K = s.shape[1], r["groups"]["count"], r["groups"]["keep"]
-    best = torch.sort(c.reshape(-1, G, n // G).max(-1).values, dim=1, descending=True).values
-    gap = best[:, K - 1] - best[:, K] if K < G else torch.full((h.shape[0],), math.inf, dtype=DT)
-    kept = c.reshape(-1, G, n // G).max(-1).values >= best[:, K - 1:K]
-    c = torch.sort(c.masked_fill(~kept.repeat_interleave(n // G, dim=1), -math.inf), dim=1, descending=True).values
+    T, n, G, K = h.shape[0], s.shape[1], r["groups"]["count"], r["groups"]["keep"]
+    rel = lambda ca, cb, sa, sb: (ca - cb) / torch.maximum(sa, sb)
+    best, arg = c.reshape(T, G, n // G).max(-1)
+    sbest = torch.gather(s.reshape(T, G, n // G), 2, arg[:, :, None])[:, :, 0]
+    order = torch.sort(best, dim=1, descending=True).indices
+    at = lambda t, k: torch.gather(t, 1, order[:, k:k + 1])[:, 0]
+    gap = rel(at(best, K - 1), at(best, K), at(sbest, K - 1), at(sbest, K)) if K < G else torch.full((T,), math.inf, dtype=DT)
+    kept = best >= at(best, K - 1)[:, None]
+    order = torch.sort(c.masked_fill(~kept.repeat_interleave(n // G, dim=1), -math.inf), dim=1, descending=True).indices
     if r["top"] < n // G * K:
-        gap = torch.minimum(gap, c[:, r["top"] - 1] - c[:, r["top"]])
+        k = r["top"]
+        gap = torch.minimum(gap, rel(at(c, k - 1), at(c, k), at(s, k - 1), at(s, k)))
     return gap
 
 

@@ -95,11 +95,11 @@ def test_oracle_turn_and_yarn():
     a = 3 * 100.0 ** (-2.0 / 4)      # position 3, pair (2, 3)
     assert torch.allclose(y[3, 2], x[3, 2] * math.cos(a) - x[3, 3] * math.sin(a)) and torch.allclose(y[3, 3], x[3, 3] * math.cos(a) + x[3, 2] * math.sin(a))
     # scaling: the fastest pairs keep their frequency, the slowest are divided by the factor, lengths grow by the multiplier
-    rot = {"base": 10000.0, "dims": 32, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}
+    rot = {"base": 10000.0, "dims": 32, "scaling": {"factor": 6.0, "original": 4096, "fast": 24.0, "slow": 2.0}}
     f, mult = ok.yarn(rot)
     plain = [10000.0 ** (-2.0 * i / 32) for i in range(16)]
-    assert f[0] == plain[0] and abs(f[15] - plain[15] / 8.0) < 1e-15 and abs(mult - (0.1 * math.log(8.0) + 1.0)) < 1e-15
-    assert all(p / 8.0 <= q <= p for p, q in zip(plain, f)) and any(p / 8.0 < q < p for p, q in zip(plain, f))
+    assert f[0] == plain[0] and abs(f[15] - plain[15] / 6.0) < 1e-15 and abs(mult - (0.1 * math.log(6.0) + 1.0)) < 1e-15
+    assert all(p / 6.0 <= q <= p for p, q in zip(plain, f)) and any(p / 6.0 < q < p for p, q in zip(plain, f))
     z = torch.randn(3, 32, dtype=ok.DT)
     assert torch.allclose(ok.turn(z, [5, 6, 7], rot).pow(2).sum(-1), mult ** 2 * z.pow(2).sum(-1))
 
