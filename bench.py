@@ -2,7 +2,7 @@
 """Headline benchmark: output tokens/s at fixed concurrency (BASELINE.json `metric`).
 
   python bench.py --gpus N --steps K --warmup W [--workload c3|c2|c1] [--impl ours|reference]
-  python bench.py --designs [safupel|girolorn|zezilix|balenex]   (a layer-list design beside the closest other model of equal size; one JSON line per size)
+  python bench.py --designs [safupel|girolorn|zezilix|balenex|kogonex]   (a layer-list design beside the closest other model of equal size; one JSON line per size)
 
 A "step" is one whole job of the workload: every request prefilled (2k-token prompts, 8192 tokens
 per engine step as the continuous-batching scheduler cuts them) and decoded greedily to its output length.
@@ -621,6 +621,33 @@ def balenex_configs(z):
     return bal, design_configs(DESIGN_SIZES[z["safupel"]])[0]
 
 
+KOGONEX_SIZES = {
+    # attention over cached latents and a gated delta rule with grouped experts (Kogonex) at sizes that resemble real layers:
+    # latents of 512 with keys of 64 unrotated + 64 rotated numbers and values of 128, a window of 1024 positions, delta heads
+    # of 128 x 128; the model beside it is the closest one the engine has, the design with latent attention, matrix-valued
+    # recurrences and experts (Zezilix) of the same width, depth, heads and expert sizes
+    "w2048": dict(width=2048, vocab=32000, reps=2, heads=16, dim=64, rot=64, vdim=128, kv_rank=512, window=1024, d_heads=16, d_kv=16, d_dim=128, d_vdim=128, conv=4, rank=128,
+                  experts=16, identity=4, groups=4, keep=2, top=3, eff=1024, zezilix="w2048"),
+    "w4096": dict(width=4096, vocab=32000, reps=1, heads=32, dim=64, rot=64, vdim=128, kv_rank=512, window=1024, d_heads=32, d_kv=32, d_dim=128, d_vdim=128, conv=4, rank=128,
+                  experts=8, identity=2, groups=2, keep=1, top=3, eff=3584, zezilix="w4096"),
+}
+
+
+def kogonex_configs(z):
+    rot = {"base": 1000000.0, "dims": z["rot"], "scaling": {"factor": 16.0, "original": 4096, "fast": 24.0, "slow": 2.0}}
+    lat = {"dim": z["dim"], "heads": z["heads"], "kv_rank": z["kv_rank"], "mask": {"size": z["window"]}, "rot": rot, "rot_dim": z["rot"],
+           "scale": (z["dim"] + z["rot"]) ** -0.5, "vdim": z["vdim"]}
+    delta = {"conv": z["conv"], "dim": z["d_dim"], "heads": z["d_heads"], "kv_heads": z["d_kv"], "vdim": z["d_vdim"], "decay_rank": z["rank"]}
+    moe = {"expert": {"ff": z["eff"]}, "kind": "moe", "router": {"experts": z["experts"], "groups": {"count": z["groups"], "keep": z["keep"]}, "identity": z["identity"], "top": z["top"]}}
+    layers = []
+    for r in range(z["reps"]):
+        layers += [{"mixer": lat, "mlp": moe, "type": "latent_attention"}, {"mixer": delta, "mlp": moe, "type": "channel_delta"},
+                   {"mixer": delta, "mlp": moe, "type": "channel_delta"}, {"mixer": dict(lat, kv_from=4 * r), "mlp": moe, "type": "latent_attention"}]
+    kog = {"architecture": "Kogonex", "embedding": {"bigram": {"buckets": 65536, "mul_prev": 7919, "mul_cur": 104729}}, "layers": layers, "norm": {"eps": 1e-6},
+           "vocab": z["vocab"], "width": z["width"]}
+    return kog, zezilix_configs(ZEZILIX_SIZES[z["zezilix"]])[0]
+
+
 def time_raw_steps(kge, llm, batch_np, steps, warmup):
     """Wall-clock seconds per synchronous engine step (metadata upload, kernels, sampled ids back), after warm-up."""
     import ctypes as C
@@ -652,7 +679,7 @@ def raw_batch(B, ctx, q, bs, vocab, seed):
 
 
 def run_designs(args):
-    """--designs [safupel|girolorn|zezilix|balenex]: a layer-list design next to a Llama (or the closest other design) of equal size (random weights): one prefill step of 4 x 2048 tokens,
+    """--designs [safupel|girolorn|zezilix|balenex|kogonex]: a layer-list design next to a Llama (or the closest other design) of equal size (random weights): one prefill step of 4 x 2048 tokens,
     one decode step of 64 requests at context 2048, wall-clock per step plus per-kernel device times against the roofline."""
     from kge_loader import load
     kge = load()
@@ -661,7 +688,7 @@ def run_designs(args):
     B, ctx, PB, bs = 64, 2048, 4, args.block_size
     which = args.designs
     sizes, make, arms = {"girolorn": (GIROLORN_SIZES, girolorn_configs, ("girolorn", "llama")), "zezilix": (ZEZILIX_SIZES, zezilix_configs, ("zezilix", "girolorn")),
-                         "balenex": (BALENEX_SIZES, balenex_configs, ("balenex", "safupel")),
+                         "balenex": (BALENEX_SIZES, balenex_configs, ("balenex", "safupel")), "kogonex": (KOGONEX_SIZES, kogonex_configs, ("kogonex", "zezilix")),
                          "safupel": (DESIGN_SIZES, design_configs, ("safupel", "llama"))}[which]
     if args.sizes:
         sizes = {k: v for k, v in sizes.items() if k in args.sizes.split(",")}
@@ -729,7 +756,7 @@ def main():
     ap.add_argument("--tp-exchange", default="peer", choices=["peer", "nccl"], help="TP data path: peer memory (default) or NCCL")
     ap.add_argument("--tp-timeout", type=float, default=420.0, help="seconds the tensor-parallel leg may take at N > 1")
     ap.add_argument("--sizes", default="", help="with --designs: the sizes to run, with commas between them (all by default)")
-    ap.add_argument("--designs", nargs="?", const="safupel", default=None, choices=["safupel", "girolorn", "zezilix", "balenex"],
+    ap.add_argument("--designs", nargs="?", const="safupel", default=None, choices=["safupel", "girolorn", "zezilix", "balenex", "kogonex"],
                     help="instead of the workload: a layer-list design (safupel, the default, or girolorn) beside a Llama of equal "
                     "size, prefill and decode steps with per-kernel rooflines (one GPU, random weights)")
     args = ap.parse_args()

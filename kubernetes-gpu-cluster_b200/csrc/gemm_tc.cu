@@ -120,7 +120,7 @@ struct GemmParams {
   int glu = 0;               // gated pair: 0 silu(gate) * up; 1 clamped: g = min(gate, limit), u = clamp(up, +-limit), g * sigmoid(alpha g) * (u + 1)
   float glu_alpha = 0.f, glu_limit = 0.f;
   // grouped rows (mixture of experts): token rows come in groups padded to multiples of 256, tile_group[i] names the weight
-  // slice of rows [256 i, 256 (i + 1)), and slice g starts at weight row g * group_rows of the stacked weight tensor
+  // slice of rows [256 i, 256 (i + 1)) (negative: no rows, y is left alone), and slice g starts at weight row g * group_rows of the stacked weight tensor
   const int32_t* tile_group = nullptr;
   int group_rows = 0;
 };
@@ -276,6 +276,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant
   const int w_first = SPLIT ? (int)blockIdx.x / S : TWO ? (int)blockIdx.x / 2 : (int)blockIdx.x;
   const int w_step = SPLIT ? (1 << 30) : TWO ? (int)gridDim.x / 2 : (int)gridDim.x;
   auto m_tile_of = [&](int w) { return TWO ? 2 * (w / p.n_tiles) + mrank : w / p.n_tiles; };
+  // grouped rows: a tile beyond the last group has no work (every role reads the table after pdl_wait and skips alike)
+  auto no_rows = [&](int w) { return p.tile_group != nullptr && p.tile_group[((w % p.n_tiles) * TOKN) >> 8] < 0; };
   // PAIR: every TMA of a stage completes on the leader's (rank 0) full barrier
   auto lead_full = [&](int s) { return PAIR ? mapa_u32(full_bar(s), 0u) : full_bar(s); };
   const int kb0f = crank * p.kb_per_split, kb1f = min(p.kb_total, kb0f + p.kb_per_split);
@@ -376,6 +378,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant
       bool first_seg = true;
       while (it.next(w, kb0, kb1)) {
         const int n_tile = w % p.n_tiles, m_tile = m_tile_of(w);
+        if (no_rows(w)) continue;
         const int woff = p.tile_group ? p.tile_group[(n_tile * TOKN) >> 8] * p.group_rows : 0;
         for (int kb = kb0; kb < kb1; ++kb) {
           if (first_seg && kb - kb0 < pre) {
@@ -404,6 +407,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant
       const uint64_t adesc0 = umma_desc_sw128(smem_base), bdesc0 = umma_desc_sw128(smem_base + A_BYTES);
       uint64_t adesc = adesc0, bdesc = bdesc0;
       while (it.next(w, kb0, kb1)) {
+        if (no_rows(w)) continue;
         mbar_wait(tempty_bar(acc), acc_phase ^ 1);
         tc_fence_after();
         const uint32_t d_tmem = tmem_base + acc * TOKN;
@@ -435,6 +439,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant
     int w, kb0, kb1;
     while (it.next(w, kb0, kb1)) {
       const int n_tile = w % p.n_tiles, m_tile = m_tile_of(w);
+      if (no_rows(w)) continue;
       const int n = m_tile * ROWS_OUT + (GATED ? (et & 63) : et);   // output column of this thread's row
       const int t0 = n_tile * TOKN;
       mbar_wait(tfull_bar(acc), acc_phase);

@@ -283,7 +283,7 @@ struct MoeRouteArgs {
   int32_t* choice_expert = nullptr; float* choice_weight = nullptr;     // scratch [T * top] each
   // pad > 1: every expert's rows start at a multiple of `pad` (group_off holds the padded offsets; perm_* have rows_padded
   // entries, -1 in perm_token / perm_dest marks a row without a pair), and tile_group [rows_padded / pad] names the expert
-  // of every tile of `pad` rows - what the grouped tensor-core GEMM reads
+  // of every tile of `pad` rows (-1: none) - what the grouped tensor-core GEMM reads
   int pad = 0, rows_padded = 0; int32_t* tile_group = nullptr;
   const float* correction = nullptr; int groups = 1, groups_keep = 1, identity = 0; int32_t* pair_row = nullptr;
   int elt = KGE_ELT_BF16;

@@ -167,12 +167,12 @@ __global__ void __launch_bounds__(1024) moe_group_kernel(MoeRouteArgs a) {
   __syncthreads();
   if (a.pad > 1) {
     // padded groups: rows that carry no pair are marked (the gather writes zeros there, the scatter skips them), and every
-    // tile of `pad` rows learns its expert; tiles beyond the last group compute on zero rows with the first expert's weights
+    // tile of `pad` rows learns its expert (-1 beyond the last group: the GEMM skips it)
     for (int i = threadIdx.x; i < a.rows_padded; i += blockDim.x) { a.perm_token[i] = -1; a.perm_dest[i] = -1; a.perm_weight[i] = 0.f; }
     for (int i = threadIdx.x; i < a.rows_padded / a.pad; i += blockDim.x) {
       int e = 0;
       while (e + 1 < En && i * a.pad >= a.group_off[e + 1]) ++e;
-      a.tile_group[i] = i * a.pad < a.group_off[En] ? e : 0;
+      a.tile_group[i] = i * a.pad < a.group_off[En] ? e : -1;
     }
     __syncthreads();
   }
