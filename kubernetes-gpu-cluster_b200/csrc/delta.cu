@@ -24,22 +24,21 @@ __device__ __forceinline__ void dl_cp4(float* dst, const float* src) {
 __device__ __forceinline__ void dl_cp16(float* dst, const float* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src));
 }
-template <int N> __device__ __forceinline__ void dl_ld(const float* p, float (&v)[N]) {
-  if constexpr (N == 4) ld4(p, v);
-  else { const float2 t = *reinterpret_cast<const float2*>(p); v[0] = t.x; v[1] = t.y; }
-}
-template <int N> __device__ __forceinline__ void dl_st(float* p, const float (&v)[N]) {
-  if constexpr (N == 4) st4(p, v);
-  else *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
-}
+// two fp32 lanes per instruction: a pair holds two neighbouring key channels of one column
+typedef unsigned long long f2;
+__device__ __forceinline__ f2 pk(float lo, float hi) { f2 r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi)); return r; }
+__device__ __forceinline__ void upk(f2 v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
+__device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c) { f2 r; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c)); return r; }
+__device__ __forceinline__ f2 mul2(f2 a, f2 b) { f2 r; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b)); return r; }
+__device__ __forceinline__ float sum2(f2 v) { float a, b; upk(v, a, b); return a + b; }
 
-// KQ lanes x KPT channels cover dim; CPT columns per thread; a block owns `cols` value columns from blockIdx.x * cols on.
+// KQ lanes x KPT channels cover dim; CPT (four) columns per thread; a block owns `cols` value columns from blockIdx.x * cols on.
 // VEC: operand rows in 16-byte pieces, state rows and outputs in pieces of CPT columns.
-template <int KQ, int KPT, int CPT, int CT, bool VEC>
+template <int KQ, int KPT, int CT, bool VEC>
 __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a, int cols) {
   pdl_launch_dependents();
   pdl_wait();
-  constexpr int DK = KQ * KPT;
+  constexpr int DK = KQ * KPT, CPT = 4, NP = KPT / 2;
   extern __shared__ __align__(16) float dl_sm[];
   const int vld = (cols + 3) & ~3, per_tok = 3 * DK + vld;
   float* beta_s = dl_sm + 2 * CT * per_tok;          // [2][CT]
@@ -51,20 +50,25 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a, int cols) 
   const int kq = tid % KQ, col = (tid / KQ) * CPT;   // this thread's channel slice and first column (within the block)
   const bool fresh = a.positions[r0] == 0;
   float* Sg = a.state + (int64_t)a.slots[b] * a.slot_stride + (int64_t)h * dim * vdim + c0;
-  // channel of register i: chunk i / 4 of four channels, the KQ lanes' chunks side by side
-  float S[KPT][CPT];
+  // channels of pair i: chunk i / 2 of four channels, the KQ lanes' chunks side by side
+  auto chan = [&](int i) { return ((i >> 1) * KQ + kq) * 4 + (i & 1) * 2; };
+  f2 S[NP][CPT];
 #pragma unroll
-  for (int i = 0; i < KPT; ++i) {
-    const int k = ((i >> 2) * KQ + kq) * 4 + (i & 3);
+  for (int i = 0; i < NP; ++i) {
+    float x[2][4] = {};
 #pragma unroll
-    for (int j = 0; j < CPT; ++j) S[i][j] = 0.f;
-    if (!fresh && k < dim) {
-      if (VEC) { if (col < nc) dl_ld<CPT>(Sg + (int64_t)k * vdim + col, S[i]); }
-      else {
+    for (int e = 0; e < 2; ++e) {
+      const int k = chan(i) + e;
+      if (!fresh && k < dim) {
+        if (VEC) { if (col < nc) ld4(Sg + (int64_t)k * vdim + col, x[e]); }
+        else {
 #pragma unroll
-        for (int j = 0; j < CPT; ++j) if (col + j < nc) S[i][j] = Sg[(int64_t)k * vdim + col + j];
+          for (int j = 0; j < CPT; ++j) if (col + j < nc) x[e][j] = Sg[(int64_t)k * vdim + col + j];
+        }
       }
     }
+#pragma unroll
+    for (int j = 0; j < CPT; ++j) S[i][j] = pk(x[0][j], x[1][j]);
   }
   if (dim < DK || nc < vld) {                        // channels and columns that are never staged stay zero
     for (int i = tid; i < 2 * CT * per_tok; i += nt) dl_sm[i] = 0.f;
@@ -104,94 +108,105 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a, int cols) 
     const float* d = dl_sm + s * CT * per_tok;
     float* op = a.o32 + (int64_t)t0 * HV + (int64_t)h * vdim + c0 + col;
     for (int t = 0; t < n; ++t, d += per_tok, op += HV) {
-      float k[KPT], dk[CPT], dq[CPT], kq_dot = 0.f;
+      f2 k[NP], dk2[CPT], dq2[CPT], kq2 = 0ull;
 #pragma unroll
-      for (int j = 0; j < CPT; ++j) dk[j] = dq[j] = 0.f;
+      for (int j = 0; j < CPT; ++j) dk2[j] = dq2[j] = 0ull;
 #pragma unroll
       for (int c = 0; c < KPT / 4; ++c) {
         const int o = (c * KQ + kq) * 4;
-        float kk[4], qq[4], gg[4];
-        ld4(d + o, kk); ld4(d + DK + o, qq); ld4(d + 2 * DK + o, gg);
+        const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(d + o), qq = *reinterpret_cast<const ulonglong2*>(d + DK + o), gg = *reinterpret_cast<const ulonglong2*>(d + 2 * DK + o);
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          k[c * 4 + i] = kk[i];
-          kq_dot = fmaf(kk[i], qq[i], kq_dot);
+        for (int e = 0; e < 2; ++e) {
+          const int i = c * 2 + e;
+          const f2 ke = e ? kk.y : kk.x, qe = e ? qq.y : qq.x, ge = e ? gg.y : gg.x;
+          k[i] = ke;
+          kq2 = fma2(ke, qe, kq2);
 #pragma unroll
           for (int j = 0; j < CPT; ++j) {
-            const float x = S[c * 4 + i][j] * gg[i];
-            S[c * 4 + i][j] = x;
-            dk[j] = fmaf(x, kk[i], dk[j]);
-            dq[j] = fmaf(x, qq[i], dq[j]);
+            const f2 x = mul2(S[i][j], ge);
+            S[i][j] = x;
+            dk2[j] = fma2(x, ke, dk2[j]);
+            dq2[j] = fma2(x, qe, dq2[j]);
           }
         }
       }
       const float be = beta_s[s * CT + t];
-      float v[CPT], u[CPT];
-      dl_ld<CPT>(d + 3 * DK + col, v);
-      if constexpr (CPT == 2) {
-        // four sums over the KQ lanes: the lanes split them in two exchanges, so each ends with one sum; then every lane
-        // fetches the two sums along k, and the lanes that hold a sum along q write its output
-        const bool b0 = kq & 1, b1 = kq & 2;
-        float x0 = b0 ? dq[0] : dk[0], x1 = b0 ? dq[1] : dk[1];
-        x0 += __shfl_xor_sync(0xffffffffu, b0 ? dk[0] : dq[0], 1);
-        x1 += __shfl_xor_sync(0xffffffffu, b0 ? dk[1] : dq[1], 1);
-        float y = b1 ? x1 : x0;
-        y += __shfl_xor_sync(0xffffffffu, b1 ? x0 : x1, 2);
+      float v[CPT], u[CPT], dk[CPT], dq[CPT], kq_dot = sum2(kq2);
+      ld4(d + 3 * DK + col, v);
 #pragma unroll
-        for (int off = 4; off < KQ; off <<= 1) y += __shfl_xor_sync(0xffffffffu, y, off);
+      for (int j = 0; j < CPT; ++j) { dk[j] = sum2(dk2[j]); dq[j] = sum2(dq2[j]); }
 #pragma unroll
-        for (int off = 1; off < KQ; off <<= 1) kq_dot += __shfl_xor_sync(0xffffffffu, kq_dot, off);
+      for (int off = 1; off < KQ; off <<= 1) kq_dot += __shfl_xor_sync(0xffffffffu, kq_dot, off);
+      if constexpr (KQ >= 8) {
+        // eight sums over the KQ lanes: three exchanges split them, so each lane ends with one; then every lane fetches the
+        // four sums along k, and the lanes that hold a sum along q write its output
+        const bool b0 = kq & 1, b1 = kq & 2, b2 = kq & 4;
+        float x[4], z[2];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) x[j] = (b0 ? dq[j] : dk[j]) + __shfl_xor_sync(0xffffffffu, b0 ? dk[j] : dq[j], 1);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) z[j] = (b1 ? x[2 + j] : x[j]) + __shfl_xor_sync(0xffffffffu, b1 ? x[j] : x[2 + j], 2);
+        float y = (b2 ? z[1] : z[0]) + __shfl_xor_sync(0xffffffffu, b2 ? z[0] : z[1], 4);
+        if constexpr (KQ == 16) y += __shfl_xor_sync(0xffffffffu, y, 8);
         const int g0 = lane & ~(KQ - 1);
-        u[0] = be * (v[0] - __shfl_sync(0xffffffffu, y, g0));
-        u[1] = be * (v[1] - __shfl_sync(0xffffffffu, y, g0 + 2));
-        if (b0 && kq < 4) {
-          const int j = b1 ? 1 : 0;
-          if (col + j < nc) op[j] = fmaf(kq_dot, b1 ? u[1] : u[0], y);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) u[j] = be * (v[j] - __shfl_sync(0xffffffffu, y, g0 + (j >> 1) * 2 + (j & 1) * 4));
+        if (b0 && kq < 8) {
+          const int j = (b1 ? 2 : 0) + (b2 ? 1 : 0);
+          const float uj = b1 ? (b2 ? u[3] : u[2]) : (b2 ? u[1] : u[0]);
+          if (col + j < nc) op[j] = fmaf(kq_dot, uj, y);
         }
       } else {
 #pragma unroll
-        for (int off = KQ / 2; off > 0; off >>= 1) {
-          kq_dot += __shfl_xor_sync(0xffffffffu, kq_dot, off);
+        for (int off = KQ / 2; off > 0; off >>= 1)
 #pragma unroll
           for (int j = 0; j < CPT; ++j) { dk[j] += __shfl_xor_sync(0xffffffffu, dk[j], off); dq[j] += __shfl_xor_sync(0xffffffffu, dq[j], off); }
-        }
 #pragma unroll
         for (int j = 0; j < CPT; ++j) { u[j] = be * (v[j] - dk[j]); dq[j] = fmaf(kq_dot, u[j], dq[j]); }
         if (kq == 0 && col < nc) {
-          if (VEC) dl_st<CPT>(op, dq);
+          if (VEC) st4(op, dq);
           else {
 #pragma unroll
             for (int j = 0; j < CPT; ++j) if (col + j < nc) op[j] = dq[j];
           }
         }
       }
+      f2 uu[CPT];
 #pragma unroll
-      for (int i = 0; i < KPT; ++i)
+      for (int j = 0; j < CPT; ++j) uu[j] = pk(u[j], u[j]);
 #pragma unroll
-        for (int j = 0; j < CPT; ++j) S[i][j] = fmaf(k[i], u[j], S[i][j]);
+      for (int i = 0; i < NP; ++i)
+#pragma unroll
+        for (int j = 0; j < CPT; ++j) S[i][j] = fma2(k[i], uu[j], S[i][j]);
     }
   }
 #pragma unroll
-  for (int i = 0; i < KPT; ++i) {
-    const int k = ((i >> 2) * KQ + kq) * 4 + (i & 3);
-    if (k < dim) {
-      if (VEC) { if (col < nc) dl_st<CPT>(Sg + (int64_t)k * vdim + col, S[i]); }
-      else {
+  for (int i = 0; i < NP; ++i) {
+    float x[2][4];
 #pragma unroll
-        for (int j = 0; j < CPT; ++j) if (col + j < nc) Sg[(int64_t)k * vdim + col + j] = S[i][j];
+    for (int j = 0; j < CPT; ++j) upk(S[i][j], x[0][j], x[1][j]);
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int k = chan(i) + e;
+      if (k < dim) {
+        if (VEC) { if (col < nc) st4(Sg + (int64_t)k * vdim + col, x[e]); }
+        else {
+#pragma unroll
+          for (int j = 0; j < CPT; ++j) if (col + j < nc) Sg[(int64_t)k * vdim + col + j] = x[e][j];
+        }
       }
     }
   }
 }
 
-template <int KQ, int KPT, int CPT, int CT>
+template <int KQ, int KPT, int CT>
 int delta_launch(const DeltaArgs& a, bool vec, cudaStream_t st) {
   // up to four warps per block; fewer (more blocks) for heads with few columns
-  const int warp_cols = 32 / KQ * CPT;
+  const int warp_cols = 32 / KQ * 4;
   const int warps = std::min(4, (a.vdim + warp_cols - 1) / warp_cols), cols = warps * warp_cols;
   const dim3 grid((a.vdim + cols - 1) / cols, a.H, a.B), block(warps * 32);
   const size_t smem = (size_t)(2 * CT * (3 * KQ * KPT + ((cols + 3) & ~3)) + 2 * CT) * 4;
-  auto kern = vec ? delta_scan_kernel<KQ, KPT, CPT, CT, true> : delta_scan_kernel<KQ, KPT, CPT, CT, false>;
+  auto kern = vec ? delta_scan_kernel<KQ, KPT, CT, true> : delta_scan_kernel<KQ, KPT, CT, false>;
   if (smem > 48 * 1024) KGE_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   KGE_CUDA_OK(launch_pdl(kern, grid, block, smem, st, a, cols));
   return 0;
@@ -204,16 +219,16 @@ int delta_scan(const DeltaArgs& a, cudaStream_t st) {
   KGE_REQUIRE(a.dim > 0 && a.dim <= 256 && a.vdim > 0 && a.G > 0 && a.H % a.G == 0 && a.H <= 65535 && a.B <= 65535, "delta_scan: %d heads on %d of %d x %d", a.H, a.G, a.dim, a.vdim);
   const bool vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && a.ld % 4 == 0 && a.slot_stride % 4 == 0 &&
                    ((reinterpret_cast<uintptr_t>(a.qkv) | reinterpret_cast<uintptr_t>(a.decay) | reinterpret_cast<uintptr_t>(a.o32) | reinterpret_cast<uintptr_t>(a.state)) & 15) == 0;
-  if (a.T == a.B) {               // one row per request: the state is the traffic - 16-byte pieces of it, one token per stage
-    if (a.dim <= 32) return delta_launch<4, 8, 4, 1>(a, vec, st);
-    if (a.dim <= 64) return delta_launch<4, 16, 4, 1>(a, vec, st);
-    if (a.dim <= 128) return delta_launch<8, 16, 4, 1>(a, vec, st);
-    return delta_launch<16, 16, 4, 1>(a, vec, st);
+  if (a.T == a.B) {               // one row per request: one token per stage
+    if (a.dim <= 32) return delta_launch<4, 8, 1>(a, vec, st);
+    if (a.dim <= 64) return delta_launch<4, 16, 1>(a, vec, st);
+    if (a.dim <= 128) return delta_launch<8, 16, 1>(a, vec, st);
+    return delta_launch<16, 16, 1>(a, vec, st);
   }
-  if (a.dim <= 32) return delta_launch<4, 8, 2, 8>(a, vec, st);
-  if (a.dim <= 64) return delta_launch<4, 16, 2, 8>(a, vec, st);
-  if (a.dim <= 128) return delta_launch<8, 16, 2, 8>(a, vec, st);
-  return delta_launch<16, 16, 2, 4>(a, vec, st);
+  if (a.dim <= 32) return delta_launch<4, 8, 8>(a, vec, st);
+  if (a.dim <= 64) return delta_launch<4, 16, 8>(a, vec, st);
+  if (a.dim <= 128) return delta_launch<8, 16, 8>(a, vec, st);
+  return delta_launch<16, 16, 4>(a, vec, st);
 }
 
 }  // namespace kge

@@ -505,7 +505,7 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
         if (h.shared_gate) HB_OK(L.s_sg = b.mat({fp + "shared.sg"}, {1}, d, ws));
         max_ff = std::max(max_ff, h.shared_ff);
       }
-      max_top = std::max(max_top, h.top); max_eff = std::max(max_eff, h.expert_ff); max_E = std::max(max_E, h.experts + h.identity);
+      max_top = std::max(max_top, h.top); max_eff = std::max(max_eff, h.expert_ff); max_E = std::max(max_E, h.experts + h.identity); max_gate = std::max(max_gate, h.experts + h.identity);
     }
   }
 #undef HB_OK
@@ -1194,7 +1194,14 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
       const int np_pad = (np / 256 + h.experts + 1) * 256;
       const bool grouped = !e->f32 && !decode_only && np >= 512 && h.expert_ff % 64 == 0 && d % 8 == 0 && e->moe_xperm && np_pad <= e->moe_rows_padded;
       if (grouped) { ra.pad = 256; ra.rows_padded = np_pad; ra.tile_group = e->moe_tile_group; }
-      HFWD(C_MOE, Td * es + (double)h.experts * d * es, 2.0 * Td * h.experts, moe_route(ra, st));
+      if (T > 256 && !L.s_sg && ra.E <= 512) {
+        // many rows: the router's logits as one matrix product with fp32 sums
+        LinearArgs rl;
+        rl.x = e->hx; rl.ldx = d; rl.w = L.router.w; rl.bias = L.router_b; rl.y = e->gates32; rl.ldy = ra.E; rl.T = T; rl.N = ra.E; rl.K = d; rl.elt = elt; rl.out_f32 = true;
+        HFWD(C_MOE, Td * es + (double)ra.E * d * es, 2.0 * Td * ra.E, linear_any(rl, st));
+        ra.logits = e->gates32;
+        HFWD(C_MOE, 4.0 * T * ra.E, 0, moe_route(ra, st));
+      } else HFWD(C_MOE, Td * es + (double)ra.E * d * es, 2.0 * Td * ra.E, moe_route(ra, st));
       ++e->launches;
       const double wexp = (double)std::min(h.experts, np) * h.expert_ff * d * es;      // weights of the experts that are touched (at most)
       if (grouped) {

@@ -285,6 +285,7 @@ struct MoeRouteArgs {
   // entries, -1 in perm_token / perm_dest marks a row without a pair), and tile_group [rows_padded / pad] names the expert
   // of every tile of `pad` rows (-1: none) - what the grouped tensor-core GEMM reads
   int pad = 0, rows_padded = 0; int32_t* tile_group = nullptr;
+  const float* logits = nullptr;          // fp32 [T, E]: the router's logits, ready (bias in), instead of h and w_router
   const float* correction = nullptr; int groups = 1, groups_keep = 1, identity = 0; int32_t* pair_row = nullptr;
   int elt = KGE_ELT_BF16;
 };

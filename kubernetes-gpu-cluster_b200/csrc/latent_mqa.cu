@@ -1,10 +1,11 @@
 // Attention of all query heads of a request over its cached latent rows: every head's query has already been multiplied by
 // the head's key up-projection, so one row [c | turned key part] per token serves all heads as key (the whole row) and as
 // value (its c part), and a row is read once per 16 (token, head) pairs instead of once per head.
-// A CTA of four warps owns 16 query rows - consecutive (token, head) pairs of one request - and walks its part of the
-// visible keys in tiles of 32, staged in shared memory by cp.async one tile ahead:
-//   S = Q K^T   mma.sync m16n8k16, each warp 8 keys over all kv_rank + rot_part columns, fp32 scores to shared memory
-//   softmax     four rows per warp, one key per lane: window mask, running maximum and sum in fp32, P in bfloat16
+// A CTA of eight warps owns 16 query rows - consecutive (token, head) pairs of one request - and walks its part of the
+// visible keys in tiles of 32, staged in shared memory by cp.async three tiles ahead:
+//   S = Q K^T   mma.sync m16n8k16, each warp every eighth 16-column step of all 32 keys (its part of Q stays in registers),
+//               the warps' fp32 parts summed through shared memory
+//   softmax     two rows per warp, one key per lane: window mask, running maximum and sum in fp32, P in bfloat16
 //   O += P C    each warp its share of the kv_rank columns, fp32 accumulators in registers
 // Decode steps split the key range over several CTAs (too few requests to fill the GPU otherwise); a second kernel merges
 // their (m, l, O) and adds the sink's share of the denominator.  HBM-bound: a row's bytes are used for 2 * 16 heads' flops.
@@ -17,7 +18,7 @@ namespace kge {
 
 namespace {
 
-constexpr int LM_WARPS = 4, LM_KT = 32, LM_ROWS = 16, LM_PAD = 8;
+constexpr int LM_WARPS = 8, LM_KT = 32, LM_ROWS = 16, LM_PAD = 8, LM_ST = 4, LM_KSW = 5;      // LM_KSW: 16-column steps of a row per warp at most
 constexpr float LM_LOG2E = 1.4426950408889634f;
 typedef __nv_bfloat16 lm_bf16;
 
@@ -40,7 +41,7 @@ __device__ __forceinline__ void lm_mma(float (&c)[4], const uint32_t (&a)[4], ui
 
 constexpr int LM_SLD = LM_KT + 4, LM_PLD = LM_KT + 8;
 size_t lm_smem(int dim) {
-  return (size_t)(LM_ROWS + 2 * LM_KT) * (dim + LM_PAD) * 2 + (size_t)LM_ROWS * LM_SLD * 4 + (size_t)LM_ROWS * LM_PLD * 2 + 3 * LM_ROWS * 4;
+  return (size_t)LM_ST * LM_KT * (dim + LM_PAD) * 2 + (size_t)LM_WARPS * LM_ROWS * LM_SLD * 4 + (size_t)LM_ROWS * LM_PLD * 2 + 3 * LM_ROWS * 4;
 }
 
 // VP: 16-column pairs of the output per warp
@@ -50,10 +51,9 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_mqa_kernel(LatentMqaArgs
   pdl_wait();
   extern __shared__ __align__(16) unsigned char lm_raw[];
   const int dim = a.kv_rank + a.rot_part, ld = dim + LM_PAD, H = a.H;
-  lm_bf16* Qs = reinterpret_cast<lm_bf16*>(lm_raw);
-  lm_bf16* Ks = Qs + LM_ROWS * ld;
-  float* Ss = reinterpret_cast<float*>(Ks + 2 * LM_KT * ld);
-  lm_bf16* Ps = reinterpret_cast<lm_bf16*>(Ss + LM_ROWS * LM_SLD);
+  lm_bf16* Ks = reinterpret_cast<lm_bf16*>(lm_raw);
+  float* Ss = reinterpret_cast<float*>(Ks + LM_ST * LM_KT * ld);     // [warps][16][32]: every warp's part of the scores
+  lm_bf16* Ps = reinterpret_cast<lm_bf16*>(Ss + LM_WARPS * LM_ROWS * LM_SLD);
   float* cs = reinterpret_cast<float*>(Ps + LM_ROWS * LM_PLD);      // [16] correction of this tile, then [16] m, [16] l
   const int b = a.req0 + blockIdx.z, rs = a.qsl[b], nrows = (a.qsl[b + 1] - rs) * H, R0 = blockIdx.x * LM_ROWS;
   if (R0 >= nrows) return;
@@ -62,84 +62,103 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_mqa_kernel(LatentMqaArgs
   const int lo_min = a.window > 0 ? max(0, pos_first - a.window + 1) : 0;
   const int ntiles = (pos_last - lo_min) / LM_KT + 1, per = (ntiles + a.splits - 1) / a.splits;
   const int t0 = blockIdx.y * per, t1 = min(ntiles, t0 + per);
-  const int chunks = dim >> 3;
+  const int chunks = dim >> 3, bs_shift = 31 - __clz(a.block_size);
   const int32_t* bt = a.block_table + (int64_t)b * a.max_blocks;
   const lm_bf16* cache = (const lm_bf16*)a.cache;
-  // Q rows (rows beyond the request's repeat its last one; they are never written)
-  const lm_bf16* q = (const lm_bf16*)a.q + (int64_t)rs * H * dim;
-  for (int i = tid; i < LM_ROWS * chunks; i += LM_WARPS * 32) {
-    const int r = i / chunks, c = i % chunks;
-    lm_cp16(lm_saddr(Qs + r * ld + c * 8), q + (int64_t)min(R0 + r, nrows - 1) * dim + c * 8, true);
-  }
-  // a warp stages 8 of a tile's 32 rows; the first eight lanes look up where they live
-  auto stage = [&](int kt) {
-    lm_bf16* dst = Ks + (kt & 1) * LM_KT * ld + warp * 8 * ld;
-    const int j = lo_min + kt * LM_KT + warp * 8 + (lane & 7);
-    const int jc = min(j, pos_last);
-    const int64_t row = (int64_t)bt[jc / a.block_size] * a.block_size + jc % a.block_size;
-#pragma unroll
-    for (int r = 0; r < 8; ++r) {
-      const int64_t rr = __shfl_sync(0xffffffffu, row, r);
-      const bool ok = lo_min + kt * LM_KT + warp * 8 + r <= pos_last;
-      const lm_bf16* src = cache + rr * dim;
-      for (int c = lane; c < chunks; c += 32) lm_cp16(lm_saddr(dst + r * ld + c * 8), src + c * 8, ok);
-    }
+  // a warp stages 4 of a tile's 32 rows; where they live is looked up a tile earlier than it is needed
+  auto lookup = [&](int kt) -> int64_t {
+    const int j = min(lo_min + kt * LM_KT + warp * 4 + (lane & 3), pos_last);
+    return kt < t1 ? ((int64_t)bt[j >> bs_shift] << bs_shift) + (j & (a.block_size - 1)) : 0;
   };
-  if (t0 < t1) stage(t0);
-  asm volatile("cp.async.commit_group;");
+  auto stage = [&](int kt, int64_t row) {
+    if (kt < t1) {
+      lm_bf16* dst = Ks + ((kt - t0) % LM_ST * LM_KT + warp * 4) * ld;
+#pragma unroll
+      for (int r = 0; r < 4; ++r) {
+        const int64_t rr = __shfl_sync(0xffffffffu, row, r);
+        const bool ok = lo_min + kt * LM_KT + warp * 4 + r <= pos_last;
+        const lm_bf16* src = cache + rr * dim;
+        for (int c = lane; c < chunks; c += 32) lm_cp16(lm_saddr(dst + r * ld + c * 8), src + c * 8, ok);
+      }
+    }
+    asm volatile("cp.async.commit_group;");
+  };
+#pragma unroll
+  for (int i = 0; i < LM_ST - 1; ++i) stage(t0 + i, lookup(t0 + i));
+  int64_t nrow = lookup(t0 + LM_ST - 1);
+  // this warp's 16-column steps (warp, warp + 8, ..) of the 16 query rows, as A fragments (rows beyond the request's repeat its last one; they are never written)
+  const int ksteps = dim >> 4, vpairs = a.kv_rank >> 4;
+  uint32_t qf[LM_KSW][4];
+  {
+    const lm_bf16* q = (const lm_bf16*)a.q + (int64_t)rs * H * dim + (lane & 3) * 2;
+    const lm_bf16 *q0 = q + (int64_t)min(R0 + (lane >> 2), nrows - 1) * dim, *q1 = q + (int64_t)min(R0 + (lane >> 2) + 8, nrows - 1) * dim;
+#pragma unroll
+    for (int i = 0; i < LM_KSW; ++i) {
+      const int c = (warp + i * LM_WARPS) * 16;
+      const bool in = c < dim;
+      qf[i][0] = in ? *reinterpret_cast<const uint32_t*>(q0 + c) : 0u;
+      qf[i][1] = in ? *reinterpret_cast<const uint32_t*>(q1 + c) : 0u;
+      qf[i][2] = in ? *reinterpret_cast<const uint32_t*>(q0 + c + 8) : 0u;
+      qf[i][3] = in ? *reinterpret_cast<const uint32_t*>(q1 + c + 8) : 0u;
+    }
+  }
   float o[VP][2][4];
 #pragma unroll
   for (int v = 0; v < VP; ++v)
 #pragma unroll
     for (int n = 0; n < 2; ++n) o[v][n][0] = o[v][n][1] = o[v][n][2] = o[v][n][3] = 0.f;
-  float m[4], l[4];
-  int rpos[4], rlo[4];
+  float m[2], l[2];
+  int rpos[2], rlo[2];
 #pragma unroll
-  for (int i = 0; i < 4; ++i) {                       // the rows whose softmax this warp keeps
-    const int r = R0 + warp * 4 + i;
+  for (int i = 0; i < 2; ++i) {                       // the rows whose softmax this warp keeps
+    const int r = R0 + warp * 2 + i;
     m[i] = -INFINITY; l[i] = 0.f;
     rpos[i] = r < nrows ? a.positions[rs + r / H] : -1;
     rlo[i] = a.window > 0 ? max(0, rpos[i] - a.window + 1) : 0;
   }
   const float scale2 = a.scale * LM_LOG2E;
-  const int ksteps = dim >> 4, vpairs = a.kv_rank >> 4;
   for (int kt = t0; kt < t1; ++kt) {
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();                                  // this tile has landed; the other stage's readers are done
-    if (kt + 1 < t1) stage(kt + 1);
-    asm volatile("cp.async.commit_group;");
-    const lm_bf16* K = Ks + (kt & 1) * LM_KT * ld;
+    asm volatile("cp.async.wait_group %0;" ::"n"(LM_ST - 2) : "memory");
+    __syncthreads();                                  // this tile has landed; the readers of the stage refilled next are done
+    stage(kt + LM_ST - 1, nrow);
+    nrow = lookup(kt + LM_ST);
+    const lm_bf16* K = Ks + (kt - t0) % LM_ST * LM_KT * ld;
     {
-      float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
-      const uint32_t qa = lm_saddr(Qs + (lane & 15) * ld + (lane >> 4) * 8);
-      const lm_bf16* kr = K + (warp * 8 + (lane & 7)) * ld;
-      int ks = 0;
-#pragma unroll 4
-      for (; ks + 1 < ksteps; ks += 2) {
-        uint32_t a0[4], a1[4], bb[4];
-        lm_ldm4(a0, qa + ks * 32);
-        lm_ldm4(a1, qa + ks * 32 + 32);
-        lm_ldm4(bb, lm_saddr(kr + ks * 16 + (lane >> 3) * 8));
-        lm_mma(s0, a0, bb[0], bb[1]);
-        lm_mma(s1, a1, bb[2], bb[3]);
+      // this warp's columns of all 32 keys: four independent 16 x 8 products, summed over the warps below
+      float sc[4][4];
+#pragma unroll
+      for (int n = 0; n < 4; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
+      const lm_bf16* kr = K + (lane & 15) * ld + (lane >> 4) * 8;      // ldmatrix rows: 16 keys x two 8-column halves
+#pragma unroll
+      for (int i = 0; i < LM_KSW; ++i) {
+        const int ks = warp + i * LM_WARPS;
+        if (ks < ksteps) {
+#pragma unroll
+          for (int g = 0; g < 2; ++g) {
+            uint32_t bb[4];                           // keys g * 16 .. + 7: halves 0 and 2; + 8 .. 15: halves 1 and 3
+            lm_ldm4(bb, lm_saddr(kr + g * 16 * ld + ks * 16));
+            lm_mma(sc[2 * g], qf[i], bb[0], bb[2]);
+            lm_mma(sc[2 * g + 1], qf[i], bb[1], bb[3]);
+          }
+        }
       }
-      if (ks < ksteps) {
-        uint32_t a0[4], bb[4];
-        lm_ldm4(a0, qa + ks * 32);
-        lm_ldm4(bb, lm_saddr(kr + ks * 16 + ((lane >> 3) & 1) * 8));
-        lm_mma(s0, a0, bb[0], bb[1]);
+      float* d0 = Ss + (warp * LM_ROWS + (lane >> 2)) * LM_SLD + (lane & 3) * 2;
+#pragma unroll
+      for (int n = 0; n < 4; ++n) {
+        *reinterpret_cast<float2*>(d0 + n * 8) = make_float2(sc[n][0], sc[n][1]);
+        *reinterpret_cast<float2*>(d0 + 8 * LM_SLD + n * 8) = make_float2(sc[n][2], sc[n][3]);
       }
-      float* d0 = Ss + (lane >> 2) * LM_SLD + warp * 8 + (lane & 3) * 2;
-      *reinterpret_cast<float2*>(d0) = make_float2((s0[0] + s1[0]) * scale2, (s0[1] + s1[1]) * scale2);
-      *reinterpret_cast<float2*>(d0 + 8 * LM_SLD) = make_float2((s0[2] + s1[2]) * scale2, (s0[3] + s1[3]) * scale2);
     }
     __syncthreads();
     {
       const int j = lo_min + kt * LM_KT + lane;
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int r = warp * 4 + i;
-        const float s = (j <= rpos[i] && j >= rlo[i]) ? Ss[r * LM_SLD + lane] : -INFINITY;
+      for (int i = 0; i < 2; ++i) {
+        const int r = warp * 2 + i;
+        float s = 0.f;
+#pragma unroll
+        for (int w = 0; w < LM_WARPS; ++w) s += Ss[(w * LM_ROWS + r) * LM_SLD + lane];
+        s = (j <= rpos[i] && j >= rlo[i]) ? s * scale2 : -INFINITY;
         const float mn = fmaxf(m[i], warp_max(s));
         const float p = s == -INFINITY ? 0.f : exp2f(s - mn);
         const float corr = mn == -INFINITY ? 1.f : exp2f(m[i] - mn);
@@ -176,7 +195,7 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_mqa_kernel(LatentMqaArgs
   }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
 #pragma unroll
-  for (int i = 0; i < 4; ++i) if (lane == 0) { cs[LM_ROWS + warp * 4 + i] = m[i]; cs[2 * LM_ROWS + warp * 4 + i] = l[i]; }
+  for (int i = 0; i < 2; ++i) if (lane == 0) { cs[LM_ROWS + warp * 2 + i] = m[i]; cs[2 * LM_ROWS + warp * 2 + i] = l[i]; }
   __syncthreads();
   const int64_t grow = (int64_t)rs * H + R0;          // this tile's first row among all (token, head) pairs of the step
   if (a.splits > 1) {
@@ -269,12 +288,12 @@ int lm_launch(const LatentMqaArgs& a, cudaStream_t st) {
 }  // namespace
 
 bool latent_mqa_ok(int H, int kv_rank, int rot_part, int block_size) {
-  return H > 0 && kv_rank % 16 == 0 && rot_part % 16 == 0 && kv_rank > 0 && kv_rank <= 512 && kv_rank + rot_part <= 640 && block_size > 0;
+  return H > 0 && kv_rank % 16 == 0 && rot_part % 16 == 0 && kv_rank > 0 && kv_rank <= 512 && kv_rank + rot_part <= 16 * LM_KSW * LM_WARPS && block_size > 0 && (block_size & (block_size - 1)) == 0;
 }
-// parts the key range is cut into: enough CTAs for two per SM, at least two tiles of keys each
+// parts the key range is cut into: a CTA per SM (their stages fill its shared memory), at least two tiles of keys each
 int latent_mqa_splits(int B, int H, int max_q, int64_t keys) {
   const int64_t tiles = (int64_t)B * ((max_q * H + LM_ROWS - 1) / LM_ROWS);
-  const int64_t want = 296 / std::max<int64_t>(tiles, 1), most = keys / (2 * LM_KT);
+  const int64_t want = 148 / std::max<int64_t>(tiles, 1), most = keys / (2 * LM_KT);
   return (int)std::max<int64_t>(1, std::min<int64_t>(std::min(want, most), 16));
 }
 int64_t latent_mqa_workspace(int T, int H, int kv_rank, int splits) { return splits > 1 ? (int64_t)splits * T * H * (kv_rank + 2) * 4 : 0; }
@@ -285,7 +304,7 @@ int latent_mqa(const LatentMqaArgs& a, cudaStream_t st) {
   KGE_REQUIRE(a.splits == 1 || (a.max_q == 1 && a.workspace && a.workspace_bytes >= latent_mqa_workspace(a.T, a.H, a.kv_rank, a.splits)), "latent_mqa: %d parts need one row per request and a workspace", a.splits);
   KGE_REQUIRE(((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.cache) | reinterpret_cast<uintptr_t>(a.out)) & 15) == 0, "latent_mqa: rows must be 16-byte aligned");
   const int pairs = (a.kv_rank / 16 + LM_WARPS - 1) / LM_WARPS;
-  if (int rc = pairs <= 2 ? lm_launch<2>(a, st) : pairs <= 4 ? lm_launch<4>(a, st) : lm_launch<8>(a, st)) return rc;
+  if (int rc = pairs <= 1 ? lm_launch<1>(a, st) : pairs <= 2 ? lm_launch<2>(a, st) : lm_launch<4>(a, st)) return rc;
   // one row per request: the requests' rows follow one another from the first request's on
   if (a.splits > 1) KGE_CUDA_OK(launch_pdl(latent_mqa_merge_kernel, dim3((unsigned)(a.B * a.H)), dim3(128), 0, st, a, (int64_t)a.req0 * a.H));
   return 0;

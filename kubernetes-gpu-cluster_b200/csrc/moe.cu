@@ -40,30 +40,9 @@ __device__ __forceinline__ float dot_part(const float* h, const float* w, int d,
   return acc;
 }
 
-// One block per token: its eight warps share the experts' dot products (fp32, lanes summed by shuffles - the same order
-// whatever the launch holds) and, where asked, one more row whose sigmoid is a per-token gate; then the first warp picks
-// the top-k, each lane scanning its share of the scores.
-template <typename E>
-__global__ void __launch_bounds__(256) moe_score_kernel(MoeRouteArgs a) {
-  pdl_launch_dependents();
-  pdl_wait();
-  extern __shared__ float sc[];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x;
-  const E* h = (const E*)a.h + (int64_t)t * a.ldh;
-  constexpr int per = 16 / (int)sizeof(E);
-  const bool vec = a.d % per == 0 && a.ldh % per == 0 && (reinterpret_cast<uintptr_t>(a.h) & 15) == 0 && (reinterpret_cast<uintptr_t>(a.w_router) & 15) == 0 &&
-                   (reinterpret_cast<uintptr_t>(a.w_extra) & 15) == 0;
-  const int nrows = a.E + (a.w_extra ? 1 : 0);
-  for (int e = warp; e < nrows; e += 8) {
-    const E* w = e < a.E ? (const E*)a.w_router + (int64_t)e * a.d : (const E*)a.w_extra;
-    const float acc = warp_sum(dot_part(h, w, a.d, lane, vec));
-    if (lane == 0) {
-      if (e < a.E) sc[e] = a.b_router ? acc + ldf((const E*)a.b_router + e) : acc;
-      else a.extra_sigmoid[t] = 1.f / (1.f + expf(-acc));
-    }
-  }
-  __syncthreads();
-  if (warp != 0) return;
+// One warp: scores from a token's logits in sc (E entries, with room for the choice scores and the groups' best behind them),
+// the top-k choice and its weights; each lane scans its share of the scores.
+__device__ __forceinline__ void moe_pick(const MoeRouteArgs& a, int t, float* sc, int lane) {
   if (a.score_fn == 0) {
     for (int e = lane; e < a.E; e += 32) sc[e] = 1.f / (1.f + expf(-sc[e]));
   } else if (a.score_fn == 1) {
@@ -144,6 +123,45 @@ __global__ void __launch_bounds__(256) moe_score_kernel(MoeRouteArgs a) {
     }
     if (a.weight_scale != 1.f) for (int k = 0; k < a.top; ++k) cw[k] *= a.weight_scale;
   }
+}
+
+// One block per token: its eight warps share the experts' dot products (fp32, lanes summed by shuffles - the same order
+// whatever the launch holds) and, where asked, one more row whose sigmoid is a per-token gate; then the first warp picks
+// the top-k, each lane scanning its share of the scores.
+template <typename E>
+__global__ void __launch_bounds__(256) moe_score_kernel(MoeRouteArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ float sc[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x;
+  const E* h = (const E*)a.h + (int64_t)t * a.ldh;
+  constexpr int per = 16 / (int)sizeof(E);
+  const bool vec = a.d % per == 0 && a.ldh % per == 0 && (reinterpret_cast<uintptr_t>(a.h) & 15) == 0 && (reinterpret_cast<uintptr_t>(a.w_router) & 15) == 0 &&
+                   (reinterpret_cast<uintptr_t>(a.w_extra) & 15) == 0;
+  const int nrows = a.E + (a.w_extra ? 1 : 0);
+  for (int e = warp; e < nrows; e += 8) {
+    const E* w = e < a.E ? (const E*)a.w_router + (int64_t)e * a.d : (const E*)a.w_extra;
+    const float acc = warp_sum(dot_part(h, w, a.d, lane, vec));
+    if (lane == 0) {
+      if (e < a.E) sc[e] = a.b_router ? acc + ldf((const E*)a.b_router + e) : acc;
+      else a.extra_sigmoid[t] = 1.f / (1.f + expf(-acc));
+    }
+  }
+  __syncthreads();
+  if (warp == 0) moe_pick(a, t, sc, lane);
+}
+
+// The logits come from a matrix product (many rows): a warp per token does the rest.
+__global__ void __launch_bounds__(256) moe_pick_kernel(MoeRouteArgs a, int per_warp) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ float sc_all[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * 8 + warp;
+  if (t >= a.T) return;
+  float* sc = sc_all + warp * per_warp;
+  for (int e = lane; e < a.E; e += 32) sc[e] = a.logits[(int64_t)t * a.E + e];
+  __syncwarp();
+  moe_pick(a, t, sc, lane);
 }
 
 __global__ void __launch_bounds__(1024) moe_group_kernel(MoeRouteArgs a) {
@@ -232,8 +250,12 @@ int moe_route(const MoeRouteArgs& a, cudaStream_t st) {
               "moe_route: padded groups need tile_group and %d rows or more", a.T * a.top + (a.E - a.identity) * (a.pad - 1));
   KGE_REQUIRE(a.groups >= 1 && a.E % a.groups == 0 && a.groups_keep >= 1 && a.groups_keep <= a.groups && a.identity >= 0 && a.identity < a.E &&
               (a.identity == 0 || a.pair_row), "moe_route: %d groups (%d kept), %d identity experts of %d", a.groups, a.groups_keep, a.identity, a.E);
-  const size_t smem = (size_t)(a.correction || a.groups > 1 ? 2 * a.E + a.groups : a.E) * 4;
-  cudaError_t ce = a.elt == KGE_ELT_F32 ? launch_pdl(moe_score_kernel<float>, dim3(a.T), dim3(256), smem, st, a)
+  const int per = a.correction || a.groups > 1 ? 2 * a.E + a.groups : a.E;
+  const size_t smem = (size_t)per * 4;
+  KGE_REQUIRE(!a.logits || (!a.w_extra && smem * 8 <= 48 * 1024), "moe_route: %d router outputs with ready logits", a.E);
+  cudaError_t ce;
+  if (a.logits) ce = launch_pdl(moe_pick_kernel, dim3((a.T + 7) / 8), dim3(256), smem * 8, st, a, per);
+  else ce = a.elt == KGE_ELT_F32 ? launch_pdl(moe_score_kernel<float>, dim3(a.T), dim3(256), smem, st, a)
                                         : launch_pdl(moe_score_kernel<__nv_bfloat16>, dim3(a.T), dim3(256), smem, st, a);
   KGE_CUDA_OK(ce);
   KGE_CUDA_OK(launch_pdl(moe_group_kernel, dim3(1), dim3(1024), (size_t)2 * a.E * 4, st, a));

@@ -157,6 +157,107 @@ __global__ void __launch_bounds__(256) short_conv_silu_heads_kernel(ConvHeadsArg
   }
 }
 
+// The same for two to four taps and 16-byte rows: a warp keeps its channels' weights and the last taps - 1 inputs in registers
+// over a strip of TS tokens, so every input row is read once, and requests all rows of the strip before it uses the first.
+// MAXP: passes of 128 channels (heads of up to 128 * MAXP channels).
+template <typename E, int TAPS, int TS, int MAXP>
+__global__ void __launch_bounds__(256) short_conv_silu_heads_strip_kernel(ConvHeadsArgs a, int items) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int lane = threadIdx.x & 31;
+  const int64_t item = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
+  const int u = (int)(item % items);
+  const int64_t strip = item / items;
+  if (strip * TS >= a.T) return;
+  const int t0 = (int)strip * TS, nt = min(TS, a.T - t0);
+  const bool unit = u < a.unit_heads;
+  const int c0 = unit ? u * a.head_dim : a.unit_heads * a.head_dim + (u - a.unit_heads) * 128;
+  const int n = unit ? a.head_dim : min(128, a.C - c0);
+  const int ml = min(t0 + lane % TS, a.T - 1);                      // lane i knows token t0 + i's request, first row and position
+  const int mb = a.token_req[ml], mr = a.qsl[mb], mp = a.positions[ml];
+  const E* x = (const E*)a.x;
+  float cur[MAXP][TS][4], win[MAXP][TAPS - 1][4], w[MAXP][TAPS][4];
+#pragma unroll
+  for (int p = 0; p < MAXP; ++p) {
+    const int k = (p * 32 + lane) * 4;
+    if (k < n) {
+#pragma unroll
+      for (int i = 0; i < TS; ++i) if (i < nt) ld4(x + (int64_t)(t0 + i) * a.ldx + c0 + k, cur[p][i]);
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) ld4((const E*)a.w + (int64_t)j * a.C + c0 + k, w[p][j]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < TS; ++i) {
+    if (i >= nt) break;
+    const int t = t0 + i, r0 = __shfl_sync(0xffffffffu, mr, i), pos = __shfl_sync(0xffffffffu, mp, i), b = __shfl_sync(0xffffffffu, mb, i);
+    const bool fill = i == 0 || t == r0;                             // the inputs before this row: rows of the step, the slot's, or zeros
+    float* sp = a.state + (int64_t)a.slots[b] * a.slot_stride;
+    float ss = 0.f, y[MAXP][4];
+#pragma unroll
+    for (int p = 0; p < MAXP; ++p) {
+      const int k = (p * 32 + lane) * 4, c = c0 + k;
+#pragma unroll
+      for (int q = 0; q < 4; ++q) y[p][q] = 0.f;
+      if (k < n) {
+        if (fill) {
+#pragma unroll
+          for (int j = 0; j < TAPS - 1; ++j) {
+            const int back = TAPS - 1 - j, row = t - back;
+            if (pos - back < 0) { win[p][j][0] = win[p][j][1] = win[p][j][2] = win[p][j][3] = 0.f; }
+            else if (row >= r0) ld4(x + (int64_t)row * a.ldx + c, win[p][j]);
+            else ld4(sp + (int64_t)(TAPS - 1 - (r0 - row)) * a.C + c, win[p][j]);
+          }
+        }
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          float acc = 0.f;
+#pragma unroll
+          for (int j = 0; j < TAPS - 1; ++j) acc = fmaf(w[p][j][q], win[p][j][q], acc);
+          acc = fmaf(w[p][TAPS - 1][q], cur[p][i][q], acc);
+#pragma unroll
+          for (int j = 0; j + 1 < TAPS - 1; ++j) win[p][j][q] = win[p][j + 1][q];
+          win[p][TAPS - 2][q] = cur[p][i][q];
+          y[p][q] = acc / (1.f + expf(-acc));
+          ss = fmaf(y[p][q], y[p][q], ss);
+        }
+        if (a.inline_save) {                                         // one row per request: this lane alone touches these channels of the slot
+#pragma unroll
+          for (int j = 0; j < TAPS - 1; ++j) st4(sp + (int64_t)j * a.C + c, win[p][j]);
+        }
+      }
+    }
+    float f = 1.f;
+    if (unit) {
+      f = 1.f / sqrtf(warp_sum(ss) + a.unit_eps);
+      if (u < a.scaled_heads) f *= a.head_scale;
+    }
+#pragma unroll
+    for (int p = 0; p < MAXP; ++p) {
+      const int k = (p * 32 + lane) * 4;
+      if (k < n) {
+#pragma unroll
+        for (int q = 0; q < 4; ++q) y[p][q] *= f;
+        st4(a.y + (int64_t)t * a.ldy + c0 + k, y[p]);
+      }
+    }
+  }
+}
+
+template <typename E, int TAPS, int TS>
+cudaError_t launch_strip(const ConvHeadsArgs& a, int items, cudaStream_t st) {
+  const dim3 grid((unsigned)(((int64_t)((a.T + TS - 1) / TS) * items + 7) / 8));
+  return a.head_dim <= 128 ? launch_pdl(short_conv_silu_heads_strip_kernel<E, TAPS, TS, 1>, grid, dim3(256), 0, st, a, items)
+                           : launch_pdl(short_conv_silu_heads_strip_kernel<E, TAPS, TS, 2>, grid, dim3(256), 0, st, a, items);
+}
+template <typename E>
+cudaError_t launch_strips(const ConvHeadsArgs& a, int items, cudaStream_t st) {
+  const bool many = a.T >= 32 && a.T > a.B;                         // prompt pieces: strips of eight rows; single tokens: a warp per (row, head)
+  if (a.taps == 2) return many ? launch_strip<E, 2, 8>(a, items, st) : launch_strip<E, 2, 1>(a, items, st);
+  if (a.taps == 3) return many ? launch_strip<E, 3, 8>(a, items, st) : launch_strip<E, 3, 1>(a, items, st);
+  return many ? launch_strip<E, 4, 8>(a, items, st) : launch_strip<E, 4, 1>(a, items, st);
+}
+
 }  // namespace
 
 int short_conv_silu_heads(const ConvHeadsArgs& a0, cudaStream_t st) {
@@ -169,7 +270,8 @@ int short_conv_silu_heads(const ConvHeadsArgs& a0, cudaStream_t st) {
           ((reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(a.state)) & 15) == 0;
   const dim3 grid((unsigned)(((int64_t)a.T * items + 7) / 8));
   cudaError_t ce;
-  if (a.elt == KGE_ELT_F32) ce = a.vec ? launch_pdl(short_conv_silu_heads_kernel<float, true>, grid, dim3(256), 0, st, a, items) : launch_pdl(short_conv_silu_heads_kernel<float, false>, grid, dim3(256), 0, st, a, items);
+  if (a.vec && a.taps >= 2 && a.taps <= 4) ce = a.elt == KGE_ELT_F32 ? launch_strips<float>(a, items, st) : launch_strips<__nv_bfloat16>(a, items, st);
+  else if (a.elt == KGE_ELT_F32) ce = a.vec ? launch_pdl(short_conv_silu_heads_kernel<float, true>, grid, dim3(256), 0, st, a, items) : launch_pdl(short_conv_silu_heads_kernel<float, false>, grid, dim3(256), 0, st, a, items);
   else ce = a.vec ? launch_pdl(short_conv_silu_heads_kernel<__nv_bfloat16, true>, grid, dim3(256), 0, st, a, items) : launch_pdl(short_conv_silu_heads_kernel<__nv_bfloat16, false>, grid, dim3(256), 0, st, a, items);
   KGE_CUDA_OK(ce);
   if (a.inline_save || a.taps < 2) return 0;
