@@ -24,6 +24,14 @@ __device__ __forceinline__ void dl_cp4(float* dst, const float* src) {
 __device__ __forceinline__ void dl_cp16(float* dst, const float* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src));
 }
+template <int N> __device__ __forceinline__ void dl_ld(const float* p, float (&v)[N]) {
+  if constexpr (N == 4) ld4(p, v);
+  else { const float2 t = *reinterpret_cast<const float2*>(p); v[0] = t.x; v[1] = t.y; }
+}
+template <int N> __device__ __forceinline__ void dl_st(float* p, const float (&v)[N]) {
+  if constexpr (N == 4) st4(p, v);
+  else *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
+}
 // two fp32 lanes per instruction: a pair holds two neighbouring key channels of one column
 typedef unsigned long long f2;
 __device__ __forceinline__ f2 pk(float lo, float hi) { f2 r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi)); return r; }
@@ -32,17 +40,17 @@ __device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c) { f2 r; asm("fma.rn.f32x2 %
 __device__ __forceinline__ f2 mul2(f2 a, f2 b) { f2 r; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b)); return r; }
 __device__ __forceinline__ float sum2(f2 v) { float a, b; upk(v, a, b); return a + b; }
 
-// KQ lanes x KPT channels cover dim; CPT (four) columns per thread; a block owns `cols` value columns from blockIdx.x * cols on.
+// KQ lanes x KPT channels cover dim; CPT columns per thread; a block owns `cols` value columns from blockIdx.x * cols on.
 // VEC: operand rows in 16-byte pieces, state rows and outputs in pieces of CPT columns.
-template <int KQ, int KPT, int CT, bool VEC>
-__global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a, int cols) {
+template <int KQ, int KPT, int CPT, int CT, bool VEC>
+__global__ void __launch_bounds__(256) delta_scan_kernel(DeltaArgs a, int cols) {
   pdl_launch_dependents();
   pdl_wait();
-  constexpr int DK = KQ * KPT, CPT = 4, NP = KPT / 2;
+  constexpr int DK = KQ * KPT, NP = KPT / 2;
   extern __shared__ __align__(16) float dl_sm[];
   const int vld = (cols + 3) & ~3, per_tok = 3 * DK + vld;
   float* beta_s = dl_sm + 2 * CT * per_tok;          // [2][CT]
-  const int h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, nt = blockDim.x, lane = tid & 31, warp = tid >> 5, nw = nt >> 5;
+  const int h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, nt = blockDim.x, lane = tid & 31;
   const int r0 = a.qsl[b], r1 = a.qsl[b + 1];
   if (r0 >= r1) return;
   const int dim = a.dim, vdim = a.vdim, hk = h / (a.H / a.G), HD = a.H * dim, HV = a.H * vdim;
@@ -55,12 +63,12 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a, int cols) 
   f2 S[NP][CPT];
 #pragma unroll
   for (int i = 0; i < NP; ++i) {
-    float x[2][4] = {};
+    float x[2][CPT] = {};
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int k = chan(i) + e;
       if (!fresh && k < dim) {
-        if (VEC) { if (col < nc) ld4(Sg + (int64_t)k * vdim + col, x[e]); }
+        if (VEC) { if (col < nc) dl_ld<CPT>(Sg + (int64_t)k * vdim + col, x[e]); }
         else {
 #pragma unroll
           for (int j = 0; j < CPT; ++j) if (col + j < nc) x[e][j] = Sg[(int64_t)k * vdim + col + j];
@@ -75,6 +83,10 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a, int cols) 
     __syncthreads();
   }
   const float* src[4] = {a.qkv + (int64_t)(a.G + hk) * dim, a.qkv + (int64_t)hk * dim, a.decay + (int64_t)h * dim, a.qkv + (int64_t)2 * a.G * dim + (int64_t)h * vdim + c0};
+  constexpr int W = VEC ? 4 : 1;
+  const int piece_k = dim / W, roles = 3 * piece_k + nc / W;                    // pieces of a token's k, q, decay and value columns
+  const int tpar = max(1, nt / roles), role0 = nt >= roles ? tid % roles : tid, role_step = nt >= roles ? roles : nt;
+  const int tok0 = nt >= roles ? (tid / roles < tpar ? tid / roles : CT) : 0;  // left-over threads copy nothing
   auto beta_raw = [&](int t) -> float {
     if (t >= r1) return 0.f;
     const int64_t o = (int64_t)t * a.ldb + h;
@@ -84,13 +96,13 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a, int cols) 
   auto stage = [&](int t0, int s) {
     float* base = dl_sm + s * CT * per_tok;
     const int n = min(CT, r1 - t0);
-    for (int it = warp; it < n * 4; it += nw) {      // one warp per (token, operand)
-      const int t = it >> 2, op = it & 3;
-      const float* p = (op == 0 ? src[0] : op == 1 ? src[1] : op == 2 ? src[2] : src[3]) + (int64_t)(t0 + t) * (op == 2 ? HD : a.ld);
-      float* d = base + t * per_tok + op * DK;
-      const int w = op == 3 ? nc : dim;
-      if (VEC) for (int c = lane * 4; c < w; c += 128) dl_cp16(d + c, p + c);
-      else for (int c = lane; c < w; c += 32) dl_cp4(d + c, p + c);
+    // a thread copies one piece (16 bytes, or one number) of an operand for every `tpar`-th token of the stage
+    for (int r = role0; r < roles; r += role_step) {
+      const int op = r < piece_k ? 0 : r < 2 * piece_k ? 1 : r < 3 * piece_k ? 2 : 3, c = (r - op * piece_k) * W;
+      const int64_t step = op == 2 ? HD : a.ld;
+      const float* p = (op == 0 ? src[0] : op == 1 ? src[1] : op == 2 ? src[2] : src[3]) + (int64_t)(t0 + tok0) * step + c;
+      float* d = base + tok0 * per_tok + op * DK + c;
+      for (int t = tok0; t < n; t += tpar, p += step * tpar, d += per_tok * tpar) { if (VEC) dl_cp16(d, p); else dl_cp4(d, p); }
     }
     if (tid < CT) {
       beta_s[s * CT + tid] = 1.f / (1.f + expf(-braw));
@@ -132,12 +144,24 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a, int cols) 
       }
       const float be = beta_s[s * CT + t];
       float v[CPT], u[CPT], dk[CPT], dq[CPT], kq_dot = sum2(kq2);
-      ld4(d + 3 * DK + col, v);
+      dl_ld<CPT>(d + 3 * DK + col, v);
 #pragma unroll
       for (int j = 0; j < CPT; ++j) { dk[j] = sum2(dk2[j]); dq[j] = sum2(dq2[j]); }
 #pragma unroll
       for (int off = 1; off < KQ; off <<= 1) kq_dot += __shfl_xor_sync(0xffffffffu, kq_dot, off);
-      if constexpr (KQ >= 8) {
+      if constexpr (CPT == 2) {
+        // four sums over the KQ lanes: two exchanges split them (see below)
+        const bool b0 = kq & 1, b1 = kq & 2;
+        const float x0 = (b0 ? dq[0] : dk[0]) + __shfl_xor_sync(0xffffffffu, b0 ? dk[0] : dq[0], 1);
+        const float x1 = (b0 ? dq[1] : dk[1]) + __shfl_xor_sync(0xffffffffu, b0 ? dk[1] : dq[1], 1);
+        float y = (b1 ? x1 : x0) + __shfl_xor_sync(0xffffffffu, b1 ? x0 : x1, 2);
+#pragma unroll
+        for (int off = 4; off < KQ; off <<= 1) y += __shfl_xor_sync(0xffffffffu, y, off);
+        const int g0 = lane & ~(KQ - 1);
+        u[0] = be * (v[0] - __shfl_sync(0xffffffffu, y, g0));
+        u[1] = be * (v[1] - __shfl_sync(0xffffffffu, y, g0 + 2));
+        if (b0 && kq < 4) { const int j = b1 ? 1 : 0; if (col + j < nc) op[j] = fmaf(kq_dot, b1 ? u[1] : u[0], y); }
+      } else if constexpr (KQ >= 8) {
         // eight sums over the KQ lanes: three exchanges split them, so each lane ends with one; then every lane fetches the
         // four sums along k, and the lanes that hold a sum along q write its output
         const bool b0 = kq & 1, b1 = kq & 2, b2 = kq & 4;
@@ -147,7 +171,9 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a, int cols) 
 #pragma unroll
         for (int j = 0; j < 2; ++j) z[j] = (b1 ? x[2 + j] : x[j]) + __shfl_xor_sync(0xffffffffu, b1 ? x[j] : x[2 + j], 2);
         float y = (b2 ? z[1] : z[0]) + __shfl_xor_sync(0xffffffffu, b2 ? z[0] : z[1], 4);
-        if constexpr (KQ == 16) y += __shfl_xor_sync(0xffffffffu, y, 8);
+        
+#pragma unroll
+        for (int off = 8; off < KQ; off <<= 1) y += __shfl_xor_sync(0xffffffffu, y, off);
         const int g0 = lane & ~(KQ - 1);
 #pragma unroll
         for (int j = 0; j < 4; ++j) u[j] = be * (v[j] - __shfl_sync(0xffffffffu, y, g0 + (j >> 1) * 2 + (j & 1) * 4));
@@ -164,7 +190,7 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a, int cols) 
 #pragma unroll
         for (int j = 0; j < CPT; ++j) { u[j] = be * (v[j] - dk[j]); dq[j] = fmaf(kq_dot, u[j], dq[j]); }
         if (kq == 0 && col < nc) {
-          if (VEC) st4(op, dq);
+          if (VEC) dl_st<CPT>(op, dq);
           else {
 #pragma unroll
             for (int j = 0; j < CPT; ++j) if (col + j < nc) op[j] = dq[j];
@@ -182,14 +208,14 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a, int cols) 
   }
 #pragma unroll
   for (int i = 0; i < NP; ++i) {
-    float x[2][4];
+    float x[2][CPT];
 #pragma unroll
     for (int j = 0; j < CPT; ++j) upk(S[i][j], x[0][j], x[1][j]);
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int k = chan(i) + e;
       if (k < dim) {
-        if (VEC) { if (col < nc) st4(Sg + (int64_t)k * vdim + col, x[e]); }
+        if (VEC) { if (col < nc) dl_st<CPT>(Sg + (int64_t)k * vdim + col, x[e]); }
         else {
 #pragma unroll
           for (int j = 0; j < CPT; ++j) if (col + j < nc) Sg[(int64_t)k * vdim + col + j] = x[e][j];
@@ -199,14 +225,14 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(DeltaArgs a, int cols) 
   }
 }
 
-template <int KQ, int KPT, int CT>
+template <int KQ, int KPT, int CPT, int CT>
 int delta_launch(const DeltaArgs& a, bool vec, cudaStream_t st) {
-  // up to four warps per block; fewer (more blocks) for heads with few columns
-  const int warp_cols = 32 / KQ * 4;
-  const int warps = std::min(4, (a.vdim + warp_cols - 1) / warp_cols), cols = warps * warp_cols;
+  // up to eight warps per block; fewer (more blocks) for heads with few columns
+  const int warp_cols = 32 / KQ * CPT;
+  const int warps = std::min(8, (a.vdim + warp_cols - 1) / warp_cols), cols = warps * warp_cols;
   const dim3 grid((a.vdim + cols - 1) / cols, a.H, a.B), block(warps * 32);
   const size_t smem = (size_t)(2 * CT * (3 * KQ * KPT + ((cols + 3) & ~3)) + 2 * CT) * 4;
-  auto kern = vec ? delta_scan_kernel<KQ, KPT, CT, true> : delta_scan_kernel<KQ, KPT, CT, false>;
+  auto kern = vec ? delta_scan_kernel<KQ, KPT, CPT, CT, true> : delta_scan_kernel<KQ, KPT, CPT, CT, false>;
   if (smem > 48 * 1024) KGE_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   KGE_CUDA_OK(launch_pdl(kern, grid, block, smem, st, a, cols));
   return 0;
@@ -220,15 +246,15 @@ int delta_scan(const DeltaArgs& a, cudaStream_t st) {
   const bool vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && a.ld % 4 == 0 && a.slot_stride % 4 == 0 &&
                    ((reinterpret_cast<uintptr_t>(a.qkv) | reinterpret_cast<uintptr_t>(a.decay) | reinterpret_cast<uintptr_t>(a.o32) | reinterpret_cast<uintptr_t>(a.state)) & 15) == 0;
   if (a.T == a.B) {               // one row per request: one token per stage
-    if (a.dim <= 32) return delta_launch<4, 8, 1>(a, vec, st);
-    if (a.dim <= 64) return delta_launch<4, 16, 1>(a, vec, st);
-    if (a.dim <= 128) return delta_launch<8, 16, 1>(a, vec, st);
-    return delta_launch<16, 16, 1>(a, vec, st);
+    if (a.dim <= 32) return delta_launch<4, 8, 4, 1>(a, vec, st);
+    if (a.dim <= 64) return delta_launch<4, 16, 4, 1>(a, vec, st);
+    if (a.dim <= 128) return delta_launch<8, 16, 4, 1>(a, vec, st);
+    return delta_launch<16, 16, 4, 1>(a, vec, st);
   }
-  if (a.dim <= 32) return delta_launch<4, 8, 8>(a, vec, st);
-  if (a.dim <= 64) return delta_launch<4, 16, 8>(a, vec, st);
-  if (a.dim <= 128) return delta_launch<8, 16, 8>(a, vec, st);
-  return delta_launch<16, 16, 4>(a, vec, st);
+  if (a.dim <= 32) return delta_launch<4, 8, 2, 16>(a, vec, st);
+  if (a.dim <= 64) return delta_launch<4, 16, 2, 16>(a, vec, st);
+  if (a.dim <= 128) return delta_launch<8, 16, 2, 16>(a, vec, st);
+  return delta_launch<16, 16, 2, 8>(a, vec, st);
 }
 
 }  // namespace kge

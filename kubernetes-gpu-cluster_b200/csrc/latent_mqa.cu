@@ -2,10 +2,10 @@
 // the head's key up-projection, so one row [c | turned key part] per token serves all heads as key (the whole row) and as
 // value (its c part), and a row is read once per 16 (token, head) pairs instead of once per head.
 // A CTA of eight warps owns 16 query rows - consecutive (token, head) pairs of one request - and walks its part of the
-// visible keys in tiles of 32, staged in shared memory by cp.async three tiles ahead:
-//   S = Q K^T   mma.sync m16n8k16, each warp every eighth 16-column step of all 32 keys (its part of Q stays in registers),
+// visible keys in tiles of 64, staged in shared memory by cp.async in halves of 32, up to three halves ahead:
+//   S = Q K^T   mma.sync m16n8k16, each warp every eighth 16-column step of all 64 keys (its part of Q stays in registers),
 //               the warps' fp32 parts summed through shared memory
-//   softmax     two rows per warp, one key per lane: window mask, running maximum and sum in fp32, P in bfloat16
+//   softmax     two rows per warp, two keys per lane: window mask, running maximum and sum in fp32, P in bfloat16
 //   O += P C    each warp its share of the kv_rank columns, fp32 accumulators in registers
 // Decode steps split the key range over several CTAs (too few requests to fill the GPU otherwise); a second kernel merges
 // their (m, l, O) and adds the sink's share of the denominator.  HBM-bound: a row's bytes are used for 2 * 16 heads' flops.
@@ -18,7 +18,7 @@ namespace kge {
 
 namespace {
 
-constexpr int LM_WARPS = 8, LM_KT = 32, LM_ROWS = 16, LM_PAD = 8, LM_ST = 4, LM_KSW = 5;      // LM_KSW: 16-column steps of a row per warp at most
+constexpr int LM_WARPS = 8, LM_KH = 32, LM_KT = 2 * LM_KH, LM_ROWS = 16, LM_PAD = 8, LM_KSW = 5;      // LM_KSW: 16-column steps of a row per warp at most
 constexpr float LM_LOG2E = 1.4426950408889634f;
 typedef __nv_bfloat16 lm_bf16;
 
@@ -40,19 +40,19 @@ __device__ __forceinline__ void lm_mma(float (&c)[4], const uint32_t (&a)[4], ui
 }
 
 constexpr int LM_SLD = LM_KT + 4, LM_PLD = LM_KT + 8;
-size_t lm_smem(int dim) {
-  return (size_t)LM_ST * LM_KT * (dim + LM_PAD) * 2 + (size_t)LM_WARPS * LM_ROWS * LM_SLD * 4 + (size_t)LM_ROWS * LM_PLD * 2 + 3 * LM_ROWS * 4;
+size_t lm_smem(int dim, int st) {
+  return (size_t)st * LM_KH * (dim + LM_PAD) * 2 + (size_t)LM_WARPS * LM_ROWS * LM_SLD * 4 + (size_t)LM_ROWS * LM_PLD * 2 + 3 * LM_ROWS * 4;
 }
 
-// VP: 16-column pairs of the output per warp
-template <int VP>
+// VP: 16-column pairs of the output per warp; ST: stages of 32 keys (two are computed on, the others are in flight)
+template <int VP, int ST>
 __global__ void __launch_bounds__(LM_WARPS * 32) latent_mqa_kernel(LatentMqaArgs a) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) unsigned char lm_raw[];
   const int dim = a.kv_rank + a.rot_part, ld = dim + LM_PAD, H = a.H;
   lm_bf16* Ks = reinterpret_cast<lm_bf16*>(lm_raw);
-  float* Ss = reinterpret_cast<float*>(Ks + LM_ST * LM_KT * ld);     // [warps][16][32]: every warp's part of the scores
+  float* Ss = reinterpret_cast<float*>(Ks + ST * LM_KH * ld);     // [warps][16][64]: every warp's part of the scores
   lm_bf16* Ps = reinterpret_cast<lm_bf16*>(Ss + LM_WARPS * LM_ROWS * LM_SLD);
   float* cs = reinterpret_cast<float*>(Ps + LM_ROWS * LM_PLD);      // [16] correction of this tile, then [16] m, [16] l
   const int b = a.req0 + blockIdx.z, rs = a.qsl[b], nrows = (a.qsl[b + 1] - rs) * H, R0 = blockIdx.x * LM_ROWS;
@@ -65,27 +65,38 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_mqa_kernel(LatentMqaArgs
   const int chunks = dim >> 3, bs_shift = 31 - __clz(a.block_size);
   const int32_t* bt = a.block_table + (int64_t)b * a.max_blocks;
   const lm_bf16* cache = (const lm_bf16*)a.cache;
-  // a warp stages 4 of a tile's 32 rows; where they live is looked up a tile earlier than it is needed
-  auto lookup = [&](int kt) -> int64_t {
-    const int j = min(lo_min + kt * LM_KT + warp * 4 + (lane & 3), pos_last);
-    return kt < t1 ? ((int64_t)bt[j >> bs_shift] << bs_shift) + (j & (a.block_size - 1)) : 0;
+  // a warp copies 4 of a stage's 32 rows, the lanes sharing their 16-byte pieces evenly (the same pieces every time); where the
+  // rows live is looked up a step before it is needed
+  const int h1 = 2 * t1;                              // stages of 32 keys: 2 t0 .. 2 t1 - 1
+  auto lookup = [&](int hk) -> int {
+    const int j = min(lo_min + hk * LM_KH + warp * 4 + (lane & 3), pos_last);
+    return hk < h1 ? (bt[j >> bs_shift] << bs_shift) + (j & (a.block_size - 1)) : 0;
   };
-  auto stage = [&](int kt, int64_t row) {
-    if (kt < t1) {
-      lm_bf16* dst = Ks + ((kt - t0) % LM_ST * LM_KT + warp * 4) * ld;
+  constexpr int NPC = 10;                             // pieces per lane at most: 4 rows of 80
+  int pr_[NPC];                                       // row (of the warp's four) and piece, packed; -1: none
 #pragma unroll
-      for (int r = 0; r < 4; ++r) {
-        const int64_t rr = __shfl_sync(0xffffffffu, row, r);
-        const bool ok = lo_min + kt * LM_KT + warp * 4 + r <= pos_last;
-        const lm_bf16* src = cache + rr * dim;
-        for (int c = lane; c < chunks; c += 32) lm_cp16(lm_saddr(dst + r * ld + c * 8), src + c * 8, ok);
+  for (int i = 0; i < NPC; ++i) {
+    const int idx = lane + 32 * i;
+    pr_[i] = idx < 4 * chunks ? (idx / chunks) << 16 | (idx % chunks) : -1;
+  }
+  int slot = 0;                                       // where the next stage goes
+  auto stage = [&](int hk, int row) {
+    if (hk < h1) {
+      lm_bf16* dst = Ks + (slot * LM_KH + warp * 4) * ld;
+      const int left = pos_last - (lo_min + hk * LM_KH + warp * 4);      // the last of the warp's rows that exists
+#pragma unroll
+      for (int i = 0; i < NPC; ++i) {
+        const int r = pr_[i] >> 16, c = (pr_[i] & 0xffff) * 8;
+        const int rr = __shfl_sync(0xffffffffu, row, r & 3);
+        if (pr_[i] >= 0) lm_cp16(lm_saddr(dst + r * ld + c), cache + (int64_t)rr * dim + c, r <= left);
       }
     }
+    slot = slot + 1 == ST ? 0 : slot + 1;
     asm volatile("cp.async.commit_group;");
   };
 #pragma unroll
-  for (int i = 0; i < LM_ST - 1; ++i) stage(t0 + i, lookup(t0 + i));
-  int64_t nrow = lookup(t0 + LM_ST - 1);
+  for (int i = 0; i < ST - 2; ++i) stage(2 * t0 + i, lookup(2 * t0 + i));
+  int nrow0 = lookup(2 * t0 + ST - 2), nrow1 = lookup(2 * t0 + ST - 1);
   // this warp's 16-column steps (warp, warp + 8, ..) of the 16 query rows, as A fragments (rows beyond the request's repeat its last one; they are never written)
   const int ksteps = dim >> 4, vpairs = a.kv_rank >> 4;
   uint32_t qf[LM_KSW][4];
@@ -117,26 +128,30 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_mqa_kernel(LatentMqaArgs
     rlo[i] = a.window > 0 ? max(0, rpos[i] - a.window + 1) : 0;
   }
   const float scale2 = a.scale * LM_LOG2E;
+  int cur = 0;                                        // the stage that holds the tile's first half
   for (int kt = t0; kt < t1; ++kt) {
-    asm volatile("cp.async.wait_group %0;" ::"n"(LM_ST - 2) : "memory");
-    __syncthreads();                                  // this tile has landed; the readers of the stage refilled next are done
-    stage(kt + LM_ST - 1, nrow);
-    nrow = lookup(kt + LM_ST);
-    const lm_bf16* K = Ks + (kt - t0) % LM_ST * LM_KT * ld;
+    asm volatile("cp.async.wait_group %0;" ::"n"(ST - 4) : "memory");
+    __syncthreads();                                  // this tile's two stages have landed; the readers of the stages refilled next are done
+    stage(2 * kt + ST - 2, nrow0);
+    stage(2 * kt + ST - 1, nrow1);
+    nrow0 = lookup(2 * kt + ST);
+    nrow1 = lookup(2 * kt + ST + 1);
+    const lm_bf16* K[2] = {Ks + cur * LM_KH * ld, Ks + (cur + 1 == ST ? 0 : cur + 1) * LM_KH * ld};
+    cur = cur + 2 >= ST ? cur + 2 - ST : cur + 2;
     {
-      // this warp's columns of all 32 keys: four independent 16 x 8 products, summed over the warps below
-      float sc[4][4];
+      // this warp's columns of all 64 keys: eight independent 16 x 8 products, summed over the warps below
+      float sc[8][4];
 #pragma unroll
-      for (int n = 0; n < 4; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
-      const lm_bf16* kr = K + (lane & 15) * ld + (lane >> 4) * 8;      // ldmatrix rows: 16 keys x two 8-column halves
+      for (int n = 0; n < 8; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
+      const int ko = (lane & 15) * ld + (lane >> 4) * 8;               // ldmatrix rows: 16 keys x two 8-column halves
 #pragma unroll
       for (int i = 0; i < LM_KSW; ++i) {
         const int ks = warp + i * LM_WARPS;
         if (ks < ksteps) {
 #pragma unroll
-          for (int g = 0; g < 2; ++g) {
+          for (int g = 0; g < 4; ++g) {
             uint32_t bb[4];                           // keys g * 16 .. + 7: halves 0 and 2; + 8 .. 15: halves 1 and 3
-            lm_ldm4(bb, lm_saddr(kr + g * 16 * ld + ks * 16));
+            lm_ldm4(bb, lm_saddr(K[g >> 1] + ko + (g & 1) * 16 * ld + ks * 16));
             lm_mma(sc[2 * g], qf[i], bb[0], bb[2]);
             lm_mma(sc[2 * g + 1], qf[i], bb[1], bb[3]);
           }
@@ -144,51 +159,55 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_mqa_kernel(LatentMqaArgs
       }
       float* d0 = Ss + (warp * LM_ROWS + (lane >> 2)) * LM_SLD + (lane & 3) * 2;
 #pragma unroll
-      for (int n = 0; n < 4; ++n) {
+      for (int n = 0; n < 8; ++n) {
         *reinterpret_cast<float2*>(d0 + n * 8) = make_float2(sc[n][0], sc[n][1]);
         *reinterpret_cast<float2*>(d0 + 8 * LM_SLD + n * 8) = make_float2(sc[n][2], sc[n][3]);
       }
     }
     __syncthreads();
     {
-      const int j = lo_min + kt * LM_KT + lane;
+      const int j = lo_min + kt * LM_KT + lane * 2;   // two keys per lane
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
         const int r = warp * 2 + i;
-        float s = 0.f;
+        float x = 0.f, y = 0.f;
 #pragma unroll
-        for (int w = 0; w < LM_WARPS; ++w) s += Ss[(w * LM_ROWS + r) * LM_SLD + lane];
-        s = (j <= rpos[i] && j >= rlo[i]) ? s * scale2 : -INFINITY;
-        const float mn = fmaxf(m[i], warp_max(s));
-        const float p = s == -INFINITY ? 0.f : exp2f(s - mn);
-        const float corr = mn == -INFINITY ? 1.f : exp2f(m[i] - mn);
-        l[i] = l[i] * corr + warp_sum(p);
+        for (int w = 0; w < LM_WARPS; ++w) {
+          const float2 v = *reinterpret_cast<const float2*>(Ss + (w * LM_ROWS + r) * LM_SLD + lane * 2);
+          x += v.x; y += v.y;
+        }
+        x = (j <= rpos[i] && j >= rlo[i]) ? x * scale2 : -INFINITY;
+        y = (j + 1 <= rpos[i] && j + 1 >= rlo[i]) ? y * scale2 : -INFINITY;
+        const float mn = fmaxf(m[i], warp_max(fmaxf(x, y)));
+        const float base = mn == -INFINITY ? 0.f : mn;      // no key yet: every weight is 0
+        const float px = exp2f(x - base), py = exp2f(y - base), corr = exp2f(m[i] - base);
+        l[i] = l[i] * corr + warp_sum(px + py);
         m[i] = mn;
-        Ps[r * LM_PLD + lane] = __float2bfloat16_rn(p);
+        *reinterpret_cast<__nv_bfloat162*>(Ps + r * LM_PLD + lane * 2) = __floats2bfloat162_rn(px, py);
         if (lane == 0) cs[r] = corr;
       }
     }
     __syncthreads();
     {
       const float c0 = cs[lane >> 2], c1 = cs[(lane >> 2) + 8];
-      uint32_t p0[4], p1[4];
+      uint32_t pf[4][4];
       const uint32_t pa = lm_saddr(Ps + (lane & 15) * LM_PLD + (lane >> 4) * 8);
-      lm_ldm4(p0, pa);
-      lm_ldm4(p1, pa + 32);
+#pragma unroll
+      for (int g = 0; g < 4; ++g) lm_ldm4(pf[g], pa + g * 32);
 #pragma unroll
       for (int v = 0; v < VP; ++v) {
         const int pr = warp + v * LM_WARPS;
         if (pr < vpairs) {
 #pragma unroll
           for (int n = 0; n < 2; ++n) { o[v][n][0] *= c0; o[v][n][1] *= c0; o[v][n][2] *= c1; o[v][n][3] *= c1; }
-          uint32_t b0[4], b1[4];
-          const uint32_t va = lm_saddr(K + (lane & 15) * ld + pr * 16 + (lane >> 4) * 8);
-          lm_ldm4t(b0, va);
-          lm_ldm4t(b1, va + 16 * ld * 2);
-          lm_mma(o[v][0], p0, b0[0], b0[1]);
-          lm_mma(o[v][1], p0, b0[2], b0[3]);
-          lm_mma(o[v][0], p1, b1[0], b1[1]);
-          lm_mma(o[v][1], p1, b1[2], b1[3]);
+          const int vo = (lane & 15) * ld + pr * 16 + (lane >> 4) * 8;
+#pragma unroll
+          for (int g = 0; g < 4; ++g) {
+            uint32_t bb[4];
+            lm_ldm4t(bb, lm_saddr(K[g >> 1] + vo + (g & 1) * 16 * ld));
+            lm_mma(o[v][0], pf[g], bb[0], bb[1]);
+            lm_mma(o[v][1], pf[g], bb[2], bb[3]);
+          }
         }
       }
     }
@@ -277,12 +296,16 @@ __global__ void __launch_bounds__(128) latent_mqa_merge_kernel(LatentMqaArgs a, 
   }
 }
 
+template <int VP, int ST>
+int lm_launch_st(const LatentMqaArgs& a, cudaStream_t st) {
+  const size_t smem = lm_smem(a.kv_rank + a.rot_part, ST);
+  KGE_CUDA_OK(cudaFuncSetAttribute(latent_mqa_kernel<VP, ST>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  KGE_CUDA_OK(launch_pdl(latent_mqa_kernel<VP, ST>, dim3((a.max_q * a.H + LM_ROWS - 1) / LM_ROWS, a.splits, a.B), dim3(LM_WARPS * 32), smem, st, a));
+  return 0;
+}
 template <int VP>
 int lm_launch(const LatentMqaArgs& a, cudaStream_t st) {
-  const size_t smem = lm_smem(a.kv_rank + a.rot_part);
-  KGE_CUDA_OK(cudaFuncSetAttribute(latent_mqa_kernel<VP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-  KGE_CUDA_OK(launch_pdl(latent_mqa_kernel<VP>, dim3((a.max_q * a.H + LM_ROWS - 1) / LM_ROWS, a.splits, a.B), dim3(LM_WARPS * 32), smem, st, a));
-  return 0;
+  return lm_smem(a.kv_rank + a.rot_part, 5) <= 227 * 1024 ? lm_launch_st<VP, 5>(a, st) : lm_launch_st<VP, 4>(a, st);
 }
 
 }  // namespace
@@ -290,10 +313,10 @@ int lm_launch(const LatentMqaArgs& a, cudaStream_t st) {
 bool latent_mqa_ok(int H, int kv_rank, int rot_part, int block_size) {
   return H > 0 && kv_rank % 16 == 0 && rot_part % 16 == 0 && kv_rank > 0 && kv_rank <= 512 && kv_rank + rot_part <= 16 * LM_KSW * LM_WARPS && block_size > 0 && (block_size & (block_size - 1)) == 0;
 }
-// parts the key range is cut into: a CTA per SM (their stages fill its shared memory), at least two tiles of keys each
+// parts the key range is cut into: a CTA per SM (their stages fill its shared memory), at least 64 keys each
 int latent_mqa_splits(int B, int H, int max_q, int64_t keys) {
   const int64_t tiles = (int64_t)B * ((max_q * H + LM_ROWS - 1) / LM_ROWS);
-  const int64_t want = 148 / std::max<int64_t>(tiles, 1), most = keys / (2 * LM_KT);
+  const int64_t want = 148 / std::max<int64_t>(tiles, 1), most = keys / LM_KT;
   return (int)std::max<int64_t>(1, std::min<int64_t>(std::min(want, most), 16));
 }
 int64_t latent_mqa_workspace(int T, int H, int kv_rank, int splits) { return splits > 1 ? (int64_t)splits * T * H * (kv_rank + 2) * 4 : 0; }
