@@ -227,9 +227,9 @@ __global__ void __launch_bounds__(256) delta_scan_kernel(DeltaArgs a, int cols) 
 
 template <int KQ, int KPT, int CPT, int CT>
 int delta_launch(const DeltaArgs& a, bool vec, cudaStream_t st) {
-  // up to eight warps per block; fewer (more blocks) for heads with few columns
+  // up to eight warps per block (four in one-token steps); fewer (more blocks) for heads with few columns
   const int warp_cols = 32 / KQ * CPT;
-  const int warps = std::min(8, (a.vdim + warp_cols - 1) / warp_cols), cols = warps * warp_cols;
+  const int warps = std::min(CT == 1 ? 4 : 8, (a.vdim + warp_cols - 1) / warp_cols), cols = warps * warp_cols;
   const dim3 grid((a.vdim + cols - 1) / cols, a.H, a.B), block(warps * 32);
   const size_t smem = (size_t)(2 * CT * (3 * KQ * KPT + ((cols + 3) & ~3)) + 2 * CT) * 4;
   auto kern = vec ? delta_scan_kernel<KQ, KPT, CPT, CT, true> : delta_scan_kernel<KQ, KPT, CPT, CT, false>;

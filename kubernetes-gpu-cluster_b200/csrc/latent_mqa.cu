@@ -1,11 +1,11 @@
 // Attention of all query heads of a request over its cached latent rows: every head's query has already been multiplied by
 // the head's key up-projection, so one row [c | turned key part] per token serves all heads as key (the whole row) and as
 // value (its c part), and a row is read once per 16 (token, head) pairs instead of once per head.
-// A CTA of eight warps owns 16 query rows - consecutive (token, head) pairs of one request - and walks its part of the
+// A CTA of sixteen warps owns 16 query rows - consecutive (token, head) pairs of one request - and walks its part of the
 // visible keys in tiles of 64, staged in shared memory by cp.async in halves of 32, up to three halves ahead:
-//   S = Q K^T   mma.sync m16n8k16, each warp every eighth 16-column step of all 64 keys (its part of Q stays in registers),
+//   S = Q K^T   mma.sync m16n8k16, each warp every eighth 16-column step of half the keys (its part of Q stays in registers),
 //               the warps' fp32 parts summed through shared memory
-//   softmax     two rows per warp, two keys per lane: window mask, running maximum and sum in fp32, P in bfloat16
+//   softmax     one row per warp, two keys per lane: window mask, running maximum and sum in fp32, P in bfloat16
 //   O += P C    each warp its share of the kv_rank columns, fp32 accumulators in registers
 // Decode steps split the key range over several CTAs (too few requests to fill the GPU otherwise); a second kernel merges
 // their (m, l, O) and adds the sink's share of the denominator.  HBM-bound: a row's bytes are used for 2 * 16 heads' flops.
@@ -18,7 +18,7 @@ namespace kge {
 
 namespace {
 
-constexpr int LM_WARPS = 8, LM_KH = 32, LM_KT = 2 * LM_KH, LM_ROWS = 16, LM_PAD = 8, LM_KSW = 5;      // LM_KSW: 16-column steps of a row per warp at most
+constexpr int LM_WARPS = 16, LM_KW = 8, LM_KH = 32, LM_KT = 2 * LM_KH, LM_ROWS = 16, LM_PAD = 8, LM_KSW = 5;      // LM_KW: warps that share a row's columns; LM_KSW: 16-column steps per warp at most
 constexpr float LM_LOG2E = 1.4426950408889634f;
 typedef __nv_bfloat16 lm_bf16;
 
@@ -39,9 +39,11 @@ __device__ __forceinline__ void lm_mma(float (&c)[4], const uint32_t (&a)[4], ui
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
+__device__ __forceinline__ float lm_ex2(float x) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x)); return y; }
+
 constexpr int LM_SLD = LM_KT + 4, LM_PLD = LM_KT + 8;
 size_t lm_smem(int dim, int st) {
-  return (size_t)st * LM_KH * (dim + LM_PAD) * 2 + (size_t)LM_WARPS * LM_ROWS * LM_SLD * 4 + (size_t)LM_ROWS * LM_PLD * 2 + 3 * LM_ROWS * 4;
+  return (size_t)st * LM_KH * (dim + LM_PAD) * 2 + (size_t)LM_KW * LM_ROWS * LM_SLD * 4 + (size_t)LM_ROWS * LM_PLD * 2 + 3 * LM_ROWS * 4;
 }
 
 // VP: 16-column pairs of the output per warp; ST: stages of 32 keys (two are computed on, the others are in flight)
@@ -52,8 +54,8 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_mqa_kernel(LatentMqaArgs
   extern __shared__ __align__(16) unsigned char lm_raw[];
   const int dim = a.kv_rank + a.rot_part, ld = dim + LM_PAD, H = a.H;
   lm_bf16* Ks = reinterpret_cast<lm_bf16*>(lm_raw);
-  float* Ss = reinterpret_cast<float*>(Ks + ST * LM_KH * ld);     // [warps][16][64]: every warp's part of the scores
-  lm_bf16* Ps = reinterpret_cast<lm_bf16*>(Ss + LM_WARPS * LM_ROWS * LM_SLD);
+  float* Ss = reinterpret_cast<float*>(Ks + ST * LM_KH * ld);     // [8][16][64]: the warps' parts of the scores
+  lm_bf16* Ps = reinterpret_cast<lm_bf16*>(Ss + LM_KW * LM_ROWS * LM_SLD);
   float* cs = reinterpret_cast<float*>(Ps + LM_ROWS * LM_PLD);      // [16] correction of this tile, then [16] m, [16] l
   const int b = a.req0 + blockIdx.z, rs = a.qsl[b], nrows = (a.qsl[b + 1] - rs) * H, R0 = blockIdx.x * LM_ROWS;
   if (R0 >= nrows) return;
@@ -65,29 +67,29 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_mqa_kernel(LatentMqaArgs
   const int chunks = dim >> 3, bs_shift = 31 - __clz(a.block_size);
   const int32_t* bt = a.block_table + (int64_t)b * a.max_blocks;
   const lm_bf16* cache = (const lm_bf16*)a.cache;
-  // a warp copies 4 of a stage's 32 rows, the lanes sharing their 16-byte pieces evenly (the same pieces every time); where the
+  // a warp copies 2 of a stage's 32 rows, the lanes sharing their 16-byte pieces evenly (the same pieces every time); where the
   // rows live is looked up a step before it is needed
   const int h1 = 2 * t1;                              // stages of 32 keys: 2 t0 .. 2 t1 - 1
   auto lookup = [&](int hk) -> int {
-    const int j = min(lo_min + hk * LM_KH + warp * 4 + (lane & 3), pos_last);
+    const int j = min(lo_min + hk * LM_KH + warp * 2 + (lane & 1), pos_last);
     return hk < h1 ? (bt[j >> bs_shift] << bs_shift) + (j & (a.block_size - 1)) : 0;
   };
-  constexpr int NPC = 10;                             // pieces per lane at most: 4 rows of 80
-  int pr_[NPC];                                       // row (of the warp's four) and piece, packed; -1: none
+  constexpr int NPC = 5;                              // pieces per lane at most: 2 rows of 80
+  int pr_[NPC];                                       // row (of the warp's two) and piece, packed; -1: none
 #pragma unroll
   for (int i = 0; i < NPC; ++i) {
     const int idx = lane + 32 * i;
-    pr_[i] = idx < 4 * chunks ? (idx / chunks) << 16 | (idx % chunks) : -1;
+    pr_[i] = idx < 2 * chunks ? (idx / chunks) << 16 | (idx % chunks) : -1;
   }
   int slot = 0;                                       // where the next stage goes
   auto stage = [&](int hk, int row) {
     if (hk < h1) {
-      lm_bf16* dst = Ks + (slot * LM_KH + warp * 4) * ld;
-      const int left = pos_last - (lo_min + hk * LM_KH + warp * 4);      // the last of the warp's rows that exists
+      lm_bf16* dst = Ks + (slot * LM_KH + warp * 2) * ld;
+      const int left = pos_last - (lo_min + hk * LM_KH + warp * 2);      // the last of the warp's rows that exists
 #pragma unroll
       for (int i = 0; i < NPC; ++i) {
         const int r = pr_[i] >> 16, c = (pr_[i] & 0xffff) * 8;
-        const int rr = __shfl_sync(0xffffffffu, row, r & 3);
+        const int rr = __shfl_sync(0xffffffffu, row, r & 1);
         if (pr_[i] >= 0) lm_cp16(lm_saddr(dst + r * ld + c), cache + (int64_t)rr * dim + c, r <= left);
       }
     }
@@ -97,7 +99,9 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_mqa_kernel(LatentMqaArgs
 #pragma unroll
   for (int i = 0; i < ST - 2; ++i) stage(2 * t0 + i, lookup(2 * t0 + i));
   int nrow0 = lookup(2 * t0 + ST - 2), nrow1 = lookup(2 * t0 + ST - 1);
-  // this warp's 16-column steps (warp, warp + 8, ..) of the 16 query rows, as A fragments (rows beyond the request's repeat its last one; they are never written)
+  // a warp takes 32 of a tile's 64 keys and every eighth 16-column step of their rows
+  const int kw = warp % LM_KW, half = warp / LM_KW;
+  // its steps (kw, kw + 8, ..) of the 16 query rows, as A fragments (rows beyond the request's repeat its last one; they are never written)
   const int ksteps = dim >> 4, vpairs = a.kv_rank >> 4;
   uint32_t qf[LM_KSW][4];
   {
@@ -105,7 +109,7 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_mqa_kernel(LatentMqaArgs
     const lm_bf16 *q0 = q + (int64_t)min(R0 + (lane >> 2), nrows - 1) * dim, *q1 = q + (int64_t)min(R0 + (lane >> 2) + 8, nrows - 1) * dim;
 #pragma unroll
     for (int i = 0; i < LM_KSW; ++i) {
-      const int c = (warp + i * LM_WARPS) * 16;
+      const int c = (kw + i * LM_KW) * 16;
       const bool in = c < dim;
       qf[i][0] = in ? *reinterpret_cast<const uint32_t*>(q0 + c) : 0u;
       qf[i][1] = in ? *reinterpret_cast<const uint32_t*>(q1 + c) : 0u;
@@ -118,14 +122,13 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_mqa_kernel(LatentMqaArgs
   for (int v = 0; v < VP; ++v)
 #pragma unroll
     for (int n = 0; n < 2; ++n) o[v][n][0] = o[v][n][1] = o[v][n][2] = o[v][n][3] = 0.f;
-  float m[2], l[2];
-  int rpos[2], rlo[2];
-#pragma unroll
-  for (int i = 0; i < 2; ++i) {                       // the rows whose softmax this warp keeps
-    const int r = R0 + warp * 2 + i;
-    m[i] = -INFINITY; l[i] = 0.f;
-    rpos[i] = r < nrows ? a.positions[rs + r / H] : -1;
-    rlo[i] = a.window > 0 ? max(0, rpos[i] - a.window + 1) : 0;
+  float m, l;
+  int rpos, rlo;
+  {                                                   // the row whose softmax this warp keeps
+    const int r = R0 + warp;
+    m = -INFINITY; l = 0.f;
+    rpos = r < nrows ? a.positions[rs + r / H] : -1;
+    rlo = a.window > 0 ? max(0, rpos - a.window + 1) : 0;
   }
   const float scale2 = a.scale * LM_LOG2E;
   int cur = 0;                                        // the stage that holds the tile's first half
@@ -139,27 +142,28 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_mqa_kernel(LatentMqaArgs
     const lm_bf16* K[2] = {Ks + cur * LM_KH * ld, Ks + (cur + 1 == ST ? 0 : cur + 1) * LM_KH * ld};
     cur = cur + 2 >= ST ? cur + 2 - ST : cur + 2;
     {
-      // this warp's columns of all 64 keys: eight independent 16 x 8 products, summed over the warps below
-      float sc[8][4];
+      // this warp's columns of its 32 keys: four independent 16 x 8 products, summed over the warps below
+      float sc[4][4];
+      const lm_bf16* Kw = half ? K[1] : K[0];
 #pragma unroll
-      for (int n = 0; n < 8; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
+      for (int n = 0; n < 4; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
       const int ko = (lane & 15) * ld + (lane >> 4) * 8;               // ldmatrix rows: 16 keys x two 8-column halves
 #pragma unroll
       for (int i = 0; i < LM_KSW; ++i) {
-        const int ks = warp + i * LM_WARPS;
+        const int ks = kw + i * LM_KW;
         if (ks < ksteps) {
 #pragma unroll
-          for (int g = 0; g < 4; ++g) {
+          for (int g = 0; g < 2; ++g) {
             uint32_t bb[4];                           // keys g * 16 .. + 7: halves 0 and 2; + 8 .. 15: halves 1 and 3
-            lm_ldm4(bb, lm_saddr(K[g >> 1] + ko + (g & 1) * 16 * ld + ks * 16));
+            lm_ldm4(bb, lm_saddr(Kw + ko + g * 16 * ld + ks * 16));
             lm_mma(sc[2 * g], qf[i], bb[0], bb[2]);
             lm_mma(sc[2 * g + 1], qf[i], bb[1], bb[3]);
           }
         }
       }
-      float* d0 = Ss + (warp * LM_ROWS + (lane >> 2)) * LM_SLD + (lane & 3) * 2;
+      float* d0 = Ss + (kw * LM_ROWS + (lane >> 2)) * LM_SLD + half * LM_KH + (lane & 3) * 2;
 #pragma unroll
-      for (int n = 0; n < 8; ++n) {
+      for (int n = 0; n < 4; ++n) {
         *reinterpret_cast<float2*>(d0 + n * 8) = make_float2(sc[n][0], sc[n][1]);
         *reinterpret_cast<float2*>(d0 + 8 * LM_SLD + n * 8) = make_float2(sc[n][2], sc[n][3]);
       }
@@ -167,22 +171,21 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_mqa_kernel(LatentMqaArgs
     __syncthreads();
     {
       const int j = lo_min + kt * LM_KT + lane * 2;   // two keys per lane
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int r = warp * 2 + i;
+      {
+        const int r = warp;
         float x = 0.f, y = 0.f;
 #pragma unroll
-        for (int w = 0; w < LM_WARPS; ++w) {
+        for (int w = 0; w < LM_KW; ++w) {
           const float2 v = *reinterpret_cast<const float2*>(Ss + (w * LM_ROWS + r) * LM_SLD + lane * 2);
           x += v.x; y += v.y;
         }
-        x = (j <= rpos[i] && j >= rlo[i]) ? x * scale2 : -INFINITY;
-        y = (j + 1 <= rpos[i] && j + 1 >= rlo[i]) ? y * scale2 : -INFINITY;
-        const float mn = fmaxf(m[i], warp_max(fmaxf(x, y)));
+        x = (j <= rpos && j >= rlo) ? x * scale2 : -INFINITY;
+        y = (j + 1 <= rpos && j + 1 >= rlo) ? y * scale2 : -INFINITY;
+        const float mn = fmaxf(m, warp_max(fmaxf(x, y)));
         const float base = mn == -INFINITY ? 0.f : mn;      // no key yet: every weight is 0
-        const float px = exp2f(x - base), py = exp2f(y - base), corr = exp2f(m[i] - base);
-        l[i] = l[i] * corr + warp_sum(px + py);
-        m[i] = mn;
+        const float px = lm_ex2(x - base), py = lm_ex2(y - base), corr = lm_ex2(m - base);
+        l = l * corr + warp_sum(px + py);
+        m = mn;
         *reinterpret_cast<__nv_bfloat162*>(Ps + r * LM_PLD + lane * 2) = __floats2bfloat162_rn(px, py);
         if (lane == 0) cs[r] = corr;
       }
@@ -213,8 +216,7 @@ __global__ void __launch_bounds__(LM_WARPS * 32) latent_mqa_kernel(LatentMqaArgs
     }
   }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
-#pragma unroll
-  for (int i = 0; i < 2; ++i) if (lane == 0) { cs[LM_ROWS + warp * 2 + i] = m[i]; cs[2 * LM_ROWS + warp * 2 + i] = l[i]; }
+  if (lane == 0) { cs[LM_ROWS + warp] = m; cs[2 * LM_ROWS + warp] = l; }
   __syncthreads();
   const int64_t grow = (int64_t)rs * H + R0;          // this tile's first row among all (token, head) pairs of the step
   if (a.splits > 1) {
@@ -311,7 +313,7 @@ int lm_launch(const LatentMqaArgs& a, cudaStream_t st) {
 }  // namespace
 
 bool latent_mqa_ok(int H, int kv_rank, int rot_part, int block_size) {
-  return H > 0 && kv_rank % 16 == 0 && rot_part % 16 == 0 && kv_rank > 0 && kv_rank <= 512 && kv_rank + rot_part <= 16 * LM_KSW * LM_WARPS && block_size > 0 && (block_size & (block_size - 1)) == 0;
+  return H > 0 && kv_rank % 16 == 0 && rot_part % 16 == 0 && kv_rank > 0 && kv_rank <= 512 && kv_rank + rot_part <= 16 * LM_KSW * LM_KW && block_size > 0 && (block_size & (block_size - 1)) == 0;
 }
 // parts the key range is cut into: a CTA per SM (their stages fill its shared memory), at least 64 keys each
 int latent_mqa_splits(int B, int H, int max_q, int64_t keys) {
@@ -327,7 +329,7 @@ int latent_mqa(const LatentMqaArgs& a, cudaStream_t st) {
   KGE_REQUIRE(a.splits == 1 || (a.max_q == 1 && a.workspace && a.workspace_bytes >= latent_mqa_workspace(a.T, a.H, a.kv_rank, a.splits)), "latent_mqa: %d parts need one row per request and a workspace", a.splits);
   KGE_REQUIRE(((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.cache) | reinterpret_cast<uintptr_t>(a.out)) & 15) == 0, "latent_mqa: rows must be 16-byte aligned");
   const int pairs = (a.kv_rank / 16 + LM_WARPS - 1) / LM_WARPS;
-  if (int rc = pairs <= 1 ? lm_launch<1>(a, st) : pairs <= 2 ? lm_launch<2>(a, st) : lm_launch<4>(a, st)) return rc;
+  if (int rc = pairs <= 1 ? lm_launch<1>(a, st) : lm_launch<2>(a, st)) return rc;
   // one row per request: the requests' rows follow one another from the first request's on
   if (a.splits > 1) KGE_CUDA_OK(launch_pdl(latent_mqa_merge_kernel, dim3((unsigned)(a.B * a.H)), dim3(128), 0, st, a, (int64_t)a.req0 * a.H));
   return 0;

@@ -135,6 +135,20 @@ __device__ __forceinline__ uint4 load8(const __nv_bfloat16* row, int k, int K, b
   return u.v;
 }
 
+// one output from its sums (row scale applied): the gated pair, or bias and activation; then the multiplier
+template <typename O>
+__device__ __forceinline__ void linear_store(const LinearArgs& a, O* dst, const __nv_bfloat16* bias, int n, float s1, float s2) {
+  float v;
+  if (a.w2) v = glu_apply(a, s1, s2);
+  else {
+    v = s1 + (bias ? ldf(bias + n) : 0.f);
+    v = a.act == ACT_EXP_DECAY ? exp_decay(a.act_coef[n], v) : act_apply(a.act, v);
+  }
+  v *= a.alpha;
+  if (a.accumulate) v += ldf(dst);
+  stf(dst, v);
+}
+
 template <typename O, bool DUAL, int MBK>
 __global__ void __launch_bounds__(256) linear_mma_kernel(LinearArgs a) {
   pdl_launch_dependents();
@@ -244,6 +258,113 @@ __global__ void __launch_bounds__(256) linear_mma_kernel(LinearArgs a) {
     }
 }
 
+// Few rows, 16-byte aligned operands: the weights are the traffic, so they stream through a ring of four k-tiles filled by
+// cp.async three ahead; tiles of 64 rows x 64 weight rows (gated pairs: 32 of each matrix), the same fragments and the same
+// order of summation as above.  Row tiles of 16 without rows (experts with few tokens) are not multiplied.
+constexpr int SBK = 64, SST = 4, SLD = SBK + MPAD;
+constexpr size_t LINEAR_STREAM_SMEM = (size_t)SST * (LBM + LBN) * SLD * 2;
+
+template <typename O, bool DUAL>
+__global__ void __launch_bounds__(256) linear_stream_kernel(LinearArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  typedef __nv_bfloat16 E;
+  constexpr int BN = DUAL ? LBN / 2 : LBN, NT = BN / 32;      // outputs per tile; 8-output tiles per warp
+  const int z = blockIdx.z;
+  int r0 = 0, r1 = a.T;
+  if (a.group_off) { r0 = a.group_off[z]; r1 = a.group_off[z + 1]; }
+  const int m0 = r0 + blockIdx.y * LBM;
+  if (m0 >= r1) return;
+  const int n0 = blockIdx.x * BN, mrows = r1 - m0;
+  const E* x = (const E*)a.x + z * a.x_zs;
+  const E* w = (const E*)a.w + z * a.w_zs;
+  const E* w2 = DUAL ? (const E*)a.w2 + z * a.w_zs : nullptr;
+  const E* bias = a.bias ? (const E*)a.bias + z * a.b_zs : nullptr;
+  O* y = (O*)a.y + z * a.y_zs;
+  extern __shared__ __align__(16) unsigned char ls_raw[];
+  E* xs = reinterpret_cast<E*>(ls_raw);                       // [SST][LBM][SLD]
+  E* ws = xs + SST * LBM * SLD;                               // [SST][LBN][SLD]
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int wm = (warp >> 2) * 32, wn = (warp & 3) * (NT * 8);
+  // staging: thread -> rows tid / 8 and tid / 8 + 32 of both tiles, eight k at (tid % 8) * 8
+  const int sr = tid >> 3, sk = (tid & 7) * 8;
+  const E *xp[2], *wp[2];
+#pragma unroll
+  for (int u = 0; u < 2; ++u) {
+    const int gr = m0 + sr + 32 * u;
+    xp[u] = gr < r1 ? x + (int64_t)(a.xrows ? a.xrows[gr] : gr) * a.ldx : nullptr;
+    const int n = n0 + (DUAL ? sr : sr + 32 * u);
+    wp[u] = n < a.N ? (DUAL && u ? w2 : w) + (int64_t)n * a.K : nullptr;
+  }
+  auto cp = [&](E* dst, const E* row, int k) {
+    const bool ok = row != nullptr && k < a.K;
+    const int sz = ok ? 16 : 0;
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(ok ? row + k : w), "r"(sz));
+  };
+  const int nk = (a.K + SBK - 1) / SBK;
+  auto stage = [&](int kt) {
+    if (kt < nk) {
+      const int st = kt % SST, k = kt * SBK + sk;
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        if (sr + 32 * u < ((mrows + 15) & ~15)) cp(xs + (st * LBM + sr + 32 * u) * SLD + sk, xp[u], k);
+        cp(ws + (st * LBN + sr + 32 * u) * SLD + sk, wp[u], k);
+      }
+    }
+    asm volatile("cp.async.commit_group;");
+  };
+#pragma unroll
+  for (int i = 0; i < SST - 1; ++i) stage(i);
+  float acc[2][NT][4] = {}, acc2[DUAL ? 2 : 1][NT][4] = {};
+  for (int kt = 0; kt < nk; ++kt) {
+    asm volatile("cp.async.wait_group %0;" ::"n"(SST - 2) : "memory");
+    __syncthreads();                                          // this k-tile has landed; the readers of the one refilled next are done
+    stage(kt + SST - 1);
+    const E* xt = xs + kt % SST * LBM * SLD;
+    const E* wt = ws + kt % SST * LBN * SLD;
+#pragma unroll
+    for (int ks = 0; ks < SBK / 16; ++ks) {
+      const int kc = ks * 16 + (lane & 3) * 2;
+      uint32_t b[NT][2], c[DUAL ? NT : 1][2];
+#pragma unroll
+      for (int j = 0; j < NT; ++j) {
+        const E* p = wt + (wn + j * 8 + (lane >> 2)) * SLD + kc;
+        b[j][0] = *reinterpret_cast<const uint32_t*>(p); b[j][1] = *reinterpret_cast<const uint32_t*>(p + 8);
+        if (DUAL) { c[j][0] = *reinterpret_cast<const uint32_t*>(p + 32 * SLD); c[j][1] = *reinterpret_cast<const uint32_t*>(p + 32 * SLD + 8); }
+      }
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        if (wm + i * 16 < mrows) {
+          const E* p = xt + (wm + i * 16 + (lane >> 2)) * SLD + kc;
+          const uint32_t af[4] = {*reinterpret_cast<const uint32_t*>(p), *reinterpret_cast<const uint32_t*>(p + 8 * SLD), *reinterpret_cast<const uint32_t*>(p + 8),
+                                  *reinterpret_cast<const uint32_t*>(p + 8 * SLD + 8)};
+#pragma unroll
+          for (int j = 0; j < NT; ++j) {
+            mma_bf16_16816(acc[i][j], af, b[j][0], b[j][1]);
+            if (DUAL) mma_bf16_16816(acc2[i][j], af, c[j][0], c[j][1]);
+          }
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i)
+#pragma unroll
+    for (int hh = 0; hh < 2; ++hh) {
+      const int r = m0 + wm + i * 16 + (lane >> 2) + hh * 8;
+      if (r >= r1) continue;
+      const float sc = a.row_scale ? a.row_scale[r] : 1.f;
+      const int yr = a.yrows ? a.yrows[r] : r;
+#pragma unroll
+      for (int j = 0; j < NT; ++j)
+#pragma unroll
+        for (int q = 0; q < 2; ++q) {
+          const int n = n0 + wn + j * 8 + (lane & 3) * 2 + q;
+          if (n < a.N) linear_store(a, y + (int64_t)yr * a.ldy + n, bias, n, sc * acc[i][j][hh * 2 + q], DUAL ? sc * acc2[DUAL ? i : 0][j][hh * 2 + q] : 0.f);
+        }
+    }
+}
+
 int linear_any(const LinearArgs& a, cudaStream_t st) {
   KGE_REQUIRE(a.x && a.w && a.y && a.N > 0 && a.K > 0 && a.nz > 0, "linear_any: bad arguments");
   KGE_REQUIRE(a.act != ACT_EXP_DECAY || (a.act_coef && !a.w2), "linear_any: the decay needs its coefficients");
@@ -255,7 +376,14 @@ int linear_any(const LinearArgs& a, cudaStream_t st) {
   const bool f32 = a.elt == KGE_ELT_F32;
   KGE_REQUIRE(!f32 || a.out_f32, "linear_any: float32 storage writes float32");
   if (f32) ce = a.w2 ? launch_pdl(linear_any_kernel<float, float, true>, grid, block, 0, st, a) : launch_pdl(linear_any_kernel<float, float, false>, grid, block, 0, st, a);
-  else if (a.T <= 256) {       // few rows: the weights are the traffic
+  else if (a.T <= 256 && ((reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(a.w2)) & 15) == 0 && a.K % 8 == 0 && a.ldx % 8 == 0 &&
+           a.x_zs % 8 == 0 && a.w_zs % 8 == 0) {
+    if (a.w2) grid.x = (a.N + LBN / 2 - 1) / (LBN / 2);
+    auto kern = a.out_f32 ? (a.w2 ? linear_stream_kernel<float, true> : linear_stream_kernel<float, false>)
+                          : (a.w2 ? linear_stream_kernel<__nv_bfloat16, true> : linear_stream_kernel<__nv_bfloat16, false>);
+    KGE_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)LINEAR_STREAM_SMEM));
+    ce = launch_pdl(kern, grid, block, LINEAR_STREAM_SMEM, st, a);
+  } else if (a.T <= 256) {       // few rows: the weights are the traffic
     if (a.out_f32) ce = a.w2 ? launch_pdl(linear_mma_kernel<float, true, 64>, grid, block, 0, st, a) : launch_pdl(linear_mma_kernel<float, false, 64>, grid, block, 0, st, a);
     else ce = a.w2 ? launch_pdl(linear_mma_kernel<__nv_bfloat16, true, 64>, grid, block, 0, st, a) : launch_pdl(linear_mma_kernel<__nv_bfloat16, false, 64>, grid, block, 0, st, a);
   } else if (a.out_f32) ce = a.w2 ? launch_pdl(linear_mma_kernel<float, true, 32>, grid, block, 0, st, a) : launch_pdl(linear_mma_kernel<float, false, 32>, grid, block, 0, st, a);
