@@ -258,7 +258,7 @@ __global__ void __launch_bounds__(256) linear_mma_kernel(LinearArgs a) {
     }
 }
 
-// Few rows, 16-byte aligned operands: the weights are the traffic, so they stream through a ring of four k-tiles filled by
+// Few rows, 16-byte aligned operands, long sums: the weights are the traffic, so they stream through a ring of four k-tiles filled by
 // cp.async three ahead; tiles of 64 rows x 64 weight rows (gated pairs: 32 of each matrix), the same fragments and the same
 // order of summation as above.  Row tiles of 16 without rows (experts with few tokens) are not multiplied.
 constexpr int SBK = 64, SST = 4, SLD = SBK + MPAD;
@@ -376,7 +376,7 @@ int linear_any(const LinearArgs& a, cudaStream_t st) {
   const bool f32 = a.elt == KGE_ELT_F32;
   KGE_REQUIRE(!f32 || a.out_f32, "linear_any: float32 storage writes float32");
   if (f32) ce = a.w2 ? launch_pdl(linear_any_kernel<float, float, true>, grid, block, 0, st, a) : launch_pdl(linear_any_kernel<float, float, false>, grid, block, 0, st, a);
-  else if (a.T <= 256 && ((reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(a.w2)) & 15) == 0 && a.K % 8 == 0 && a.ldx % 8 == 0 &&
+  else if (a.T <= 256 && a.K >= 256 && ((reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(a.w2)) & 15) == 0 && a.K % 8 == 0 && a.ldx % 8 == 0 &&
            a.x_zs % 8 == 0 && a.w_zs % 8 == 0) {
     if (a.w2) grid.x = (a.N + LBN / 2 - 1) / (LBN / 2);
     auto kern = a.out_f32 ? (a.w2 ? linear_stream_kernel<float, true> : linear_stream_kernel<float, false>)
