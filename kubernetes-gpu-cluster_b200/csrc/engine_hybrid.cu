@@ -530,7 +530,7 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
     e->latq_rows = lat_tc ? std::min(Rm, Tm) : Tm;
     e->qabs = aalloc((int64_t)e->latq_rows * max_abs, es); e->olat = aalloc((int64_t)e->latq_rows * max_olat, es);
     if (!e->qabs || !e->olat) return fail(b.err);
-    if (lat_ws > 0) { e->ws_lat_bytes = lat_ws; e->ws_lat = aalloc(lat_ws, 1); if (!e->ws_lat) return fail(b.err); }
+    if (lat_ws > 0) { e->ws_lat_bytes = lat_ws; e->ws_lat = aalloc(lat_ws, 1); if (!e->ws_lat) return fail(b.err); cudaMemsetAsync(e->ws_lat, 0, (size_t)lat_ws, e->stream); }
     if (lat_tc) {
       // scratch pages for the expanded path: any single request of a step fits (its new rows, the window before them and the
       // rounding to pages and 64-key tiles); steps with more requests go through it in groups
@@ -993,7 +993,6 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
             // a decode step may be replayed as a graph while its contexts grow: sized for the longest context its table holds
             la.splits = latent_mqa_splits(D, H, 1, std::min<int64_t>(window > 0 ? window : (int64_t)1 << 30, (int64_t)max_blocks * bs));
             HFWD(cat, ab, af, latent_mqa(la, st));
-            if (la.splits > 1) ++e->launches;
           }
           if (Ta > D) {
             la.req0 = D; la.B = B - D; la.max_q = maxq; la.splits = 1; la.T = Ta;

@@ -405,8 +405,8 @@ int latent_expand_write(void* k_scratch, void* v_scratch, const void* kv, const 
 // Attention of H query heads over the latent rows (queries already multiplied by the key up-projection: q_abs [T, H, kv_rank +
 // rot_part]): scores scale * q . row, a window (0: the causal prefix), sinks as in AttnBiasArgs, out [T, H, kv_rank] = the
 // weighted sum of the rows' c parts.  bfloat16, kv_rank up to 512 and kv_rank + rot_part up to 640, both multiples of 16:
-// latent_mqa (mma.sync, keys staged once for all heads, key range split over `splits` CTAs of a row tile and merged by a
-// second kernel; workspace of latent_mqa_workspace bytes).
+// latent_mqa (mma.sync, keys staged once for all heads, key range split over `splits` CTAs of a row tile and merged by the
+// last of them; workspace of latent_mqa_workspace bytes, zero before the first launch).
 struct LatentMqaArgs {
   const void* q = nullptr; void* out = nullptr; const void* cache = nullptr;
   const int32_t* block_table = nullptr; int max_blocks = 0; const int32_t* qsl = nullptr; const int32_t* positions = nullptr;

@@ -7,8 +7,8 @@
 //               the warps' fp32 parts summed through shared memory
 //   softmax     one row per warp, two keys per lane: window mask, running maximum and sum in fp32, P in bfloat16
 //   O += P C    each warp its share of the kv_rank columns, fp32 accumulators in registers
-// Decode steps split the key range over several CTAs (too few requests to fill the GPU otherwise); a second kernel merges
-// their (m, l, O) and adds the sink's share of the denominator.  HBM-bound: a row's bytes are used for 2 * 16 heads' flops.
+// Decode steps split the key range over several CTAs (too few requests to fill the GPU otherwise); the CTA
+// that finishes last merges their (m, l, O) and adds the sink's share of the denominator.  HBM-bound: a row's bytes are used for 2 * 16 heads' flops.
 #include <cuda.h>
 
 #include <algorithm>
@@ -65,6 +65,8 @@ constexpr int LM_SLD = LM_KT + 4, LM_PLD = LM_KT + 8;
 size_t lm_smem(int dim, int st) {
   return 1024 + (size_t)st * ((dim + 63) / 64) * LM_BLK + (size_t)LM_KW * LM_ROWS * LM_SLD * 4 + (size_t)LM_ROWS * LM_PLD * 2 + 3 * LM_ROWS * 4 + (size_t)2 * st * 8;
 }
+
+constexpr int LM_COUNTERS = 256;                            // arrival counters of the row tiles, ahead of the parts in the workspace (at most 74: two parts or more of each share 148 SMs)
 
 // VP: 16-column pairs of the output per warp; ST: stages of 32 keys (two are computed on, the others in flight)
 template <int VP, int ST>
@@ -243,9 +245,16 @@ __global__ void __launch_bounds__(LM_WARPS * 32 + 32) latent_mqa_kernel(const __
   lm_sync();
   const int64_t grow = (int64_t)rs * H + R0;          // this tile's first row among all (token, head) pairs of the step
   if (a.splits > 1) {
-    float* po = (float*)a.workspace + ((int64_t)blockIdx.y * a.T * H + grow) * a.kv_rank;
-    float* pm = (float*)a.workspace + (int64_t)a.splits * a.T * H * a.kv_rank + ((int64_t)blockIdx.y * a.T * H + grow) * 2;
-    if (tid < LM_ROWS && R0 + tid < nrows) { pm[tid * 2] = cs[LM_ROWS + tid]; pm[tid * 2 + 1] = cs[2 * LM_ROWS + tid]; }
+    // partial results to the workspace; the CTA of this row tile that arrives last merges them, splits in ascending order of their keys
+    const int64_t rows = (int64_t)a.T * H;
+    int* count = reinterpret_cast<int*>(a.workspace) + (int64_t)blockIdx.z * gridDim.x + blockIdx.x;
+    float* part = reinterpret_cast<float*>(a.workspace) + LM_COUNTERS;
+    float* po = part + ((int64_t)blockIdx.y * rows + grow) * a.kv_rank;
+    float* pm = part + (int64_t)a.splits * rows * a.kv_rank;
+    if (tid < LM_ROWS && R0 + tid < nrows) {
+      float* q = pm + ((int64_t)blockIdx.y * rows + grow + tid) * 2;
+      q[0] = cs[LM_ROWS + tid]; q[1] = cs[2 * LM_ROWS + tid];
+    }
 #pragma unroll
     for (int v = 0; v < VP; ++v) {
       const int pr = warp + v * LM_WARPS;
@@ -258,6 +267,37 @@ __global__ void __launch_bounds__(LM_WARPS * 32 + 32) latent_mqa_kernel(const __
             if (R0 + r < nrows) *reinterpret_cast<float2*>(po + (int64_t)r * a.kv_rank + pr * 16 + n * 8 + (lane & 3) * 2) = make_float2(o[v][n][2 * h], o[v][n][2 * h + 1]);
           }
       }
+    }
+    __threadfence();                                  // this CTA's part is visible device-wide before it counts itself
+    lm_sync();
+    if (tid == 0) reinterpret_cast<int*>(cs)[0] = atomicAdd(count, 1) == a.splits - 1;
+    lm_sync();
+    if (!reinterpret_cast<int*>(cs)[0]) return;
+    __threadfence();
+    if (tid == 0) *count = 0;                         // ready for the next launch
+    const int r = warp;                               // a warp merges one row
+    if (R0 + r >= nrows) return;
+    const float sk = a.sinks ? a.sinks[(R0 + r) % H] * LM_LOG2E : -INFINITY;
+    float M = sk;
+    for (int q = 0; q < a.splits; ++q) M = fmaxf(M, __ldcg(pm + ((int64_t)q * rows + grow + r) * 2));
+    float den = a.sinks ? exp2f(sk - M) : 0.f;        // the sink logit joins the denominator: no key, no value
+    for (int q = 0; q < a.splits; ++q) {
+      const float2 ml = __ldcg(reinterpret_cast<const float2*>(pm + ((int64_t)q * rows + grow + r) * 2));
+      if (ml.x != -INFINITY) den = fmaf(exp2f(ml.x - M), ml.y, den);
+    }
+    const float di = 1.f / den;
+    for (int c = lane * 4; c < a.kv_rank; c += 128) {
+      float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int q = 0; q < a.splits; ++q) {
+        const float mq = __ldcg(pm + ((int64_t)q * rows + grow + r) * 2);
+        if (mq == -INFINITY) continue;                // a part without visible keys
+        const float f = exp2f(mq - M);
+        const float4 v = __ldcg(reinterpret_cast<const float4*>(part + ((int64_t)q * rows + grow + r) * a.kv_rank + c));
+        acc.x = fmaf(f, v.x, acc.x); acc.y = fmaf(f, v.y, acc.y); acc.z = fmaf(f, v.z, acc.z); acc.w = fmaf(f, v.w, acc.w);
+      }
+      __nv_bfloat162 lo = __floats2bfloat162_rn(acc.x * di, acc.y * di), hi = __floats2bfloat162_rn(acc.z * di, acc.w * di);
+      uint2 u; u.x = *reinterpret_cast<uint32_t*>(&lo); u.y = *reinterpret_cast<uint32_t*>(&hi);
+      *reinterpret_cast<uint2*>((lm_bf16*)a.out + (grow + r) * a.kv_rank + c) = u;
     }
     return;
   }
@@ -290,37 +330,6 @@ __global__ void __launch_bounds__(LM_WARPS * 32 + 32) latent_mqa_kernel(const __
   }
 }
 
-// one block per (token, head): the splits' partial results in ascending order of their keys
-__global__ void __launch_bounds__(128) latent_mqa_merge_kernel(LatentMqaArgs a, int64_t row0) {
-  pdl_launch_dependents();
-  pdl_wait();
-  const int64_t row = row0 + blockIdx.x, rows = (int64_t)a.T * a.H;
-  const float* pm = (const float*)a.workspace + (int64_t)a.splits * rows * a.kv_rank + row * 2;
-  float M = a.sinks ? a.sinks[row % a.H] * LM_LOG2E : -INFINITY;
-  const float sk = M;
-  for (int s = 0; s < a.splits; ++s) M = fmaxf(M, pm[(int64_t)s * rows * 2]);
-  float den = a.sinks ? exp2f(sk - M) : 0.f;
-  for (int s = 0; s < a.splits; ++s) {
-    const float ms = pm[(int64_t)s * rows * 2];
-    if (ms != -INFINITY) den = fmaf(exp2f(ms - M), pm[(int64_t)s * rows * 2 + 1], den);
-  }
-  const float inv = 1.f / den;
-  for (int c = threadIdx.x * 4; c < a.kv_rank; c += 512) {
-    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 4
-    for (int s = 0; s < a.splits; ++s) {
-      const float ms = pm[(int64_t)s * rows * 2];
-      if (ms == -INFINITY) continue;                  // a part without visible keys
-      const float f = exp2f(ms - M);
-      const float4 v = *reinterpret_cast<const float4*>((const float*)a.workspace + ((int64_t)s * rows + row) * a.kv_rank + c);
-      acc.x = fmaf(f, v.x, acc.x); acc.y = fmaf(f, v.y, acc.y); acc.z = fmaf(f, v.z, acc.z); acc.w = fmaf(f, v.w, acc.w);
-    }
-    __nv_bfloat162 lo = __floats2bfloat162_rn(acc.x * inv, acc.y * inv), hi = __floats2bfloat162_rn(acc.z * inv, acc.w * inv);
-    uint2 u; u.x = *reinterpret_cast<uint32_t*>(&lo); u.y = *reinterpret_cast<uint32_t*>(&hi);
-    *reinterpret_cast<uint2*>((lm_bf16*)a.out + row * a.kv_rank + c) = u;
-  }
-}
-
 template <int VP, int ST>
 int lm_launch_st(const LatentMqaArgs& a, cudaStream_t st) {
   const int dim = a.kv_rank + a.rot_part;
@@ -347,18 +356,16 @@ int latent_mqa_splits(int B, int H, int max_q, int64_t keys) {
   const int64_t want = 148 / std::max<int64_t>(tiles, 1), most = keys / LM_KT;
   return (int)std::max<int64_t>(1, std::min<int64_t>(std::min(want, most), 16));
 }
-int64_t latent_mqa_workspace(int T, int H, int kv_rank, int splits) { return splits > 1 ? (int64_t)splits * T * H * (kv_rank + 2) * 4 : 0; }
+int64_t latent_mqa_workspace(int T, int H, int kv_rank, int splits) { return splits > 1 ? LM_COUNTERS * 4 + (int64_t)splits * T * H * (kv_rank + 2) * 4 : 0; }
 
 int latent_mqa(const LatentMqaArgs& a, cudaStream_t st) {
   if (a.B <= 0) return 0;
   KGE_REQUIRE(latent_mqa_ok(a.H, a.kv_rank, a.rot_part, a.block_size) && a.B <= 65535 && a.splits >= 1, "latent_mqa: %d heads over rows of %d + %d", a.H, a.kv_rank, a.rot_part);
   KGE_REQUIRE(a.splits == 1 || (a.max_q == 1 && a.workspace && a.workspace_bytes >= latent_mqa_workspace(a.T, a.H, a.kv_rank, a.splits)), "latent_mqa: %d parts need one row per request and a workspace", a.splits);
+  KGE_REQUIRE(a.splits == 1 || (int64_t)a.B * ((a.H + LM_ROWS - 1) / LM_ROWS) <= LM_COUNTERS, "latent_mqa: %d parts of too many row tiles", a.splits);
   KGE_REQUIRE(((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.cache) | reinterpret_cast<uintptr_t>(a.out)) & 15) == 0, "latent_mqa: rows must be 16-byte aligned");
   const int pairs = (a.kv_rank / 16 + LM_WARPS - 1) / LM_WARPS;
-  if (int rc = pairs <= 1 ? lm_launch<1>(a, st) : lm_launch<2>(a, st)) return rc;
-  // one row per request: the requests' rows follow one another from the first request's on
-  if (a.splits > 1) KGE_CUDA_OK(launch_pdl(latent_mqa_merge_kernel, dim3((unsigned)(a.B * a.H)), dim3(128), 0, st, a, (int64_t)a.req0 * a.H));
-  return 0;
+  return pairs <= 1 ? lm_launch<1>(a, st) : lm_launch<2>(a, st);
 }
 
 }  // namespace kge
