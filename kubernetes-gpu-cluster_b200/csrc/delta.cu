@@ -12,6 +12,7 @@
 
 #include "common.cuh"
 #include "elt_access.cuh"
+#include "f32x2.cuh"
 #include "hybrid_ops.h"
 
 namespace kge {
@@ -32,13 +33,7 @@ template <int N> __device__ __forceinline__ void dl_st(float* p, const float (&v
   if constexpr (N == 4) st4(p, v);
   else *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
 }
-// two fp32 lanes per instruction: a pair holds two neighbouring key channels of one column
-typedef unsigned long long f2;
-__device__ __forceinline__ f2 pk(float lo, float hi) { f2 r; asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi)); return r; }
-__device__ __forceinline__ void upk(f2 v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
-__device__ __forceinline__ f2 fma2(f2 a, f2 b, f2 c) { f2 r; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c)); return r; }
-__device__ __forceinline__ f2 mul2(f2 a, f2 b) { f2 r; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b)); return r; }
-__device__ __forceinline__ float sum2(f2 v) { float a, b; upk(v, a, b); return a + b; }
+// a packed pair holds two neighbouring key channels of one column
 
 // KQ lanes x KPT channels cover dim; CPT columns per thread; a block owns `cols` value columns from blockIdx.x * cols on.
 // VEC: operand rows in 16-byte pieces, state rows and outputs in pieces of CPT columns.

@@ -97,6 +97,17 @@ struct HybridLayerW {
   HybMat g2;
   int off_b = 0;
   float* decay_coef = nullptr;
+  // selective scan: `proj` holds [x | z], conv_w the convolution transposed [taps, channels] with its bias conv_b, xproj the rows
+  // [dt | B | C] that read its output, dtproj the steps' second projection (with their bias), ssm_a = -exp(A_log) [channels, n_state] and
+  // ssm_d (fp32).  Windowed attention beside a state-space dual recurrence: `proj` holds [q | k | v | g | z | x | B | C | dt] (offsets
+  // off_k, off_v, off_mg, off_z, off_x, off_dt), `o` / `o2` / side_norm as below, ssm_a = exp(A_log), ssm_d and ssm_dt_bias [m_heads], wkv_norm
+  // the weight of the gated norm
+  HybMat xproj, dtproj;
+  float *ssm_a = nullptr, *ssm_d = nullptr, *ssm_dt_bias = nullptr;
+  int off_z = 0, off_x = 0, off_dt = 0;
+  // Dynamic Tanh (0: mixer, 1: feed-forward): its scalar and its shift (the weight is norm1 / norm2)
+  float dyt_alpha[2] = {0.f, 0.f};
+  void* dyt_b[2] = {nullptr, nullptr};
   float* router_corr = nullptr;               // [router outputs] fp32: added to the scores for the choice
   // dense clamped gated unit: [gate | up] rows in one block (`up` names the second half)
   void* ff_gate = nullptr;
@@ -139,6 +150,10 @@ struct kge_engine {
   // layer-list ("hybrid") models: fp32 residual stream, their own activation arena and the recurrent-state pool
   std::vector<kge::HybridLayerW> hyb;
   float *res32 = nullptr, *gates32 = nullptr, *logits32 = nullptr, *state = nullptr, *mo32 = nullptr;
+  float final_alpha = 0.f;                   // Dynamic Tanh in the place of the final norm (weight final_w, shift final_b)
+  float* sgate32 = nullptr;                  // [tokens]: the shared expert's per-token gate where the router's logits come from a matrix product
+  float* dt32 = nullptr;                     // [tokens, channels]: step sizes of a selective scan
+  void* bcbuf = nullptr;                     // [tokens, dt_rank + 2 n_state]: a selective scan's [dt | B | C] rows
   float* y32 = nullptr;                      // [tokens, d]: a sublayer's sum when it has more sources than one combine pass takes
   void* embed_norm_w = nullptr;              // weight of the norm the embedding goes through (models that have one)
   void* bigram = nullptr;                    // second embedding table, picked by the token and the one before it

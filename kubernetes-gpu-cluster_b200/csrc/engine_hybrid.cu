@@ -2,9 +2,9 @@
 // linear recurrence, attention and a matrix memory side by side, attention alone with rotary positions, a soft cap
 // and sink logits, a WKV recurrence, attention through latents (every head's keys and values or the latents themselves in
 // the cache), windowed attention with kept first tokens beside gated linear attention, windowed attention over pooled
-// blocks, or a gated delta rule) and a feed-forward (dense or mixture of experts),
-// reading ONE norm of an fp32 residual stream, a norm each in sequence (optionally with a norm of each result as
-// well), or a norm each of a hyper-connected residual (several copies of the stream).  This file loads such a model (weights in the engine's storage
+// blocks, a gated delta rule, a selective scan, or windowed attention beside a state-space dual recurrence) and a feed-forward
+// (dense or mixture of experts), reading ONE norm of an fp32 residual stream, a norm (or Dynamic Tanh) each in sequence (optionally with a norm of
+// each result as well), or a norm each of a hyper-connected residual (several copies of the stream).  This file loads such a model (weights in the engine's storage
 // type, fused where one activation feeds several projections), sizes its arena, paged caches and recurrent-state pool,
 // and runs its step: the same flattened batch, block tables and slot mapping as every other model, plus a state slot
 // per request.  Nothing here depends on how a prompt was cut into steps: recurrences continue from the slot, attention
@@ -118,9 +118,11 @@ struct HB {
     return true;
   }
   // a matrix [sum(lead), K] (rows stacked), or random / constant values for a model without a checkpoint
-  void* mat(const std::vector<std::string>& names, const std::vector<int64_t>& lead, int64_t inner, float dummy_scale, float dummy_const = 0.f) {
+  // (pad: with zero rows behind them up to a multiple of that many)
+  void* mat(const std::vector<std::string>& names, const std::vector<int64_t>& lead, int64_t inner, float dummy_scale, float dummy_const = 0.f, int pad = 1) {
     int64_t rows = 0;
     for (auto l : lead) rows += l;
+    rows = (rows + pad - 1) / pad * pad;
     if (dummy()) {
       if (e->f32) { err = "random weights are made in bfloat16 only"; return nullptr; }
       void* p = dalloc(rows * inner, 2);
@@ -132,7 +134,31 @@ struct HB {
     }
     std::vector<float> v;
     if (!stack(names, lead, inner, &v)) return nullptr;
+    v.resize((size_t)(rows * inner), 0.f);
     return upload(v);
+  }
+  // a convolution's weights [channels, taps], transposed to [taps, channels]
+  void* conv_t(const std::string& name, int64_t C, int taps, float dummy_scale) {
+    if (dummy()) return mat({}, {C}, taps, dummy_scale);
+    std::vector<float> w, tr((size_t)C * taps);
+    if (!stack({name}, {C}, taps, &w)) return nullptr;
+    for (int64_t c = 0; c < C; ++c) for (int j = 0; j < taps; ++j) tr[(size_t)j * C + c] = w[(size_t)c * taps + j];
+    return upload(tr);
+  }
+  // Dynamic Tanh: weight, shift and scalar
+  bool dyt(const std::string& name, int d, void** w, void** shift, float* alpha) {
+    std::vector<float> a(1, 0.7f);
+    if (!dummy() && !stack({name + ".alpha"}, {1}, 1, &a)) return false;
+    *alpha = a[0];
+    return (*w = mat({name}, {d}, 1, 0.f, 1.f)) && (*shift = mat({name + ".b"}, {d}, 1, 0.f, 0.f));
+  }
+  // f(values) of a vector in fp32 (without a checkpoint: of a constant)
+  template <typename F>
+  float* mapped_f32(const std::string& name, int64_t n, float dummy_const, F f) {
+    std::vector<float> v((size_t)n, dummy_const);
+    if (!dummy() && !stack({name}, {n}, 1, &v)) return nullptr;
+    for (auto& x : v) x = f(x);
+    return upload_raw(v);
   }
 };
 
@@ -159,7 +185,8 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
   if (s.bigram_buckets > 0) HB_OK(e->bigram = b.mat({"bigram"}, {s.bigram_buckets + 1}, d, ws));
   HB_OK(e->lm_head = (bf16*)b.mat({"head"}, {s.vocab}, d, ws));
   const bool plain_norm_w = s.hyb_layernorm || s.streams > 0 || s.hyb_postnorm;      // the norm weight multiplies as it is (else it is applied as 1 + w)
-  HB_OK(e->final_w = (bf16*)b.mat({"final.norm"}, {d}, 1, 0.f, plain_norm_w ? 1.f : 0.f));
+  if (s.hyb_dyt) HB_OK(b.dyt("final.norm", d, (void**)&e->final_w, (void**)&e->final_b, &e->final_alpha));
+  else HB_OK(e->final_w = (bf16*)b.mat({"final.norm"}, {d}, 1, 0.f, plain_norm_w ? 1.f : 0.f));
   if (s.embed_norm) HB_OK(e->embed_norm_w = b.mat({"embed.norm"}, {d}, 1, 0.f, 1.f));
   e->hyb.resize(s.L);
   int64_t state_floats = s.bigram_buckets > 0 ? 4 : 0;      // the slot starts with the sequence's last token (a 16-byte piece)
@@ -169,7 +196,7 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
   int max_mo = 1;
   int max_proj = 1, max_mix = 1, max_ff = 1, max_gate = 1, max_u = 1, max_top = 0, max_eff = 1, max_E = 1;
   int max_hd = 0, max_qr = 0, max_kvr = 0, max_lkv = 0, max_lq = 0;      // WKV heads * dim; latent ranks, [k | v] and query widths
-  int max_mix2 = 0;
+  int max_mix2 = 0, max_bc = 0, max_dt = 0;
   for (int i = 0; i < s.L; ++i) {
     const HybridLayerSpec& h = s.hybrid[i];
     HybridLayerW& L = e->hyb[i];
@@ -189,9 +216,12 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
     if (s.hyb_noprenorm) {                      // the norms of the sublayers' results are the layer's only ones
       HB_OK(L.norm1b = b.mat({p + "norm1"}, {d}, 1, 0.f, 1.f));
       if (h.mlp != HybridLayerSpec::NONE) HB_OK(L.norm2b = b.mat({p + "norm2"}, {d}, 1, 0.f, 1.f));
+    } else if (s.hyb_dyt) {
+      HB_OK(b.dyt(p + "norm1", d, &L.norm1, &L.dyt_b[0], &L.dyt_alpha[0]));
+      if (h.mlp != HybridLayerSpec::NONE) HB_OK(b.dyt(p + "norm2", d, &L.norm2, &L.dyt_b[1], &L.dyt_alpha[1]));
     } else
     HB_OK(L.norm1 = b.mat({p + "norm1"}, {d}, 1, 0.f, norm_one));
-    if (!s.hyb_noprenorm && s.hyb_prenorm_pair && h.mlp != HybridLayerSpec::NONE) HB_OK(L.norm2 = b.mat({p + "norm2"}, {d}, 1, 0.f, norm_one));
+    if (!s.hyb_noprenorm && !s.hyb_dyt && s.hyb_prenorm_pair && h.mlp != HybridLayerSpec::NONE) HB_OK(L.norm2 = b.mat({p + "norm2"}, {d}, 1, 0.f, norm_one));
     if (s.hyb_postnorm && !s.hyb_noprenorm) {
       HB_OK(L.norm1b = b.mat({p + "norm1b"}, {d}, 1, 0.f, 1.f));
       if (h.mlp != HybridLayerSpec::NONE) HB_OK(L.norm2b = b.mat({p + "norm2b"}, {d}, 1, 0.f, 1.f));
@@ -392,6 +422,48 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
       state_floats += align_up64(short_conv_state_floats(C, h.conv), 4) + align_up64(delta_state_floats(H, h.dim, h.vdim), 4);      // both start 16-byte aligned
       max_proj = std::max(max_proj, L.proj.N); max_qkv32 = std::max(max_qkv32, (int)align_up64(C, 4)); max_gate = std::max(max_gate, na); max_mo = std::max(max_mo, nv);
       max_u = std::max(max_u, nv); max_mix = std::max(max_mix, nv);
+    } else if (h.mixer == HybridLayerSpec::MAMBA) {
+      const int C = h.width, N = h.n_state, R = h.decay_rank;
+      L.proj.N = 2 * C; L.proj.K = d;
+      HB_OK(L.proj.w = b.mat({mx + "in"}, {2 * C}, d, ws));
+      HB_OK(L.conv_w = b.conv_t(mx + "conv", C, h.conv, 0.5f));
+      HB_OK(L.conv_b = b.mat({mx + "conv.b"}, {C}, 1, 0.f, 0.f));
+      L.xproj.N = (int)align_up64(R + 2 * N, 8); L.xproj.K = C;      // whole 16-byte pieces per row
+      HB_OK(L.xproj.w = b.mat({mx + "x"}, {R + 2 * N}, C, ws, 0.f, 8));
+      L.dtproj.N = C; L.dtproj.K = R;
+      HB_OK(L.dtproj.w = b.mat({mx + "dt"}, {C}, R, ws));
+      HB_OK(L.dtproj.b = b.mat({mx + "dt.b"}, {C}, 1, 0.f, -3.f));
+      HB_OK(L.ssm_a = b.mapped_f32(mx + "A_log", (int64_t)C * N, 1.f, [](float v) { return -expf(v); }));
+      HB_OK(L.ssm_d = b.vec_f32(mx + "D", C, 1.f));
+      L.o.N = d; L.o.K = C;
+      HB_OK(L.o.w = b.mat({mx + "o"}, {d}, C, ws));
+      state_floats += align_up64(short_conv_state_floats(C, h.conv), 4) + align_up64(selective_state_floats(C, N), 4);
+      max_proj = std::max(max_proj, L.proj.N); max_u = std::max(max_u, C); max_mix = std::max(max_mix, C); max_bc = std::max(max_bc, L.xproj.N); max_dt = std::max(max_dt, C);
+    } else if (h.mixer == HybridLayerSpec::WINDOW_SSD) {
+      const int nq = h.heads * h.dim, nk = h.kv_heads * h.dim, nv = h.kv_heads * h.vdim, ng = h.heads * h.vdim, I = h.m_heads * h.m_vdim, C = I + 2 * h.ssd_groups * h.n_state;
+      const std::string a = mx + "left.", r = mx + "right.";
+      L.off_k = nq; L.off_v = nq + nk; L.off_mg = L.off_v + nv; L.off_z = L.off_mg + ng; L.off_x = L.off_z + I; L.off_dt = L.off_x + C;
+      L.proj.N = (int)align_up64(L.off_dt + h.m_heads, 8); L.proj.K = d;
+      HB_OK(L.proj.w = b.mat({a + "q", a + "k", a + "v", a + "g", r + "in"}, {nq, nk, nv, ng, I + C + h.m_heads}, d, ws, 0.f, 8));
+      if (h.rot_dims > 0) {
+        std::vector<double> fr((size_t)h.rot_dims / 2);
+        rotary_frequencies_banded(h.rot_dims, h.rot_base, h.rot_factor, h.rot_low, h.rot_high, h.rot_original, fr.data());
+        HB_OK(L.rot_freq = b.upload_raw(fr));
+      }
+      L.o.N = d; L.o.K = ng;
+      HB_OK(L.o.w = b.mat({a + "o"}, {d}, ng, ws));
+      L.o2.N = d; L.o2.K = I;
+      HB_OK(L.o2.w = b.mat({r + "o"}, {d}, I, ws));
+      HB_OK(L.conv_w = b.conv_t(r + "conv", C, h.conv, 0.5f));
+      HB_OK(L.conv_b = b.mat({r + "conv.b"}, {C}, 1, 0.f, 0.f));
+      HB_OK(L.ssm_dt_bias = b.vec_f32(r + "dt_bias", h.m_heads, -3.f));
+      HB_OK(L.ssm_a = b.mapped_f32(r + "A_log", h.m_heads, 1.f, [](float v) { return expf(v); }));
+      HB_OK(L.ssm_d = b.vec_f32(r + "D", h.m_heads, 1.f));
+      HB_OK(L.wkv_norm = b.mat({r + "norm"}, {I}, 1, 0.f, 1.f));
+      HB_OK(L.side_norm[0] = b.mat({a + "out"}, {d}, 1, 0.f, 1.f));
+      HB_OK(L.side_norm[1] = b.mat({r + "out"}, {d}, 1, 0.f, 1.f));
+      state_floats += align_up64(short_conv_state_floats(C, h.conv), 4) + align_up64(ssd_state_floats(h.m_heads, h.n_state, h.m_vdim), 4);
+      max_proj = std::max(max_proj, L.proj.N); max_u = std::max(max_u, (int)align_up64(C, 8)); max_mix = std::max(max_mix, ng); max_mix2 = std::max(max_mix2, I); max_mo = std::max(max_mo, I);
     } else if (h.mixer == HybridLayerSpec::LATENT) {
       const int nope = h.dim - h.rot_part, nq = h.heads * h.dim, nkv = h.kv_rank + h.rot_part, nv = h.heads * h.vdim;
       if (h.q_rank > 0) {
@@ -481,7 +553,13 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
       max_ff = std::max(max_ff, h.ff);
     } else if (h.mlp == HybridLayerSpec::MOE) {
       L.router.N = h.experts + h.identity; L.router.K = d;
-      HB_OK(L.router.w = b.mat({fp + "router"}, {L.router.N}, d, ws * 4));
+      // the row of the shared expert's per-token gate lies behind the router's: one product for both where many rows are routed
+      const bool joint = h.shared_ff > 0 && h.shared_gate && !h.router_bias;
+      if (joint) {
+        HB_OK(L.router.w = b.mat({fp + "router", fp + "shared.sg"}, {L.router.N, 1}, d, ws * 4));
+        L.s_sg = (uint8_t*)L.router.w + (int64_t)L.router.N * d * b.esz();
+        max_gate = std::max(max_gate, L.router.N + 1);
+      } else HB_OK(L.router.w = b.mat({fp + "router"}, {L.router.N}, d, ws * 4));
       if (h.router_correction) HB_OK(L.router_corr = b.vec_f32(fp + "correction", L.router.N, 0.f));
       if (h.router_bias) HB_OK(L.router_b = b.mat({fp + "router.b"}, {h.experts}, 1, 0.f, 0.f));
       // per expert [gate | up] rows in one block (what the fused gated GEMM reads), then all experts' down matrices
@@ -502,14 +580,14 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
         HB_OK(L.s_gate.w = b.mat({fp + "shared.gate", fp + "shared.up"}, {h.shared_ff, h.shared_ff}, d, ws));
         L.s_up.w = (uint8_t*)L.s_gate.w + (int64_t)h.shared_ff * d * b.esz();
         HB_OK(L.s_down.w = b.mat({fp + "shared.down"}, {d}, h.shared_ff, ws));
-        if (h.shared_gate) HB_OK(L.s_sg = b.mat({fp + "shared.sg"}, {1}, d, ws));
+        if (h.shared_gate && !joint) HB_OK(L.s_sg = b.mat({fp + "shared.sg"}, {1}, d, ws));
         max_ff = std::max(max_ff, h.shared_ff);
       }
       max_top = std::max(max_top, h.top); max_eff = std::max(max_eff, h.expert_ff); max_E = std::max(max_E, h.experts + h.identity); max_gate = std::max(max_gate, h.experts + h.identity);
     }
   }
 #undef HB_OK
-  e->slot_stride = std::max<int64_t>(s.hyb_noprenorm ? align_up64(state_floats, 4) : state_floats, 1);
+  e->slot_stride = std::max<int64_t>(s.hyb_noprenorm || s.hyb_dyt ? align_up64(state_floats, 4) : state_floats, 1);
 
   const int Tm = e->cfg.max_num_batched_tokens, Rm = e->cfg.max_num_seqs, es = b.esz();
   // 16-bit logits rows: straight out of the tensor-core GEMM when its shapes allow (then the row stride is the
@@ -524,6 +602,11 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
     e->mixes = aalloc((int64_t)5 * Tm * d, es); e->rkvg = aalloc((int64_t)4 * Tm * max_hd, es);
     if (!e->mixes || !e->rkvg) return fail(b.err);
   }
+  if (max_bc > 0) {
+    e->bcbuf = aalloc((int64_t)Tm * max_bc, es); e->dt32 = (float*)aalloc((int64_t)Tm * max_dt, 4);
+    if (!e->bcbuf || !e->dt32) return fail(b.err);
+  }
+  if (max_top > 0) { e->sgate32 = (float*)aalloc(Tm, 4); if (!e->sgate32) return fail(b.err); }
   if (max_qkv32 > 0) { e->qkv32 = (float*)aalloc((int64_t)Tm * max_qkv32, 4); if (!e->qkv32) return fail(b.err); }
   if (max_abs > 0) {
     // rows of a step that attend in the latent space: all of them, or (prompt pieces on the expanded path) one per request
@@ -673,7 +756,7 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
   return 0;
 }
 
-enum { C_GEMM_S = 0, C_GEMM_L = 1, C_ATT_DEC = 2, C_ATT_GEN = 3, C_NORM = 4, C_KVW = 5, C_ACT = 6, C_EMBED = 7, C_SAMPLE = 8, C_RGLRU = 10, C_MLSTM = 11, C_MOE = 12 };
+enum { C_GEMM_S = 0, C_GEMM_L = 1, C_ATT_DEC = 2, C_ATT_GEN = 3, C_NORM = 4, C_KVW = 5, C_ACT = 6, C_EMBED = 7, C_SAMPLE = 8, C_RGLRU = 10, C_MLSTM = 11, C_MOE = 12, C_SSD = 13, C_STEP = 14 };
 
 // KGE_TRACE_LAUNCHES=1 (diagnostics): synchronise after every launch of a step and name it on stderr
 static const bool g_trace_launches = getenv("KGE_TRACE_LAUNCHES") != nullptr;
@@ -695,9 +778,9 @@ static const bool g_trace_launches = getenv("KGE_TRACE_LAUNCHES") != nullptr;
 // shape the tensor-core GEMM takes (16-byte rows, packed operands) there; the rest, and float32 engines, run the
 // shape-agnostic kernel.
 static int dense(kge_engine* e, void* y, int ldy, const void* x, int ldx, const HybMat& m, int T, int act, bool out_f32 = false) {
-  if (!e->f32 && !out_f32 && m.K % 8 == 0 && ldx == m.K && ldy == m.N && (act == ACT_NONE || act == ACT_GELU_ERF) &&
+  if (!e->f32 && !out_f32 && m.K % 8 == 0 && ldx == m.K && ldy == m.N && (act == ACT_NONE || act == ACT_GELU_ERF || act == ACT_RELU2) &&
       ((uintptr_t)x & 15) == 0 && ((uintptr_t)m.w & 15) == 0)
-    return kge_gemm_bf16(y, x, m.w, m.b, T, m.N, m.K, act == ACT_GELU_ERF ? 3 : 0, nullptr, 0, e->stream);
+    return kge_gemm_bf16(y, x, m.w, m.b, T, m.N, m.K, act == ACT_GELU_ERF ? 3 : act == ACT_RELU2 ? 4 : 0, nullptr, 0, e->stream);
   LinearArgs a;
   a.x = x; a.ldx = ldx; a.w = m.w; a.bias = m.b; a.y = y; a.ldy = ldy; a.T = T; a.N = m.N; a.K = m.K; a.act = act;
   a.elt = e->f32 ? KGE_ELT_F32 : KGE_ELT_BF16; a.out_f32 = out_f32 || e->f32;
@@ -723,8 +806,9 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
   // launch buys nothing there, and hundreds of long-running CTAs of one kernel waiting on the previous one would only
   // hold shared memory.  Decode steps keep programmatic dependent launch (and run as CUDA graphs).
   struct PdlOff { bool on; explicit PdlOff(bool o) : on(o) { if (on) pdl_suspend(true); } ~PdlOff() { if (on) pdl_suspend(false); } } pdl_off(!decode_only);
-  // the model's norm of residual rows: RMS with the weight applied as 1 + w, or the weight-only layer norm
+  // the model's norm of residual rows: RMS with the weight applied as 1 + w, the weight-only layer norm, or Dynamic Tanh
   auto layer_norm = [&](void* y, const int32_t* rows, const void* w, int R, float out_scale) -> int {
+    if (s.hyb_dyt) return dyt_f32in(y, e->res32, rows, e->final_alpha, w, e->final_b, R, d, elt, st);      // only the final one runs by itself
     if (s.hyb_postnorm) return group_rmsnorm_f32in(y, e->res32, rows, w, R, d, s.norm_groups, s.eps, out_scale, elt, st);
     return s.hyb_layernorm ? layernorm_f32in(y, e->res32, rows, w, R, d, s.eps, out_scale, elt, st)
                            : rmsnorm_f32in(y, e->res32, rows, w, R, d, s.eps, 1.f, out_scale, elt, st);
@@ -746,8 +830,14 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
     ba.state = e->state; ba.slot_stride = e->slot_stride; ba.slots = m.sslot; ba.qsl = m.qsl; ba.positions = m.pos; ba.token_req = m.treq;
     ba.B = B; ba.T = T; ba.d = d; ba.inline_save = decode_only; ba.elt = elt;
     HFWD(C_EMBED, Td * (3 * es + 4), 0, embed_bigram(ba, st));
+  } else if (s.hyb_dyt) {
+    // the scaled embedding row and the first sublayer's input
+    DytCombineArgs da;
+    da.res = e->res32; da.ids = m.ids; da.table = e->embed; da.table_scale = s.embed_scale; da.T = T; da.d = d; da.elt = elt;
+    da.next_alpha = e->hyb[0].dyt_alpha[0]; da.next_w = e->hyb[0].norm1; da.next_b = e->hyb[0].dyt_b[0]; da.next_y = e->hx;
+    HFWD(C_EMBED, Td * (2 * es + 4), 0, dyt_combine(da, st));
   } else HFWD(C_EMBED, Td * (es + 4), 0, embed_f32(e->res32, m.ids, e->embed, T, d, elt, st));
-  bool hx_ready = s.hyb_noprenorm;      // the previous layer's last write of the streams already formed this layer's normed input
+  bool hx_ready = s.hyb_noprenorm || s.hyb_dyt;      // the previous layer's last write of the streams already formed this layer's normed input
   for (int i = 0; i < s.L; ++i) {
     const HybridLayerSpec& h = s.hybrid[i];
     const HybridLayerW& L = e->hyb[i];
@@ -788,6 +878,22 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
         else if (i + 1 < s.L) { pa.next_w = e->hyb[i + 1].norm1; pa.next_y = e->hx; hx_ready = true; }
         cb = CombineArgs(); inner_w[0] = inner_w[1] = nullptr;
         return postnorm_residual(pa, st);
+      }
+      if (s.hyb_dyt) {
+        DytCombineArgs da;
+        da.res = e->res32; da.nsrc = cb.n; da.src_scale = cb.n ? cb.scale[0] : 1.f; da.T = T; da.d = d; da.eps = s.eps; da.elt = elt;
+        for (int q = 0; q < cb.n && q < 2; ++q) { da.src[q] = cb.src[q]; da.ld[q] = cb.ld[q]; da.inner_w[q] = inner_w[q]; da.rscale[q] = cb.rscale[q]; }
+        da.pair_src = pair_src; da.pair_row = pair_src ? e->moe_prow : nullptr; da.pair_w = e->moe_cw; da.top = h.top;
+        pair_src = nullptr;
+        const bool mixer_done = sub == 0 && h.mlp != HybridLayerSpec::NONE;
+        const HybridLayerW* nx = mixer_done ? &L : i + 1 < s.L ? &e->hyb[i + 1] : nullptr;
+        if (nx) {
+          const int q = mixer_done ? 1 : 0;
+          da.next_alpha = nx->dyt_alpha[q]; da.next_w = q ? nx->norm2 : nx->norm1; da.next_b = nx->dyt_b[q]; da.next_y = e->hx;
+          if (!mixer_done) hx_ready = true;
+        }
+        cb = CombineArgs(); inner_w[0] = inner_w[1] = nullptr;
+        return dyt_combine(da, st);
       }
       if (!hyper) return flush_more();
       StreamCombineArgs sc;
@@ -1066,6 +1172,69 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
       HFWD(C_MLSTM, (double)T * nv * (4 + 2 * es), 0, wkv_norm_gate(wa, st));
       DENSE(e->obuf1, d, e->mixbuf, nv, L.o, T, ACT_NONE);
       add_src(e->obuf1, d, 1.f);
+    } else if (h.mixer == HybridLayerSpec::MAMBA) {
+      const int C = h.width, N = h.n_state, R = h.decay_rank, ldp = L.proj.N, ldbc = L.xproj.N;
+      DENSE(e->pbuf, ldp, e->hx, d, L.proj, T, ACT_NONE);                // [x | z]
+      ConvHeadsArgs ca;      // convolution with its bias, silu
+      ca.x = e->pbuf; ca.ldx = ldp; ca.y = e->ubuf; ca.ldy = C; ca.out_elt = true; ca.w = L.conv_w; ca.bias = L.conv_b; ca.C = C; ca.taps = h.conv;
+      ca.state = e->state + L.state_off; ca.slot_stride = e->slot_stride; ca.slots = m.sslot; ca.qsl = m.qsl; ca.positions = m.pos; ca.token_req = m.treq;
+      ca.B = B; ca.T = T; ca.inline_save = decode_only; ca.elt = elt;
+      HFWD(C_RGLRU, (double)T * C * 2 * es, 2.0 * T * C * h.conv, short_conv_silu_heads(ca, st));
+      if (!decode_only && h.conv > 1) ++e->launches;
+      DENSE(e->bcbuf, ldbc, e->ubuf, C, L.xproj, T, ACT_NONE);           // [dt | B | C]
+      LinearArgs dp;         // the steps: second half of their low-rank pair, bias and softplus in the epilogue, fp32
+      dp.x = e->bcbuf; dp.ldx = ldbc; dp.w = L.dtproj.w; dp.bias = L.dtproj.b; dp.y = e->dt32; dp.ldy = C; dp.T = T; dp.N = C; dp.K = R; dp.act = ACT_SOFTPLUS; dp.elt = elt; dp.out_f32 = true;
+      HFWD(C_STEP, es * ((double)R * C + (double)T * R) + 4.0 * T * C, 2.0 * T * (double)C * R, linear_any(dp, st));
+      SelectiveScanArgs sa;
+      sa.x = e->ubuf; sa.ldx = C; sa.z = at(e->pbuf, C); sa.ldz = ldp; sa.b = at(e->bcbuf, R); sa.c = at(e->bcbuf, R + N); sa.ldbc = ldbc; sa.dt = e->dt32; sa.lddt = C;
+      sa.A = L.ssm_a; sa.D = L.ssm_d; sa.out = e->mixbuf; sa.ldo = C; sa.state = e->state + L.state_off + align_up64(short_conv_state_floats(C, h.conv), 4);
+      sa.slot_stride = e->slot_stride; sa.slots = m.sslot; sa.qsl = m.qsl; sa.positions = m.pos; sa.B = B; sa.T = T; sa.C = C; sa.N = N; sa.elt = elt;
+      HFWD(C_MLSTM, 2.0 * B * selective_state_floats(C, N) * 4 + (double)T * (C * (3 * es + 4) + 2 * N * es), 6.0 * T * C * (double)N, selective_scan(sa, st));
+      DENSE(e->obuf1, d, e->mixbuf, C, L.o, T, ACT_NONE);
+      add_src(e->obuf1, d, 1.f);
+    } else if (h.mixer == HybridLayerSpec::WINDOW_SSD) {
+      const int nq = h.heads * h.dim, nk = h.kv_heads * h.dim, nv = h.kv_heads * h.vdim, ka = h.heads * h.vdim, ldp = L.proj.N;
+      const int I = h.m_heads * h.m_vdim, GN = h.ssd_groups * h.n_state, C = I + 2 * GN, ldc = (int)align_up64(C, 8);
+      DENSE(e->pbuf, ldp, e->hx, d, L.proj, T, ACT_NONE);                // every projection of both sides: [q | k | v | g | z | x | B | C | dt]
+      HeadRotaryArgs ro;     // rotation in halves, K cache <- turned keys, V cache <- values
+      ro.q = e->pbuf; ro.ldq = ldp; ro.k = at(e->pbuf, L.off_k); ro.ldk = ldp; ro.v = at(e->pbuf, L.off_v); ro.ldv = ldp; ro.eps = s.eps;
+      ro.freq = L.rot_freq; ro.rot_dims = h.rot_dims; ro.positions = m.pos; ro.slots = m.slots;
+      ro.k_cache = L.kc; ro.v_cache = L.vc; ro.T = T; ro.H = h.heads; ro.G = h.kv_heads; ro.dim = h.dim; ro.vdim = h.vdim; ro.block_size = bs; ro.elt = elt;
+      HFWD(C_KVW, (double)T * (2.0 * nq + 2.0 * nk + 2.0 * nv) * es, 0, head_norm_rotary_kvwrite(ro, st));
+      AttnBiasArgs aa;
+      aa.q = e->pbuf; aa.ldq = ldp; aa.out = e->mixbuf; aa.ldo = ka; aa.k_cache = L.kc; aa.v_cache = L.vc;
+      aa.block_table = m.btab; aa.max_blocks = max_blocks; aa.seq_lens = m.seq_lens; aa.qsl = m.qsl; aa.positions = m.pos; aa.token_req = m.treq;
+      aa.B = B; aa.T = T; aa.H = h.heads; aa.G = h.kv_heads; aa.dim = h.dim; aa.vdim = h.vdim; aa.block_size = bs; aa.window = h.window; aa.scale = h.scale; aa.elt = elt;
+      for (int r = 0; r < B; ++r) aa.max_q = std::max(aa.max_q, hm.qsl[r + 1] - hm.qsl[r]);
+      while (aa.num_decode < B && hm.qsl[aa.num_decode + 1] - hm.qsl[aa.num_decode] == 1) ++aa.num_decode;
+      double keys = 0;                                   // visible keys over all rows
+      for (int t = 0; t < T; ++t) keys += std::min(hm.pos[t] + 1, h.window);
+      // steps with prompt pieces, 64- / 128-wide heads, bfloat16: the tcgen05 kernel; decode steps and everything else: the mma.sync / per-row kernels
+      const bool tc = !e->f32 && !decode_only && ldp % 8 == 0 && ((uintptr_t)e->pbuf & 15) == 0 && paged_attn_window_tc_ok(h.heads, h.kv_heads, h.dim, h.vdim, bs, 0, 0);
+      HFWD(decode_only ? C_ATT_DEC : C_ATT_GEN, (decode_only ? keys : (double)T) * h.kv_heads * (h.dim + h.vdim) * es + (double)T * h.heads * (h.dim + h.vdim) * es,
+           2.0 * keys * h.heads * (h.dim + h.vdim),
+           tc ? paged_attn_window_tc(e->mixbuf, e->pbuf, ldp, L.kc, L.vc, nullptr, nullptr, m.btab, max_blocks, m.seq_lens, m.qsl, B, aa.max_q, h.heads, h.kv_heads, h.dim, bs,
+                                     h.scale, h.window, 0, 0, 0, nullptr, st)
+              : attn_bias_chunk(aa, st));
+      HFWD(C_ACT, (double)T * ka * 3 * es, 0, sigmoid_gate_mul(e->mixbuf, ka, at(e->pbuf, L.off_mg), ldp, T, ka, elt, st));
+      DENSE(e->obuf1, d, e->mixbuf, ka, L.o, T, ACT_NONE);
+      ConvHeadsArgs ca;      // x, B and C through their convolution (with a bias) and a silu
+      ca.x = at(e->pbuf, L.off_x); ca.ldx = ldp; ca.y = e->ubuf; ca.ldy = ldc; ca.out_elt = true; ca.w = L.conv_w; ca.bias = L.conv_b; ca.C = C; ca.taps = h.conv;
+      ca.state = e->state + L.state_off; ca.slot_stride = e->slot_stride; ca.slots = m.sslot; ca.qsl = m.qsl; ca.positions = m.pos; ca.token_req = m.treq;
+      ca.B = B; ca.T = T; ca.inline_save = decode_only; ca.elt = elt;
+      HFWD(C_RGLRU, (double)T * C * 2 * es, 2.0 * T * C * h.conv, short_conv_silu_heads(ca, st));
+      if (!decode_only && h.conv > 1) ++e->launches;
+      SsdArgs sa;
+      sa.x = e->ubuf; sa.b = at(e->ubuf, I); sa.c = at(e->ubuf, I + GN); sa.ld = ldc; sa.dt_pre = at(e->pbuf, L.off_dt); sa.lddt = ldp;
+      sa.dt_bias = L.ssm_dt_bias; sa.a_coef = L.ssm_a; sa.D = L.ssm_d; sa.o32 = e->mo32; sa.state = e->state + L.state_off + align_up64(short_conv_state_floats(C, h.conv), 4);
+      sa.slot_stride = e->slot_stride; sa.slots = m.sslot; sa.qsl = m.qsl; sa.positions = m.pos;
+      sa.B = B; sa.T = T; sa.H = h.m_heads; sa.G = h.ssd_groups; sa.N = h.n_state; sa.P = h.m_vdim; sa.elt = elt;
+      HFWD(C_SSD, 2.0 * B * ssd_state_floats(h.m_heads, h.n_state, h.m_vdim) * 4 + (double)T * (C * es + 4.0 * I + h.m_heads * es), 5.0 * T * I * (double)h.n_state, ssd_scan(sa, st));
+      HFWD(C_SSD, (double)T * I * (4 + 2 * es), 0, gated_group_rmsnorm(e->mixbuf2, I, e->mo32, at(e->pbuf, L.off_z), ldp, L.wkv_norm, T, I, h.out_norm_groups, s.eps, elt, st));
+      DENSE(e->obuf2, d, e->mixbuf2, I, L.o2, T, ACT_NONE);
+      // half the sum of the two sides, each RMS-normed over the width with its own weight
+      add_src(e->obuf1, d, 0.5f); add_src(e->obuf2, d, 0.5f);
+      inner_w[0] = L.side_norm[0]; inner_w[1] = L.side_norm[1];
     } else if (h.mixer == HybridLayerSpec::LATENT) {
       const int H = h.heads, nope = h.dim - h.rot_part, nq = H * h.dim, nv = H * h.vdim, ldp = L.proj.N, ldkv = L.lat_ukv.N;
       DENSE(e->pbuf, ldp, e->hx, d, L.proj, T, ACT_NONE);      // [dq | dkv] or [q | dkv | g] of the normed row
@@ -1139,9 +1308,9 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
     }
     if (s.hyb_prenorm_pair && h.mlp != HybridLayerSpec::NONE) {
       // the feed-forward reads a norm of the stream that already holds the mixer's output
-      { const double nsrc = cb.n + (s.hyb_postnorm ? 1 : 0); HFWD(C_ACT, Td * (8.0 * S + nsrc * es), 0, flush()); }      // post-norm models also write the next normed row
+      { const double nsrc = cb.n + (s.hyb_postnorm || s.hyb_dyt ? 1 : 0); HFWD(C_ACT, Td * (8.0 * S + nsrc * es), 0, flush()); }      // post-norm models also write the next normed row
       sub = 1;
-      if (!hyper && !s.hyb_postnorm) HFWD(C_NORM, Td * (4 + es), 0, layer_norm(e->hx, nullptr, L.norm2, T, 1.f));
+      if (!hyper && !s.hyb_postnorm && !s.hyb_dyt) HFWD(C_NORM, Td * (4 + es), 0, layer_norm(e->hx, nullptr, L.norm2, T, 1.f));
     }
     if (h.mlp == HybridLayerSpec::DENSE && h.ff_silu_bias) {
       // silu(gate h + b) * (up h + b): one product over [gate | up] with the biases, the pair formed from its rows
@@ -1172,20 +1341,21 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
       DENSE(e->obuf2, d, e->ffbuf, f, L.down, T, ACT_NONE);
       add_src(e->obuf2, d, 1.f);
     } else if (h.mlp == HybridLayerSpec::DENSE) {
-      DENSE(e->ffbuf, h.ff, e->hx, d, L.up, T, ACT_GELU_ERF);
+      DENSE(e->ffbuf, h.ff, e->hx, d, L.up, T, h.ff_relu2 ? ACT_RELU2 : ACT_GELU_ERF);
       DENSE(e->obuf2, d, e->ffbuf, h.ff, L.down, T, ACT_NONE);
       add_src(e->obuf2, d, 1.f);
     } else if (h.mlp == HybridLayerSpec::MOE) {
       MoeRouteArgs ra;
       ra.h = e->hx; ra.ldh = d; ra.w_router = L.router.w; ra.b_router = L.router_b; ra.T = T; ra.d = d; ra.E = h.experts + h.identity; ra.top = h.top;
       ra.correction = L.router_corr; ra.groups = h.router_groups; ra.groups_keep = h.groups_keep; ra.identity = h.identity; ra.pair_row = e->moe_prow;
-      const bool by_pair = s.hyb_postnorm;      // the pass that norms the result gathers the experts' rows itself: they stay in routed order
+      const bool by_pair = s.hyb_postnorm || s.hyb_dyt;      // the pass that sums the result gathers the experts' rows itself: they stay in routed order
       const bool w_out = h.route != HybridLayerSpec::ROUTE_SIGMOID_IN;      // the routing weight multiplies the expert's output (in the fp32 sum below)
       const bool clamped = h.glu == HybridLayerSpec::GLU_CLAMPED;
       const bool ungated = h.glu == HybridLayerSpec::GLU_NONE_RELU2;      // one front matrix per expert, relu(.)^2
-      ra.score_fn = h.route == HybridLayerSpec::ROUTE_SOFTMAX_TOP ? 2 : h.route == HybridLayerSpec::ROUTE_SOFTMAX_ALL ? 1 : 0; ra.renorm = false;
+      ra.score_fn = h.route == HybridLayerSpec::ROUTE_SOFTMAX_TOP ? 2 : h.route == HybridLayerSpec::ROUTE_SOFTMAX_ALL ? 1 : 0; ra.renorm = h.route == HybridLayerSpec::ROUTE_SIGMOID_NORM;
+      ra.renorm_eps = 1e-20f; ra.group_best = h.group_best;
       ra.weight_scale = h.router_scale;
-      if (L.s_sg) { ra.w_extra = L.s_sg; ra.extra_sigmoid = e->gates32; }      // the shared expert's per-token gate rides along, kept in fp32
+      if (L.s_sg) { ra.w_extra = L.s_sg; ra.extra_sigmoid = e->sgate32; }      // the shared expert's per-token gate rides along, kept in fp32
       ra.group_off = e->moe_goff; ra.perm_token = e->moe_ptok; ra.perm_weight = e->moe_pw; ra.perm_dest = e->moe_pdest;
       ra.choice_expert = e->moe_cexp; ra.choice_weight = e->moe_cw; ra.elt = elt;
       const int np = T * h.top;
@@ -1193,10 +1363,11 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
       const int np_pad = (np / 256 + h.experts + 1) * 256;
       const bool grouped = !e->f32 && !decode_only && np >= 512 && h.expert_ff % 64 == 0 && d % 8 == 0 && e->moe_xperm && np_pad <= e->moe_rows_padded;
       if (grouped) { ra.pad = 256; ra.rows_padded = np_pad; ra.tile_group = e->moe_tile_group; }
-      if (T > 256 && !L.s_sg && ra.E <= 512) {
+      const bool joint = L.s_sg && L.s_sg == (uint8_t*)L.router.w + (int64_t)ra.E * d * (int)es;
+      if (T > 256 && (!L.s_sg || joint) && ra.E <= 512) {
         // many rows: the router's logits as one matrix product with fp32 sums
         LinearArgs rl;
-        rl.x = e->hx; rl.ldx = d; rl.w = L.router.w; rl.bias = L.router_b; rl.y = e->gates32; rl.ldy = ra.E; rl.T = T; rl.N = ra.E; rl.K = d; rl.elt = elt; rl.out_f32 = true;
+        rl.x = e->hx; rl.ldx = d; rl.w = L.router.w; rl.bias = L.router_b; rl.y = e->gates32; rl.N = rl.ldy = ra.ld_logits = ra.E + (joint ? 1 : 0); rl.T = T; rl.K = d; rl.elt = elt; rl.out_f32 = true;
         HFWD(C_MOE, Td * es + (double)ra.E * d * es, 2.0 * Td * ra.E, linear_any(rl, st));
         ra.logits = e->gates32;
         HFWD(C_MOE, 4.0 * T * ra.E, 0, moe_route(ra, st));
@@ -1252,10 +1423,10 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
         if (cb.n == 4) HFWD(C_ACT, Td * (8 + 4 * es), 0, flush_more());
         add_src(at(e->moe_out, (int64_t)k * d), h.top * d, 1.f, w_out ? e->moe_cw + k : nullptr, h.top);
       }
-      if (h.shared_ff > 0) { if (cb.n == 4) HFWD(C_ACT, Td * (8 + 4 * es), 0, flush_more()); add_src(e->obuf2, d, 1.f, L.s_sg ? e->gates32 : nullptr, 1); }
+      if (h.shared_ff > 0) { if (cb.n == 4) HFWD(C_ACT, Td * (8 + 4 * es), 0, flush_more()); add_src(e->obuf2, d, 1.f, L.s_sg ? e->sgate32 : nullptr, 1); }
     }
     if (cb.n > 0 || pair_src || s.hyb_noprenorm == false) {      // post-norm models also write the next normed row
-      const double nsrc = cb.n + (pair_src ? h.top : 0) + (s.hyb_postnorm ? 1 : 0); HFWD(C_ACT, Td * (8.0 * S + nsrc * es), 0, flush());
+      const double nsrc = cb.n + (pair_src ? h.top : 0) + (s.hyb_postnorm || s.hyb_dyt ? 1 : 0); HFWD(C_ACT, Td * (8.0 * S + nsrc * es), 0, flush());
     }
     if (e->layer_dump_host && (int64_t)(i + 1) * T * d <= e->layer_dump_cap) {
       if (hyper) { if (int rc = stream_read(nullptr, nullptr, nullptr, nullptr, T, 1.f, e->y32)) return rc; }      // the sum of the streams

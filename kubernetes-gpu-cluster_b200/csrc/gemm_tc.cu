@@ -1284,7 +1284,7 @@ extern "C" int KGE_GEMM_NAME(void* y, const void* x, const void* w, const void* 
   KGE_REQUIRE(y && x && w, "kge_gemm_bf16: null pointer");
   KGE_REQUIRE(T >= 0 && N > 0 && K > 0 && K % 8 == 0, "kge_gemm_bf16: K=%d must be a positive multiple of 8", K);
   KGE_REQUIRE(((uintptr_t)x & 15) == 0 && ((uintptr_t)w & 15) == 0, "kge_gemm_bf16: x and w must be 16-byte aligned");
-  KGE_REQUIRE(act == 0 || act == 1 || act == 3, "kge_gemm_bf16: act=%d unsupported (0 none, 1 relu, 3 gelu)", act);
+  KGE_REQUIRE(act == 0 || act == 1 || act == 3 || act == 4, "kge_gemm_bf16: act=%d unsupported (0 none, 1 relu, 3 gelu, 4 squared relu)", act);
   if (T == 0) return 0;
   bool use_ws = workspace && tunable(TUN_GEMM_WS);          // stream-K through the caller's scratch, if it is large enough
   if (use_ws) {

@@ -1,7 +1,8 @@
 // RMS norms in groups for layer-list models that norm a sublayer's input AND its result: the row is cut into `groups`
 // equal consecutive parts, each divided by its own root mean square.  One block per row; the row stays in shared memory
 // (fp32) between the statistics and the write, so the residual stream is read once and written once per sublayer, and the
-// pass that adds a sublayer's result also forms the next sublayer's normed input.  Every sum of a row is formed in a
+// pass that adds a sublayer's result also forms the next sublayer's normed input; also a recurrence's output behind its gate.
+// Every sum of a row is formed in a
 // fixed order that depends on the row's width only, never on what else is in the launch.
 #include "common.cuh"
 #include "elt_access.cuh"
@@ -138,6 +139,39 @@ __global__ void __launch_bounds__(GN_THREADS) postnorm_residual_kernel(PostNormA
   }
 }
 
+// a recurrence's read-out times silu(gate), then the group norm and its weight
+template <typename E, bool VEC>
+__global__ void __launch_bounds__(GN_THREADS) gated_group_rmsnorm_kernel(E* out, int ldo, const float* y, const E* z, int ldz, const E* w, int d, int groups, float eps) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ __align__(16) float gn_sm[];
+  __shared__ float inv[GN_MAX_GROUPS], red[33];
+  constexpr int W = VEC ? 4 : 1;
+  const int t = blockIdx.x, gs = d / groups;
+  float ss = 0.f;
+  for (int c = threadIdx.x * W; c < d; c += GN_THREADS * W) {
+    float v[4], g[4];
+    if (VEC) { ld4(y + (int64_t)t * d + c, v); ld4(z + (int64_t)t * ldz + c, g); } else { v[0] = y[(int64_t)t * d + c]; g[0] = ldf(z + (int64_t)t * ldz + c); }
+#pragma unroll
+    for (int k = 0; k < W; ++k) { v[k] *= g[k] / (1.f + expf(-g[k])); gn_sm[c + k] = v[k]; ss = fmaf(v[k], v[k], ss); }
+  }
+  if (groups == 1) {                   // the sum is in the threads' registers already
+    ss = block_sum(ss, red);
+    if (threadIdx.x == 0) inv[0] = 1.f / sqrtf(ss / (float)d + eps);
+  } else {
+    __syncthreads();
+    group_inv_rms(gn_sm, d, groups, eps, inv);
+  }
+  __syncthreads();
+  for (int c = threadIdx.x * W; c < d; c += GN_THREADS * W) {
+    float o[4], wv[4];
+    if (VEC) ld4(w + c, wv); else wv[0] = ldf(w + c);
+#pragma unroll
+    for (int k = 0; k < W; ++k) o[k] = gn_sm[c + k] * inv[(c + k) / gs] * wv[k];
+    if (VEC) st4(out + (int64_t)t * ldo + c, o); else stf(out + (int64_t)t * ldo + c, o[0]);
+  }
+}
+
 template <typename E>
 __global__ void __launch_bounds__(256) silu_mul_halves_kernel(E* y, const E* gu, int64_t n, int f) {
   pdl_launch_dependents();
@@ -170,6 +204,22 @@ int group_rmsnorm_f32in(void* y, const float* x, const int32_t* rows, const void
     KGE_CUDA_OK(launch_pdl(group_rmsnorm_kernel<__nv_bfloat16>, dim3(R), dim3(GN_THREADS), smem, st, (__nv_bfloat16*)y, x, rows, (const __nv_bfloat16*)w, d, groups, eps, out_scale));
   }
   return 0;
+}
+
+template <typename E>
+static int gated_launch(E* out, int ldo, const float* y, const E* z, int ldz, const E* w, int T, int n, int groups, float eps, cudaStream_t st) {
+  const size_t smem = (size_t)n * 4;
+  const bool vec = n % 4 == 0 && ldo % 4 == 0 && ldz % 4 == 0 && (((uintptr_t)out | (uintptr_t)y | (uintptr_t)z | (uintptr_t)w) & 15) == 0;
+  auto kern = vec ? gated_group_rmsnorm_kernel<E, true> : gated_group_rmsnorm_kernel<E, false>;
+  if (int rc = opt_in_smem(kern, smem)) return rc;
+  KGE_CUDA_OK(launch_pdl(kern, dim3(T), dim3(GN_THREADS), smem, st, out, ldo, y, z, ldz, w, n, groups, eps));
+  return 0;
+}
+int gated_group_rmsnorm(void* out, int ldo, const float* y, const void* z, int ldz, const void* w, int T, int n, int groups, float eps, int elt, cudaStream_t st) {
+  if (T <= 0) return 0;
+  KGE_REQUIRE(groups >= 1 && groups <= GN_MAX_GROUPS && n % groups == 0 && n <= 51200, "gated_group_rmsnorm: %d groups of a row of %d", groups, n);
+  return elt == KGE_ELT_F32 ? gated_launch((float*)out, ldo, y, (const float*)z, ldz, (const float*)w, T, n, groups, eps, st)
+                            : gated_launch((__nv_bfloat16*)out, ldo, y, (const __nv_bfloat16*)z, ldz, (const __nv_bfloat16*)w, T, n, groups, eps, st);
 }
 
 int postnorm_residual(const PostNormArgs& a, cudaStream_t st) {

@@ -4,8 +4,8 @@
 // mixture-of-experts router, the hyper-connected residual (several streams), the WKV recurrence (also run as gated linear
 // attention), the row-wise parts of attention through latents, sliding windows with kept first tokens or pooled blocks,
 // short causal convolutions with a state, per-head norms with rotary positions in halves and rotated values, and grouped
-// RMS norms before and after a sublayer, a bigram embedding, attention over cached latents, and a gated delta rule.  Every mechanism takes its sizes and constants
-// as arguments.  `elt` names the storage type of activations and weights: KGE_ELT_BF16 or KGE_ELT_F32; what the
+// RMS norms before and after a sublayer, a bigram embedding, attention over cached latents, a gated delta rule, Dynamic Tanh, a
+// selective scan and a state-space dual recurrence.  Every mechanism takes its sizes and constants as arguments.  `elt` names the storage type of activations and weights: KGE_ELT_BF16 or KGE_ELT_F32; what the
 // mechanisms compute in 32 bits (softmax, norms, routers, residual sums, recurrent state and everything that enters a
 // recurrence besides projections and short convolutions) is 32-bit in both.
 #pragma once
@@ -21,7 +21,7 @@
 namespace kge {
 
 enum { KGE_ELT_BF16 = 0, KGE_ELT_F32 = 1 };
-enum { ACT_NONE = 0, ACT_GELU_ERF = 1, ACT_GELU_TANH = 2, ACT_SILU = 3, ACT_SIGMOID = 4, ACT_TANH = 5, ACT_RELU2 = 6, ACT_EXP_DECAY = 7 };
+enum { ACT_NONE = 0, ACT_GELU_ERF = 1, ACT_GELU_TANH = 2, ACT_SILU = 3, ACT_SIGMOID = 4, ACT_TANH = 5, ACT_RELU2 = 6, ACT_EXP_DECAY = 7, ACT_SOFTPLUS = 8 };
 
 inline size_t elt_size(int elt) { return elt == KGE_ELT_F32 ? 4 : 2; }
 
@@ -50,6 +50,22 @@ struct LinearArgs {
 };
 enum { GLU_SILU_MUL = 0, GLU_CLAMPED_SIGMOID = 1 };
 int linear_any(const LinearArgs& a, cudaStream_t st);
+
+// Dynamic Tanh in the place of a norm: y[r, :] = tanh(alpha * x[rows ? rows[r] : r, :]) * w + b, x fp32, y / w / b in elt
+int dyt_f32in(void* y, const float* x, const int32_t* rows, float alpha, const void* w, const void* b, int R, int d, int elt, cudaStream_t st);
+// A sublayer's result joins the residual stream, and the next sublayer's input (Dynamic Tanh of the new row) is formed in the same pass:
+//   res[t, :]    = x[t, :] + src_scale * sum_i rscale_i(t) * (inner_w[i] ? n(src_i[t, :]) * inner_w[i] : src_i[t, :]) + sum_k pair_w[t * top + k] * pair_src[pair_row[t * top + k], :]
+//   next_y[t, :] = tanh(next_alpha * res[t, :]) * next_w + next_b       (next_y null: none)
+// x is the stream itself, or (table != null: the embedding) table_scale * table[ids[t], :].  n: division by the row's root mean square
+// (eps inside the root).  rscale_i(t) = rscale[i][t] or 1.  Sources and weights in elt; sums, statistics and tanh in fp32.
+struct DytCombineArgs {
+  float* res = nullptr; const int32_t* ids = nullptr; const void* table = nullptr; float table_scale = 1.f;
+  const void* src[2] = {nullptr, nullptr}; int ld[2] = {0, 0}; const void* inner_w[2] = {nullptr, nullptr}; const float* rscale[2] = {nullptr, nullptr}; int nsrc = 0; float src_scale = 1.f;
+  const void* pair_src = nullptr; const int32_t* pair_row = nullptr; const float* pair_w = nullptr; int top = 0;
+  float next_alpha = 0.f; const void* next_w = nullptr; const void* next_b = nullptr; void* next_y = nullptr;
+  int T = 0, d = 0; float eps = 1e-5f; int elt = KGE_ELT_BF16;
+};
+int dyt_combine(const DytCombineArgs& a, cudaStream_t st);
 
 // res[t, :] = float(table[ids[t], :])
 int embed_f32(float* res, const int32_t* ids, const void* table, int T, int d, int elt, cudaStream_t st);
@@ -110,12 +126,13 @@ struct ShortConvArgs {
   int B = 0, T = 0; int elt = KGE_ELT_BF16;
 };
 int short_conv_state(const ShortConvArgs& a, cudaStream_t st);
-// The same convolution followed by a silu and, for the first unit_heads * head_dim channels, a division of every head of
+// The same convolution (plus `bias` [C] where given) followed by a silu and, for the first unit_heads * head_dim channels, a division of every head of
 // head_dim channels by sqrt(sum of squares + unit_eps) (and a multiplication of the first scaled_heads of them by
-// head_scale); fp32 rows out.  Weights transposed: w [taps, C].  `inline_save`: every request of the step brings one row, so the
+// head_scale); fp32 rows out, or (out_elt) rows in elt.  Weights transposed: w [taps, C].  `inline_save`: every request of the step brings one row, so the
 // kernel that reads the slot's rows also brings them up to date.
 struct ConvHeadsArgs {
-  const void* x = nullptr; int ldx = 0; float* y = nullptr; int ldy = 0; const void* w = nullptr; int C = 0, taps = 1;
+  const void* x = nullptr; int ldx = 0; void* y = nullptr; int ldy = 0; const void* w = nullptr; const void* bias = nullptr; int C = 0, taps = 1;
+  bool out_elt = false;
   int unit_heads = 0, scaled_heads = 0, head_dim = 1; float head_scale = 1.f, unit_eps = 1e-6f;
   float* state = nullptr; int64_t slot_stride = 0;
   const int32_t* slots = nullptr; const int32_t* qsl = nullptr; const int32_t* positions = nullptr; const int32_t* token_req = nullptr;
@@ -223,6 +240,9 @@ int rotate_heads_halves(void* x, int ldx, const int32_t* positions, const double
 // between lo = max(floor(c(fast)), 0) and hi = min(ceil(c(slow)), dims - 1), c(t) = dims * ln(original / (2 pi t)) / (2 ln base);
 // freq_i <- freq_i / factor * ramp_i + freq_i * (1 - ramp_i) and *mult = 0.1 ln(factor) + 1 (else 1).  Host only.
 void rotary_frequencies(int dims, double base, double factor, double original, double fast, double slow, double* freq, float* mult);
+// freq[i] = base^(-2i / dims), scaled by wavelength l = 2 pi / freq (factor 0: not): kept where l < original / high, divided by factor
+// where l > original / low, in between (1 - s) * freq / factor + s * freq with s = (original / l - low) / (high - low).  Host only.
+void rotary_frequencies_banded(int dims, double base, double factor, double low, double high, double original, double* freq);
 
 // Gated linear recurrence (RG-LRU).  yx [T, 2 * width]: the y branch's pre-activation, then the x branch (biases in).
 //   u = causal per-channel conv of x (taps weights per channel, last tap on the current token; inputs before position 0
@@ -272,7 +292,8 @@ inline int64_t mlstm_state_floats(int H, int dim, int vdim) { return (int64_t)H 
 // expert the list of (token, choice) pairs routed to it: group_off [E + 1], perm_token [T * top] (the token row of
 // every permuted row), perm_weight [T * top], perm_dest [T * top] (row t * top + choice of the output buffer).
 // `correction` (fp32 [E]) is added to the scores for the choice only.  groups > 1: neighbouring router outputs form equal
-// groups, and only those of the groups_keep groups with the largest best (corrected) score can be chosen.  The last
+// groups, and only those of the groups_keep groups with the largest score can be chosen; a group's score is the sum of its
+// group_best (1 or 2) largest (corrected) scores.  renorm divides by the sum of the chosen scores + renorm_eps.  The last
 // `identity` of the E outputs are experts without tensors: their pairs join no list (group_off has E - identity + 1
 // entries); pair_row [T * top] names every pair's permuted row, -1 for an identity expert.
 struct MoeRouteArgs {
@@ -285,7 +306,9 @@ struct MoeRouteArgs {
   // entries, -1 in perm_token / perm_dest marks a row without a pair), and tile_group [rows_padded / pad] names the expert
   // of every tile of `pad` rows (-1: none) - what the grouped tensor-core GEMM reads
   int pad = 0, rows_padded = 0; int32_t* tile_group = nullptr;
-  const float* logits = nullptr;          // fp32 [T, E]: the router's logits, ready (bias in), instead of h and w_router
+  const float* logits = nullptr;          // fp32 [T, E] (row stride ld_logits, 0: E): the router's logits, ready (bias in), instead of h and w_router;
+  int ld_logits = 0;                      // with extra_sigmoid, column E holds the extra row's product
+  float renorm_eps = 0.f; int group_best = 1;
   const float* correction = nullptr; int groups = 1, groups_keep = 1, identity = 0; int32_t* pair_row = nullptr;
   int elt = KGE_ELT_BF16;
 };
@@ -431,6 +454,37 @@ struct DeltaArgs {
 };
 int delta_scan(const DeltaArgs& a, cudaStream_t st);
 inline int64_t delta_state_floats(int H, int dim, int vdim) { return (int64_t)H * dim * vdim; }
+
+// Selective scan.  Per channel c and state number n, with the step size dt > 0 (fp32 [T, C]) and A = -exp(A_log) (fp32 [C, N]):
+//   S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n;   y_c = sum_n S[c, n] C_n + D_c x_c;   out_c = y_c * silu(z_c)
+// x, z [T, C] and the token's B and C rows (N numbers each) in elt, out in elt, all else fp32.  State per slot: S [C, N], zero at
+// position 0.  N <= 256.
+struct SelectiveScanArgs {
+  const void* x = nullptr; int ldx = 0; const void* z = nullptr; int ldz = 0; const void* b = nullptr; const void* c = nullptr; int ldbc = 0;
+  const float* dt = nullptr; int lddt = 0; const float* A = nullptr; const float* D = nullptr; void* out = nullptr; int ldo = 0;
+  float* state = nullptr; int64_t slot_stride = 0;
+  const int32_t* slots = nullptr; const int32_t* qsl = nullptr; const int32_t* positions = nullptr;
+  int B = 0, T = 0, C = 0, N = 0; int elt = KGE_ELT_BF16;
+};
+int selective_scan(const SelectiveScanArgs& a, cudaStream_t st);
+inline int64_t selective_state_floats(int C, int N) { return (int64_t)C * N; }
+
+// State-space dual recurrence: a state S [N, P] per head with ONE decay per head and token.  With dt = softplus(dt_pre + dt_bias)
+// (dt_pre in elt, row stride lddt) and head h reading B and C of group h / (H / G):
+//   S <- exp(-a_coef_h dt) S + dt B x^T;   y = S^T C + D_h x   -> o32 [T, H * P] (fp32)
+// x [T, H * P], B and C [T, G * N] in elt with one row stride ld; a_coef = exp(A_log), dt_bias and D fp32 [H].  State per slot: S [H, N, P]
+// fp32, zero at position 0.  N <= 256.
+//   gated_group_rmsnorm: out = gn(y * silu(z)) * w: the gate first, then the group norm above over the row (n columns in `groups` parts)
+struct SsdArgs {
+  const void* x = nullptr; const void* b = nullptr; const void* c = nullptr; int ld = 0; const void* dt_pre = nullptr; int lddt = 0;
+  const float* dt_bias = nullptr; const float* a_coef = nullptr; const float* D = nullptr; float* o32 = nullptr;
+  float* state = nullptr; int64_t slot_stride = 0;
+  const int32_t* slots = nullptr; const int32_t* qsl = nullptr; const int32_t* positions = nullptr;
+  int B = 0, T = 0, H = 0, G = 1, N = 0, P = 0; int elt = KGE_ELT_BF16;
+};
+int ssd_scan(const SsdArgs& a, cudaStream_t st);
+inline int64_t ssd_state_floats(int H, int N, int P) { return (int64_t)H * N * P; }
+int gated_group_rmsnorm(void* out, int ldo, const float* y, const void* z, int ldz, const void* w, int T, int n, int groups, float eps, int elt, cudaStream_t st);
 
 int sigmoid_gate_mul(void* y, int ldy, const void* g, int ldg, int T, int n, int elt, cudaStream_t st);
 

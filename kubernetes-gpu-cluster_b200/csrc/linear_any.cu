@@ -23,6 +23,7 @@ __device__ __forceinline__ float act_apply(int act, float v) {
     case ACT_SIGMOID: return 1.f / (1.f + expf(-v));
     case ACT_TANH: return tanhf(v);
     case ACT_RELU2: { const float r = fmaxf(v, 0.f); return r * r; }
+    case ACT_SOFTPLUS: return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v)));      // without overflow on either side
     default: return v;
   }
 }

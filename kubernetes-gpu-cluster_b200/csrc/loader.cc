@@ -401,7 +401,77 @@ static bool parse_kogonex(const Json& j, ModelSpec* s, std::string* err) {
   return true;
 }
 
+// Nosolix: a layer list of 'mamba1' mixers (selective scans) and 'parallel' mixers (windowed attention with an output gate
+// and rotary positions in halves whose frequencies are scaled by wavelength, beside a state-space dual recurrence), dense
+// squared-ReLU units or clamped gated experts (sigmoid scores, a choice correction, groups judged by their two best,
+// normalised weights, a gated shared expert), Dynamic Tanh before every sublayer, and a scaled embedding.
+static bool parse_nosolix(const Json& j, ModelSpec* s, std::string* err) {
+  s->model_type = "nosolix";
+  s->vocab = (int)j.int_or("vocab", 0);
+  s->d = (int)j.int_or("width", 0);
+  if (const Json* n = j.get("norm")) s->eps = (float)n->num_or("eps", 1e-5);
+  if (const Json* e = j.get("embedding")) if (e->is_obj()) s->embed_scale = (float)e->num_or("scale", 1.0);
+  s->hyb_prenorm_pair = s->hyb_dyt = true;
+  s->max_pos = 1 << 20;                 // rotary angles are computed from the position: no table bounds them
+  s->torch_dtype = "bfloat16";
+  s->bos = (int)j.int_or("bos_token_id", -1);
+  s->eos = (int)j.int_or("eos_token_id", -1);
+  if (s->vocab <= 0 || s->d <= 0) { *err = "config.json misses a required size"; return false; }
+  const Json* ls = j.get("layers");
+  if (!ls || !ls->is_arr() || ls->arr.empty()) { *err = "config.json: 'layers' must be a non-empty array"; return false; }
+  for (const Json& l : ls->arr) {
+    HybridLayerSpec h;
+    const std::string type = l.str_or("type", "");
+    const Json* m = l.get("mixer");
+    if (!m || !m->is_obj()) { *err = "config.json: a layer has no 'mixer'"; return false; }
+    if (type == "mamba1") {
+      h.mixer = HybridLayerSpec::MAMBA;
+      h.width = (int)m->int_or("inner", 0); h.n_state = (int)m->int_or("state", 0); h.decay_rank = (int)m->int_or("dt_rank", 0); h.conv = (int)m->int_or("conv", 1);
+      if (h.width <= 0 || h.n_state <= 0 || h.n_state > 256 || h.decay_rank <= 0 || h.conv < 1 || h.conv > 16) {
+        *err = "config.json: bad mamba1 sizes (state <= 256, 1 <= conv <= 16)"; return false;
+      }
+    } else if (type == "parallel") {
+      h.mixer = HybridLayerSpec::WINDOW_SSD;
+      const Json *a = m->get("left"), *r = m->get("right");
+      if (!a || !a->is_obj() || !r || !r->is_obj()) { *err = "config.json: a parallel mixer needs 'left' and 'right'"; return false; }
+      h.window = 1 << 30;               // without a mask: the whole causal prefix
+      if (const Json* mk = a->get("mask")) if (mk->is_obj()) h.window = (int)std::min<int64_t>(mk->int_or("size", 0), (int64_t)1 << 30);
+      h.heads = (int)a->int_or("heads", 0); h.kv_heads = (int)a->int_or("kv_heads", h.heads);
+      h.dim = (int)a->int_or("dim", 0); h.vdim = (int)a->int_or("vdim", h.dim);
+      h.scale = (float)a->num_or("scale", 1.0);
+      h.rot_halves = h.out_gate = true;
+      if (const Json* ro = a->get("rot")) if (ro->is_obj()) {
+        h.rot_dims = (int)ro->int_or("dims", 0); h.rot_base = ro->num_or("base", 10000.0);
+        const Json* sc = ro->get("scaling");
+        if (sc && sc->is_obj()) {
+          h.rot_factor = sc->num_or("factor", 0.0); h.rot_low = sc->num_or("low", 1.0); h.rot_high = sc->num_or("high", 4.0); h.rot_original = sc->num_or("original", 0.0);
+          if (h.rot_factor <= 0.0 || h.rot_low <= 0.0 || h.rot_high <= 0.0 || h.rot_original <= 0.0) { *err = "config.json: bad rotary scaling"; return false; }
+        }
+      }
+      if (h.heads <= 0 || h.kv_heads <= 0 || h.heads % h.kv_heads || h.dim <= 0 || h.vdim <= 0 || h.window <= 0 || h.rot_dims < 0 || h.rot_dims > h.dim ||
+          h.rot_dims % 2 || h.rot_base <= 0.0) { *err = "config.json: bad sizes of the attention side"; return false; }
+      h.m_heads = (int)r->int_or("heads", 0); h.m_vdim = (int)r->int_or("vdim", 0); h.n_state = (int)r->int_or("state", 0); h.ssd_groups = (int)r->int_or("groups", 1);
+      h.out_norm_groups = (int)r->int_or("norm_groups", 1); h.conv = (int)r->int_or("conv", 1);
+      if (h.m_heads <= 0 || h.m_vdim <= 0 || h.n_state <= 0 || h.n_state > 256 || h.ssd_groups <= 0 || h.m_heads % h.ssd_groups || h.out_norm_groups <= 0 ||
+          h.m_heads * h.m_vdim % h.out_norm_groups || h.conv < 1 || h.conv > 16) {
+        *err = "config.json: bad sizes of the recurrent side (groups divides heads, norm_groups heads * vdim, state <= 256, 1 <= conv <= 16)"; return false;
+      }
+    } else { *err = "config.json: unknown layer type '" + type + "' (mamba1, parallel)"; return false; }
+    if (!parse_hybrid_mlp(l, &h, err)) return false;
+    if (h.mlp == HybridLayerSpec::DENSE) { h.ff_relu2 = true; h.ff_limit = 0.f; }
+    if (h.mlp == HybridLayerSpec::MOE) {
+      if (h.identity > 0) { *err = "config.json: this architecture has no identity experts"; return false; }
+      if (h.expert_limit <= 0.f || (h.shared_ff > 0 && h.shared_limit <= 0.f)) { *err = "config.json: an expert needs a positive 'limit'"; return false; }
+      h.route = HybridLayerSpec::ROUTE_SIGMOID_NORM; h.glu = HybridLayerSpec::GLU_CLAMPED; h.router_correction = true; h.group_best = 2; h.shared_gate = h.shared_ff > 0;
+    }
+    s->hybrid.push_back(h);
+  }
+  s->L = (int)s->hybrid.size();
+  return true;
+}
+
 static bool parse_config(const Json& j, ModelSpec* s, std::string* err) {
+  if (j.str_or("architecture", "") == "Nosolix") return parse_nosolix(j, s, err);
   if (j.str_or("architecture", "") == "Kogonex") return parse_kogonex(j, s, err);
   if (j.str_or("architecture", "") == "Safupel") return parse_hybrid(j, s, err);
   if (j.str_or("architecture", "") == "Balenex") return parse_balenex(j, s, err);
@@ -644,21 +714,24 @@ extern "C" int kge_model_spec_json(const kge_model_dir* m, char* out, int cap) {
                "\"shared_limit\":%.9g,\"weights_of\":%d,\"tensor_index\":%d,\"q_rank\":%d,\"kv_rank\":%d,\"rot_part\":%d,\"out_gate\":%d,"
                "\"decay_rank\":%d,\"ff_limit\":%.9g,\"router_scale\":%.9g,\"window\":%d,\"keep_first\":%d,\"pool\":%d,\"tau\":%.9g,"
                "\"head_norm\":%d,\"rot_halves\":%d,\"v_rot\":%d,\"ff_silu_bias\":%d,\"latent_cache\":%d,\"kv_from\":%d,\"sink\":%d,"
-               "\"identity\":%d,\"router_groups\":%d,\"groups_keep\":%d,\"router_correction\":%d}",
+               "\"identity\":%d,\"router_groups\":%d,\"groups_keep\":%d,\"router_correction\":%d,\"n_state\":%d,\"ssd_groups\":%d,\"out_norm_groups\":%d,"
+               "\"rot_factor\":%.17g,\"rot_low\":%.17g,\"rot_high\":%.17g,\"rot_original\":%.17g,\"ff_relu2\":%d,\"group_best\":%d,\"shared_gate\":%d}",
                i ? "," : "", h.mixer, h.width, h.blocks, h.conv, h.heads, h.kv_heads, h.dim, h.vdim, h.chunk, (double)h.scale, (double)h.left_scale,
                (double)h.right_scale, h.m_heads, h.m_dim, h.m_vdim, (double)h.gate_cap, h.mlp, h.ff, h.experts, h.top, h.expert_ff, h.shared_ff,
                (double)h.softcap, h.rot_dims, h.rot_base, h.yarn_factor, h.yarn_original, h.yarn_fast, h.yarn_slow, h.route, h.glu, (double)h.expert_limit,
                (double)h.shared_limit, h.weights_of, h.tensor_index < 0 ? (int)i : h.tensor_index, h.q_rank, h.kv_rank, h.rot_part, h.out_gate ? 1 : 0,
                h.decay_rank, (double)h.ff_limit, (double)h.router_scale, h.window, h.keep_first, h.pool, (double)h.tau, h.head_norm ? 1 : 0,
                h.rot_halves ? 1 : 0, h.v_rot ? 1 : 0, h.ff_silu_bias ? 1 : 0, h.latent_cache ? 1 : 0, h.kv_from, h.sink ? 1 : 0, h.identity, h.router_groups,
-               h.groups_keep, h.router_correction ? 1 : 0);
+               h.groups_keep, h.router_correction ? 1 : 0, h.n_state, h.ssd_groups, h.out_norm_groups, h.rot_factor, h.rot_low, h.rot_high, h.rot_original,
+               h.ff_relu2 ? 1 : 0, h.group_best, h.shared_gate ? 1 : 0);
       j += buf;
     }
     snprintf(buf, sizeof buf, "],\"eps\":%.9g,\"logit_scale\":%.9g,\"logit_softcap\":%.9g,\"streams\":%d,\"residual_mult\":%.9g,\"embed_norm\":%s,"
-             "\"norm_groups\":%d,\"postnorm\":%s,\"noprenorm\":%s,\"bigram_buckets\":%lld,\"bigram_mul_prev\":%lld,\"bigram_mul_cur\":%lld}", (double)s.eps,
+             "\"norm_groups\":%d,\"postnorm\":%s,\"noprenorm\":%s,\"bigram_buckets\":%lld,\"bigram_mul_prev\":%lld,\"bigram_mul_cur\":%lld,"
+             "\"dyt\":%s,\"embed_scale\":%.9g}", (double)s.eps,
              (double)s.logit_scale, (double)s.logit_softcap, s.streams, (double)s.residual_mult, s.embed_norm ? "true" : "false", s.norm_groups,
              s.hyb_postnorm ? "true" : "false", s.hyb_noprenorm ? "true" : "false", (long long)s.bigram_buckets, (long long)s.bigram_mul_prev,
-             (long long)s.bigram_mul_cur);
+             (long long)s.bigram_mul_cur, s.hyb_dyt ? "true" : "false", (double)s.embed_scale);
     j += buf;
     KGE_REQUIRE((int)j.size() < cap, "kge_model_spec_json: buffer of %d bytes too small", cap);
     memcpy(out, j.c_str(), j.size() + 1);

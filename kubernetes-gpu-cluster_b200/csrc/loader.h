@@ -12,7 +12,7 @@ namespace kge {
 // One layer of a layer-list ("hybrid") model: which token mixer it has, that mixer's sizes and constants, and its
 // feed-forward.  Every number comes from config.json; the kernels take them as parameters.
 struct HybridLayerSpec {
-  enum Mixer { RGLRU = 0, PARALLEL = 1, ATTENTION = 2, WKV = 3, LATENT = 4, WINDOW_GLA = 5, POOLED = 6, DELTA = 7 };
+  enum Mixer { RGLRU = 0, PARALLEL = 1, ATTENTION = 2, WKV = 3, LATENT = 4, WINDOW_GLA = 5, POOLED = 6, DELTA = 7, MAMBA = 8, WINDOW_SSD = 9 };
   enum Mlp { NONE = 0, DENSE = 1, MOE = 2 };
   int mixer = RGLRU;
   // gated linear recurrence (RG-LRU): two branches of `width`, gates block-diagonal in `blocks` parts, causal conv of `conv` taps
@@ -68,10 +68,21 @@ struct HybridLayerSpec {
   int window = 0, keep_first = 0, pool = 0;
   bool head_norm = false, rot_halves = false, v_rot = false;
   float tau = 1.f;
+  // selective scan (MAMBA): `width` channels behind a causal convolution of `conv` taps with a bias and a silu, `n_state` numbers per
+  // channel, step sizes through a low-rank pair of `decay_rank` columns, a direct term per channel and a silu gate.
+  // windowed attention beside a state-space dual recurrence (WINDOW_SSD), results normed and averaged as in WINDOW_GLA.
+  //   attention side: rot_halves with frequencies scaled by wavelength (rot_factor 0: plain; see rotary_frequencies_banded), the heads'
+  //   outputs multiplied by sigmoid(W_g h) (out_gate), a window.
+  //   recurrent side: m_heads x (n_state x m_vdim) state with one decay per head and token; x, B and C (B and C on `ssd_groups`
+  //   groups of heads) pass a causal convolution of `conv` taps with a bias and a silu; the read-out plus a direct term per head is
+  //   multiplied by silu(z), then RMS-normed in out_norm_groups equal parts.
+  int n_state = 0, ssd_groups = 1, out_norm_groups = 1;
+  double rot_factor = 0.0, rot_low = 1.0, rot_high = 4.0, rot_original = 0.0;
   // feed-forward
   int mlp = NONE;
   int ff = 0;                                    // dense
   float ff_limit = 0.f;                          // dense: > 0 - a clamped gated unit (gate, up, down) with this limit; 0 - up, GELU, down
+  bool ff_relu2 = false;                         // dense: down(relu(up h)^2)
   bool ff_silu_bias = false;                     // dense: down(silu(gate h + b) * (up h + b)) + b, every projection with a bias
   int experts = 0, top = 0, expert_ff = 0, shared_ff = 0;   // mixture of experts (+ an always-on shared expert if shared_ff > 0)
   // how the experts are chosen and weighed: ROUTE_SIGMOID_IN - sigmoid scores, the weight multiplies the expert's input;
@@ -83,11 +94,13 @@ struct HybridLayerSpec {
   // neighbouring experts form that many equal groups and only those of the groups_keep groups with the largest best score
   // can be chosen; the last `identity` router outputs are experts that return their input and own no tensors: `experts`
   // counts the others)
-  enum Route { ROUTE_SIGMOID_IN = 0, ROUTE_SOFTMAX_TOP = 1, ROUTE_SOFTMAX_ALL = 2 };
+  // ROUTE_SIGMOID_NORM - sigmoid scores, weights divided by their sum (+ 1e-20) and multiplied by router_scale, multiply the
+  // expert's output; group_best: how many of a group's largest choice scores add up to the group's score
+  enum Route { ROUTE_SIGMOID_IN = 0, ROUTE_SOFTMAX_TOP = 1, ROUTE_SOFTMAX_ALL = 2, ROUTE_SIGMOID_NORM = 3 };
   int route = ROUTE_SIGMOID_IN;
   float router_scale = 1.f;
   bool router_bias = false, router_correction = false;
-  int router_groups = 1, groups_keep = 1, identity = 0;
+  int router_groups = 1, groups_keep = 1, identity = 0, group_best = 1;
   // the experts' gated unit: GLU_SILU - silu(gate) * up; GLU_CLAMPED - g = min(gate, limit), u = clamp(up, -limit, limit),
   // g * sigmoid(1.702 g) * (u + 1)
   // GLU_NONE_RELU2 - no gate: down(relu(up h)^2)
@@ -97,14 +110,14 @@ struct HybridLayerSpec {
   bool shared_gate = false;                      // the shared expert's output is multiplied by sigmoid(w_sg . h), one number per token
   int weights_of = -1;                           // >= 0: this layer owns no tensors and runs with that layer's (cache and state stay its own)
   int tensor_index = -1;                         // the 'l<i>.' prefix of this layer's tensors (-1: its place in the list)
-  bool has_cache() const { return mixer == PARALLEL || mixer == ATTENTION || (mixer == LATENT && kv_from < 0) || mixer == WINDOW_GLA || mixer == POOLED; }
+  bool has_cache() const { return mixer == PARALLEL || mixer == ATTENTION || (mixer == LATENT && kv_from < 0) || mixer == WINDOW_GLA || mixer == POOLED || mixer == WINDOW_SSD; }
   // numbers of one token's row in the paged caches (keys, then values), over all key/value heads
   int64_t cache_k_row() const { return latent_cache ? kv_rank + rot_part : (int64_t)kv_heads * dim; }
   int64_t cache_v_row() const { return latent_cache ? 0 : (int64_t)kv_heads * vdim; }
 };
 
 struct ModelSpec {
-  std::string model_type;       // "opt" | "llama" | "qwen2" | "qwen3" | "safupel" | "girolorn" | "zezilix" | "balenex" | "kogonex"
+  std::string model_type;       // "opt" | "llama" | "qwen2" | "qwen3" | "safupel" | "girolorn" | "zezilix" | "balenex" | "kogonex" | "nosolix"
   // layer-list models (config.json "architecture"): per-layer descriptions and the multiplier of the logits
   std::vector<HybridLayerSpec> hybrid;
   float logit_scale = 1.f;
@@ -120,6 +133,10 @@ struct ModelSpec {
   // named norm1 / norm2)
   int norm_groups = 1;
   bool hyb_postnorm = false, hyb_noprenorm = false;
+  // hyb_dyt: in the place of the norms, Dynamic Tanh: tanh(alpha x) * w + b with a scalar alpha and vectors w and b (no statistics);
+  // the embedding is multiplied by embed_scale
+  bool hyb_dyt = false;
+  float embed_scale = 1.f;
   // bigram embedding: row (previous token * mul_prev + token * mul_cur) mod buckets of a second table is added to the
   // token's embedding; a sequence's first token takes row `buckets` (0 buckets: none)
   int64_t bigram_buckets = 0, bigram_mul_prev = 0, bigram_mul_cur = 0;

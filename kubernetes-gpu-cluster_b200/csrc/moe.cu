@@ -66,9 +66,9 @@ __device__ __forceinline__ void moe_pick(const MoeRouteArgs& a, int t, float* sc
       float* gb = ch + a.E;                     // a group's best, -inf once it is kept
       const int gs = a.E / a.groups;
       for (int g = lane; g < a.groups; g += 32) {
-        float m = -INFINITY;
-        for (int e = 0; e < gs; ++e) m = fmaxf(m, ch[g * gs + e]);
-        gb[g] = m;
+        float m = -INFINITY, m2 = -INFINITY;      // the group's largest and second largest
+        for (int e = 0; e < gs; ++e) { const float v = ch[g * gs + e]; m2 = fmaxf(m2, fminf(m, v)); m = fmaxf(m, v); }
+        gb[g] = a.group_best > 1 && gs > 1 ? m + m2 : m;
       }
       __syncwarp();
       for (int k = 0; k < a.groups_keep; ++k) {
@@ -119,6 +119,7 @@ __device__ __forceinline__ void moe_pick(const MoeRouteArgs& a, int t, float* sc
     } else if (a.renorm) {
       float total = 0.f;
       for (int k = 0; k < a.top; ++k) total += cw[k];
+      total += a.renorm_eps;
       for (int k = 0; k < a.top; ++k) cw[k] /= total;
     }
     if (a.weight_scale != 1.f) for (int k = 0; k < a.top; ++k) cw[k] *= a.weight_scale;
@@ -159,7 +160,9 @@ __global__ void __launch_bounds__(256) moe_pick_kernel(MoeRouteArgs a, int per_w
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * 8 + warp;
   if (t >= a.T) return;
   float* sc = sc_all + warp * per_warp;
-  for (int e = lane; e < a.E; e += 32) sc[e] = a.logits[(int64_t)t * a.E + e];
+  const int64_t ld = a.ld_logits > 0 ? a.ld_logits : a.E;
+  for (int e = lane; e < a.E; e += 32) sc[e] = a.logits[(int64_t)t * ld + e];
+  if (a.extra_sigmoid && lane == 0) a.extra_sigmoid[t] = 1.f / (1.f + expf(-a.logits[(int64_t)t * ld + a.E]));
   __syncwarp();
   moe_pick(a, t, sc, lane);
 }
@@ -252,7 +255,7 @@ int moe_route(const MoeRouteArgs& a, cudaStream_t st) {
               (a.identity == 0 || a.pair_row), "moe_route: %d groups (%d kept), %d identity experts of %d", a.groups, a.groups_keep, a.identity, a.E);
   const int per = a.correction || a.groups > 1 ? 2 * a.E + a.groups : a.E;
   const size_t smem = (size_t)per * 4;
-  KGE_REQUIRE(!a.logits || (!a.w_extra && smem * 8 <= 48 * 1024), "moe_route: %d router outputs with ready logits", a.E);
+  KGE_REQUIRE(!a.logits || ((!a.extra_sigmoid || a.ld_logits > a.E) && smem * 8 <= 48 * 1024), "moe_route: %d router outputs with ready logits", a.E);
   cudaError_t ce;
   if (a.logits) ce = launch_pdl(moe_pick_kernel, dim3((a.T + 7) / 8), dim3(256), smem * 8, st, a, per);
   else ce = a.elt == KGE_ELT_F32 ? launch_pdl(moe_score_kernel<float>, dim3(a.T), dim3(256), smem, st, a)

@@ -30,6 +30,18 @@ void rotary_frequencies(int dims, double base, double factor, double original, d
   }
 }
 
+void rotary_frequencies_banded(int dims, double base, double factor, double low, double high, double original, double* freq) {
+  const double pi = 3.14159265358979323846;
+  for (int i = 0; i < dims / 2; ++i) {
+    const double f = pow(base, -2.0 * i / dims), wave = 2.0 * pi / f;
+    freq[i] = f;
+    if (factor <= 0.0 || wave < original / high) continue;
+    if (wave > original / low) { freq[i] = f / factor; continue; }
+    const double s = (original / wave - low) / (high - low);
+    freq[i] = (1.0 - s) * f / factor + s * f;
+  }
+}
+
 // sin and cos of an angle formed in double precision: whole turns are taken off in double (three operations), the rest -
 // within [-pi, pi], exact to an fp32 rounding - goes through the fp32 functions
 __device__ __forceinline__ void sincos_reduced(double ang, float* s, float* c) {

@@ -87,7 +87,7 @@ __global__ void __launch_bounds__(256) short_conv_save_kernel(ShortConvArgs a) {
 // One warp per (token, head of head_dim channels) for the unit heads and per (token, 128 channels) for the rest: the
 // convolution's sums, the silu and a head's sum of squares stay in the warp's registers.  VEC: four neighbouring channels
 // per lane and pass.
-template <typename E, bool VEC>
+template <typename E, typename O, bool VEC>
 __global__ void __launch_bounds__(256) short_conv_silu_heads_kernel(ConvHeadsArgs a, int items) {
   pdl_launch_dependents();
   pdl_wait();
@@ -111,6 +111,10 @@ __global__ void __launch_bounds__(256) short_conv_silu_heads_kernel(ConvHeadsArg
     for (int q = 0; q < W; ++q) acc[p][q] = 0.f;
     if (k < n) {
       const int c = c0 + k;
+      if (a.bias) {
+#pragma unroll
+        for (int q = 0; q < W; ++q) acc[p][q] = ldf((const E*)a.bias + c + q);
+      }
       for (int j = 0; j < taps; ++j) {
         const int back = taps - 1 - j;                  // the input of position pos - back
         if (pos - back < 0) continue;
@@ -145,14 +149,14 @@ __global__ void __launch_bounds__(256) short_conv_silu_heads_kernel(ConvHeadsArg
     f = 1.f / sqrtf(warp_sum(ss) + a.unit_eps);
     if (u < a.scaled_heads) f *= a.head_scale;
   }
-  float* y = a.y + (int64_t)t * a.ldy + c0;
+  O* y = (O*)a.y + (int64_t)t * a.ldy + c0;
 #pragma unroll
   for (int p = 0; p < MAXP; ++p) {
     const int k = (p * 32 + lane) * W;
     if (k < n) {
 #pragma unroll
       for (int q = 0; q < W; ++q) acc[p][q] *= f;
-      if constexpr (VEC) st4(y + k, acc[p]); else y[k] = acc[p][0];
+      if constexpr (VEC) st4(y + k, acc[p]); else stf(y + k, acc[p][0]);
     }
   }
 }
@@ -160,7 +164,7 @@ __global__ void __launch_bounds__(256) short_conv_silu_heads_kernel(ConvHeadsArg
 // The same for two to four taps and 16-byte rows: a warp keeps its channels' weights and the last taps - 1 inputs in registers
 // over a strip of TS tokens, so every input row is read once, and requests all rows of the strip before it uses the first.
 // MAXP: passes of 128 channels (heads of up to 128 * MAXP channels).
-template <typename E, int TAPS, int TS, int MAXP>
+template <typename E, typename O, int TAPS, int TS, int MAXP>
 __global__ void __launch_bounds__(256) short_conv_silu_heads_strip_kernel(ConvHeadsArgs a, int items) {
   pdl_launch_dependents();
   pdl_wait();
@@ -176,7 +180,7 @@ __global__ void __launch_bounds__(256) short_conv_silu_heads_strip_kernel(ConvHe
   const int ml = min(t0 + lane % TS, a.T - 1);                      // lane i knows token t0 + i's request, first row and position
   const int mb = a.token_req[ml], mr = a.qsl[mb], mp = a.positions[ml];
   const E* x = (const E*)a.x;
-  float cur[MAXP][TS][4], win[MAXP][TAPS - 1][4], w[MAXP][TAPS][4];
+  float cur[MAXP][TS][4], win[MAXP][TAPS - 1][4], w[MAXP][TAPS][4], bias[MAXP][4] = {};
 #pragma unroll
   for (int p = 0; p < MAXP; ++p) {
     const int k = (p * 32 + lane) * 4;
@@ -185,6 +189,7 @@ __global__ void __launch_bounds__(256) short_conv_silu_heads_strip_kernel(ConvHe
       for (int i = 0; i < TS; ++i) if (i < nt) ld4(x + (int64_t)(t0 + i) * a.ldx + c0 + k, cur[p][i]);
 #pragma unroll
       for (int j = 0; j < TAPS; ++j) ld4((const E*)a.w + (int64_t)j * a.C + c0 + k, w[p][j]);
+      if (a.bias) ld4((const E*)a.bias + c0 + k, bias[p]);
     }
   }
 #pragma unroll
@@ -211,7 +216,7 @@ __global__ void __launch_bounds__(256) short_conv_silu_heads_strip_kernel(ConvHe
         }
 #pragma unroll
         for (int q = 0; q < 4; ++q) {
-          float acc = 0.f;
+          float acc = bias[p][q];
 #pragma unroll
           for (int j = 0; j < TAPS - 1; ++j) acc = fmaf(w[p][j][q], win[p][j][q], acc);
           acc = fmaf(w[p][TAPS - 1][q], cur[p][i][q], acc);
@@ -238,24 +243,28 @@ __global__ void __launch_bounds__(256) short_conv_silu_heads_strip_kernel(ConvHe
       if (k < n) {
 #pragma unroll
         for (int q = 0; q < 4; ++q) y[p][q] *= f;
-        st4(a.y + (int64_t)t * a.ldy + c0 + k, y[p]);
+        st4((O*)a.y + (int64_t)t * a.ldy + c0 + k, y[p]);
       }
     }
   }
 }
 
-template <typename E, int TAPS, int TS>
+template <typename E, typename O, int TAPS, int TS>
 cudaError_t launch_strip(const ConvHeadsArgs& a, int items, cudaStream_t st) {
   const dim3 grid((unsigned)(((int64_t)((a.T + TS - 1) / TS) * items + 7) / 8));
-  return a.head_dim <= 128 ? launch_pdl(short_conv_silu_heads_strip_kernel<E, TAPS, TS, 1>, grid, dim3(256), 0, st, a, items)
-                           : launch_pdl(short_conv_silu_heads_strip_kernel<E, TAPS, TS, 2>, grid, dim3(256), 0, st, a, items);
+  return a.head_dim <= 128 ? launch_pdl(short_conv_silu_heads_strip_kernel<E, O, TAPS, TS, 1>, grid, dim3(256), 0, st, a, items)
+                           : launch_pdl(short_conv_silu_heads_strip_kernel<E, O, TAPS, TS, 2>, grid, dim3(256), 0, st, a, items);
 }
-template <typename E>
-cudaError_t launch_strips(const ConvHeadsArgs& a, int items, cudaStream_t st) {
-  const bool many = a.T >= 32 && a.T > a.B;                         // prompt pieces: strips of eight rows; single tokens: a warp per (row, head)
-  if (a.taps == 2) return many ? launch_strip<E, 2, 8>(a, items, st) : launch_strip<E, 2, 1>(a, items, st);
-  if (a.taps == 3) return many ? launch_strip<E, 3, 8>(a, items, st) : launch_strip<E, 3, 1>(a, items, st);
-  return many ? launch_strip<E, 4, 8>(a, items, st) : launch_strip<E, 4, 1>(a, items, st);
+template <typename E, typename O>
+cudaError_t launch_silu_heads(const ConvHeadsArgs& a, int items, cudaStream_t st) {
+  if (a.vec && a.taps >= 2 && a.taps <= 4) {
+    const bool many = a.T >= 32 && a.T > a.B;                       // prompt pieces: strips of eight rows; single tokens: a warp per (row, head)
+    if (a.taps == 2) return many ? launch_strip<E, O, 2, 8>(a, items, st) : launch_strip<E, O, 2, 1>(a, items, st);
+    if (a.taps == 3) return many ? launch_strip<E, O, 3, 8>(a, items, st) : launch_strip<E, O, 3, 1>(a, items, st);
+    return many ? launch_strip<E, O, 4, 8>(a, items, st) : launch_strip<E, O, 4, 1>(a, items, st);
+  }
+  const dim3 grid((unsigned)(((int64_t)a.T * items + 7) / 8));
+  return a.vec ? launch_pdl(short_conv_silu_heads_kernel<E, O, true>, grid, dim3(256), 0, st, a, items) : launch_pdl(short_conv_silu_heads_kernel<E, O, false>, grid, dim3(256), 0, st, a, items);
 }
 
 }  // namespace
@@ -266,13 +275,12 @@ int short_conv_silu_heads(const ConvHeadsArgs& a0, cudaStream_t st) {
   KGE_REQUIRE(a.taps >= 1 && a.taps <= SC_MAX_TAPS && a.C > 0 && a.head_dim > 0 && a.head_dim <= 256 && a.unit_heads * a.head_dim <= a.C,
               "short_conv_silu_heads: %d taps, %d heads of %d of %d channels", a.taps, a.unit_heads, a.head_dim, a.C);
   const int items = a.unit_heads + (a.C - a.unit_heads * a.head_dim + 127) / 128;
-  a.vec = a.C % 4 == 0 && a.head_dim % 4 == 0 && a.ldx % 4 == 0 && a.ldy % 4 == 0 && a.slot_stride % 4 == 0 &&
-          ((reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(a.state)) & 15) == 0;
-  const dim3 grid((unsigned)(((int64_t)a.T * items + 7) / 8));
+  a.vec = a.C % 4 == 0 && (a.unit_heads == 0 || a.head_dim % 4 == 0) && a.ldx % 4 == 0 && a.ldy % 4 == 0 && a.slot_stride % 4 == 0 &&
+          ((reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(a.bias) |
+            reinterpret_cast<uintptr_t>(a.state)) & 15) == 0;
   cudaError_t ce;
-  if (a.vec && a.taps >= 2 && a.taps <= 4) ce = a.elt == KGE_ELT_F32 ? launch_strips<float>(a, items, st) : launch_strips<__nv_bfloat16>(a, items, st);
-  else if (a.elt == KGE_ELT_F32) ce = a.vec ? launch_pdl(short_conv_silu_heads_kernel<float, true>, grid, dim3(256), 0, st, a, items) : launch_pdl(short_conv_silu_heads_kernel<float, false>, grid, dim3(256), 0, st, a, items);
-  else ce = a.vec ? launch_pdl(short_conv_silu_heads_kernel<__nv_bfloat16, true>, grid, dim3(256), 0, st, a, items) : launch_pdl(short_conv_silu_heads_kernel<__nv_bfloat16, false>, grid, dim3(256), 0, st, a, items);
+  if (a.elt == KGE_ELT_F32) ce = launch_silu_heads<float, float>(a, items, st);
+  else ce = a.out_elt ? launch_silu_heads<__nv_bfloat16, __nv_bfloat16>(a, items, st) : launch_silu_heads<__nv_bfloat16, float>(a, items, st);
   KGE_CUDA_OK(ce);
   if (a.inline_save || a.taps < 2) return 0;
   ShortConvArgs s;      // the slots' rows move up after every row of the step has been read
