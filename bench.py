@@ -2,7 +2,7 @@
 """Headline benchmark: output tokens/s at fixed concurrency (BASELINE.json `metric`).
 
   python bench.py --gpus N --steps K --warmup W [--workload c3|c2|c1] [--impl ours|reference]
-  python bench.py --designs [safupel|girolorn|zezilix|balenex|kogonex]   (a layer-list design beside the closest other model of equal size; one JSON line per size)
+  python bench.py --designs [safupel|girolorn|zezilix|balenex|kogonex|nosolix]   (a layer-list design beside the closest other model of equal size; one JSON line per size)
 
 A "step" is one whole job of the workload: every request prefilled (2k-token prompts, 8192 tokens
 per engine step as the continuous-batching scheduler cuts them) and decoded greedily to its output length.
@@ -648,6 +648,33 @@ def kogonex_configs(z):
     return kog, zezilix_configs(ZEZILIX_SIZES[z["zezilix"]])[0]
 
 
+NOSOLIX_SIZES = {
+    # selective scans, and windowed attention beside a state-space dual recurrence, with squared-ReLU units and grouped clamped
+    # experts (Nosolix) at sizes that resemble real layers: scans on twice the width with 16 numbers per channel, 128-wide
+    # attention heads with a window of 1024 positions, recurrent heads of 128 x 64; beside it the closest designs the engine has,
+    # of the same width, depth and heads: the one with convolved recurrences, attention and a matrix memory side by side, dense
+    # units and experts (Safupel, same expert sizes), and the one with windowed attention beside gated linear attention (Balenex)
+    "w2048": dict(width=2048, vocab=32000, reps=2, heads=16, kv=4, dim=128, window=1024, rot=128, r_heads=32, r_vdim=64, state=128, r_groups=2, conv=4,
+                  inner=4096, m_state=16, dt_rank=128, ff=8192, experts=16, groups=4, keep=2, top=2, eff=1024, sff=2048, other="w2048"),
+    "w4096": dict(width=4096, vocab=32000, reps=1, heads=32, kv=8, dim=128, window=1024, rot=128, r_heads=64, r_vdim=64, state=128, r_groups=2, conv=4,
+                  inner=8192, m_state=16, dt_rank=256, ff=14336, experts=8, groups=2, keep=1, top=2, eff=3584, sff=3584, other="w4096"),
+}
+
+
+def nosolix_configs(z):
+    left = {"dim": z["dim"], "heads": z["heads"], "kv_heads": z["kv"], "mask": {"size": z["window"]}, "scale": z["dim"] ** -0.5, "vdim": z["dim"],
+            "rot": {"base": 500000.0, "dims": z["rot"], "scaling": {"factor": 8.0, "high": 4.0, "low": 1.0, "original": 8192}}}
+    par = {"left": left, "right": {"conv": z["conv"], "groups": z["r_groups"], "heads": z["r_heads"], "norm_groups": z["r_groups"], "state": z["state"], "vdim": z["r_vdim"]}}
+    scan = {"conv": z["conv"], "dt_rank": z["dt_rank"], "inner": z["inner"], "state": z["m_state"]}
+    dense = {"ff": z["ff"], "kind": "dense"}
+    moe = {"expert": {"ff": z["eff"], "limit": 7.0}, "kind": "moe", "shared": {"ff": z["sff"], "limit": 7.0},
+           "router": {"experts": z["experts"], "groups": {"count": z["groups"], "keep": z["keep"]}, "scale": 2.5, "top": z["top"]}}
+    four = [{"mixer": par, "mlp": dense, "type": "parallel"}, {"mixer": scan, "mlp": moe, "type": "mamba1"},
+            {"mixer": scan, "mlp": dense, "type": "mamba1"}, {"mixer": par, "mlp": moe, "type": "parallel"}]
+    nos = {"architecture": "Nosolix", "embedding": {"scale": z["width"] ** 0.5}, "layers": four * z["reps"], "norm": {"eps": 1e-6}, "vocab": z["vocab"], "width": z["width"]}
+    return nos, design_configs(DESIGN_SIZES[z["other"]])[0], balenex_configs(BALENEX_SIZES[z["other"]])[0]
+
+
 def time_raw_steps(kge, llm, batch_np, steps, warmup):
     """Wall-clock seconds per synchronous engine step (metadata upload, kernels, sampled ids back), after warm-up."""
     import ctypes as C
@@ -679,7 +706,7 @@ def raw_batch(B, ctx, q, bs, vocab, seed):
 
 
 def run_designs(args):
-    """--designs [safupel|girolorn|zezilix|balenex|kogonex]: a layer-list design next to a Llama (or the closest other design) of equal size (random weights): one prefill step of 4 x 2048 tokens,
+    """--designs [safupel|girolorn|zezilix|balenex|kogonex|nosolix]: a layer-list design next to a Llama (or the closest other design) of equal size (random weights): one prefill step of 4 x 2048 tokens,
     one decode step of 64 requests at context 2048, wall-clock per step plus per-kernel device times against the roofline."""
     from kge_loader import load
     kge = load()
@@ -689,6 +716,7 @@ def run_designs(args):
     which = args.designs
     sizes, make, arms = {"girolorn": (GIROLORN_SIZES, girolorn_configs, ("girolorn", "llama")), "zezilix": (ZEZILIX_SIZES, zezilix_configs, ("zezilix", "girolorn")),
                          "balenex": (BALENEX_SIZES, balenex_configs, ("balenex", "safupel")), "kogonex": (KOGONEX_SIZES, kogonex_configs, ("kogonex", "zezilix")),
+                         "nosolix": (NOSOLIX_SIZES, nosolix_configs, ("nosolix", "safupel", "balenex")),
                          "safupel": (DESIGN_SIZES, design_configs, ("safupel", "llama"))}[which]
     if args.sizes:
         sizes = {k: v for k, v in sizes.items() if k in args.sizes.split(",")}
@@ -756,7 +784,7 @@ def main():
     ap.add_argument("--tp-exchange", default="peer", choices=["peer", "nccl"], help="TP data path: peer memory (default) or NCCL")
     ap.add_argument("--tp-timeout", type=float, default=420.0, help="seconds the tensor-parallel leg may take at N > 1")
     ap.add_argument("--sizes", default="", help="with --designs: the sizes to run, with commas between them (all by default)")
-    ap.add_argument("--designs", nargs="?", const="safupel", default=None, choices=["safupel", "girolorn", "zezilix", "balenex", "kogonex"],
+    ap.add_argument("--designs", nargs="?", const="safupel", default=None, choices=["safupel", "girolorn", "zezilix", "balenex", "kogonex", "nosolix"],
                     help="instead of the workload: a layer-list design (safupel, the default, or girolorn) beside a Llama of equal "
                     "size, prefill and decode steps with per-kernel rooflines (one GPU, random weights)")
     args = ap.parse_args()

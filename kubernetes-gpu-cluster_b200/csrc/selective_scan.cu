@@ -21,8 +21,13 @@ namespace {
 constexpr float LOG2E = 1.4426950408889634f;
 
 __device__ __forceinline__ float ex2(float v) { float r; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v)); return r; }
-// exp(v) of an exponent that 16-bit engines hold in units of log 2
-template <typename E> __device__ __forceinline__ float decay_exp(float v) { return std::is_same<E, float>::value ? expf(v) : ex2(v); }
+// exp(v) of an exponent that 16-bit engines hold in units of log 2.  A slowly decaying state is multiplied by numbers just below 1
+// thousands of times, where an exponential that errs by a unit in the last place on one side adds up; float32 engines round
+// the exact one to nearest.
+template <typename E> __device__ __forceinline__ float decay_exp(float v) {
+  if constexpr (std::is_same<E, float>::value) return (float)exp((double)v);
+  else return ex2(v);
+}
 template <typename E> __device__ __forceinline__ float silu_f(float v) { return std::is_same<E, float>::value ? v / (1.f + expf(-v)) : __fdividef(v, 1.f + ex2(-LOG2E * v)); }
 
 constexpr int SS_THREADS = 64;

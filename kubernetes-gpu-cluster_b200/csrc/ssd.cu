@@ -22,6 +22,11 @@ namespace kge {
 namespace {
 
 __device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
+// the decay of one token; float32 engines round the exact exponential to nearest (a slow decay is applied thousands of times)
+template <typename E> __device__ __forceinline__ float decay_exp(float v) {
+  if constexpr (std::is_same<E, float>::value) return (float)exp((double)v);
+  else return expf(v);
+}
 __device__ __forceinline__ float fast_ex2(float v) { float r; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v)); return r; }
 
 // ------------------------------------------------------------------------------------------------ one row per request
@@ -54,7 +59,7 @@ __global__ void __launch_bounds__(256) ssd_step_kernel(SsdArgs a) {
         bv[i] = ldf(Bp + n); cv[i] = ldf(Cp + n);
       }
     }
-    const float dt = softplus_f(pre + bias), dec = expf(-coef * dt);
+    const float dt = softplus_f(pre + bias), dec = decay_exp<E>(-coef * dt);
 #pragma unroll
     for (int k = 0; k < 4; ++k) dx[k] = dt * x[k];
 #pragma unroll
@@ -111,7 +116,7 @@ __global__ void __launch_bounds__(256) ssd_seq_kernel(SsdArgs a) {
     }
     if (tid < nt) {
       const float dt = softplus_f(ldf((const E*)a.dt_pre + (int64_t)(t0 + tid) * a.lddt + h) + bias);
-      dts[tid] = dt; dec[tid] = expf(-coef * dt);
+      dts[tid] = dt; dec[tid] = decay_exp<E>(-coef * dt);
     }
     __syncthreads();
     for (int t = 0; t < nt; ++t) {

@@ -131,6 +131,8 @@ def make_weights(cfg, seed=0):
             t = r(0.3) - 0.4
         elif last == "dt":
             t = r(1.0 / math.sqrt(shape[-1]))
+        elif last in ("o", "down") and len(parts) > 2 and "left" not in parts and "right" not in parts:
+            t = r(0.4 / math.sqrt(shape[-1]))      # results that are not normed before they join the stream
         else:
             t = r(1.5 / math.sqrt(shape[-1]))
         W[name] = t.to(torch.bfloat16).to(DT)
@@ -158,6 +160,12 @@ def bfloat16_noise(cfg, W, tokens):
     finally:
         ROUND = None
     return ((noisy - exact).pow(2).mean(-1).sqrt() / exact.pow(2).mean().sqrt()).numpy()
+
+
+def float32_noise(cfg, W, tokens):
+    """The same for 32-bit arithmetic: the distance between the oracle and its equations evaluated in float32."""
+    exact, single = forward(cfg, W, tokens), forward(cfg, {k: v.to(torch.float32) for k, v in W.items()}, tokens)
+    return ((single - exact).pow(2).mean(-1).sqrt() / exact.pow(2).mean().sqrt()).numpy()
 
 
 silu = torch.nn.functional.silu
@@ -226,7 +234,7 @@ def turn(x, rot):
     if n == 0:
         return x
     a = torch.arange(x.shape[0], dtype=DT)[:, None, None] * torch.tensor(frequencies(rot), dtype=DT)
-    c, s = torch.cos(a), torch.sin(a)
+    c, s = torch.cos(a).to(x.dtype), torch.sin(a).to(x.dtype)
     u, v = x[:, :, :n], x[:, :, n:2 * n]
     return torch.cat([u * c - v * s, v * c + u * s, x[:, :, 2 * n:]], dim=-1)
 
@@ -252,7 +260,7 @@ def dual_scan(x, B, C, a, D):
     """x [T, H, P]; B, C [T, G, N]; a (decay), D (step) [T, H] -> (y [T, H, P] without the direct term, final state [H, N, P])"""
     T, H, G = x.shape[0], x.shape[1], B.shape[1]
     g = torch.arange(H) // (H // G)
-    S = torch.zeros(H, B.shape[2], x.shape[2], dtype=DT)
+    S = torch.zeros(H, B.shape[2], x.shape[2], dtype=x.dtype)
     y = torch.zeros_like(x)
     for t in range(T):
         S = a[t][:, None, None] * S + D[t][:, None, None] * B[t, g][:, :, None] * x[t][:, None, :]

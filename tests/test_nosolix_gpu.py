@@ -1,0 +1,705 @@
+"""The Nosolix design in the engine against the plain float64 oracle (oracle/nosolix.py): every mechanism alone, whole
+prompts against pieces and token-by-token decoding, mixed batches, reused pages and state slots, keys just inside and
+just outside every window (scores peaked so that one key decides), slowly and quickly decaying states of both recurrences,
+convolution rows across every cut, rotary frequencies in all three bands, expert groups judged by their two best, the first
+tokens, long decoding, other sizes, and greedy generation through the scheduler.  float32 engines give the sharp
+comparison; bfloat16 ones are held to a rounding-sized bound."""
+import copy
+
+import numpy as np
+import pytest
+import torch
+
+from oracle import nosolix as ok
+
+pytestmark = pytest.mark.gpu
+
+
+def make_engine(kge, tmp_path, cfg, W, dtype="float32", tokens=512, bs=16, seqs=4, name="m", batched=0):
+    d = str(tmp_path / name)
+    ok.save_model_dir(d, cfg, W)
+    nb = (tokens + bs - 1) // bs
+    return kge.LLM(d, dtype=dtype, block_size=bs, num_gpu_blocks_override=nb + 1, max_model_len=nb * bs + 1, max_num_seqs=seqs,
+                   max_num_batched_tokens=batched or nb * bs, enable_prefix_caching=False)
+
+
+def run_pieces(llm, rid, tokens, pieces):
+    """Feed `tokens` in steps of the given sizes, asking for every position's logits."""
+    out, at = [], 0
+    for n in pieces:
+        llm.trace_add(rid, tokens[at:at + n])
+        out.append(llm.trace_step([(rid, n, list(range(n)))]))
+        at += n
+    assert at == len(tokens)
+    return np.concatenate(out)
+
+
+class Case:
+    """A sequence's logits in the oracle, where its choices of experts are closest, and (for 16-bit runs) what rounding alone
+    does to the logits."""
+
+    def __init__(self, cfg, W, toks, dtype="bfloat16"):
+        mg = []
+        self.toks, self.want = toks, ok.forward(cfg, W, toks, margins=mg).numpy()
+        self.margin = np.min(np.stack([m.numpy() for m in mg]), axis=0) if mg else np.full(len(toks), np.inf)
+        self.noise = ok.bfloat16_noise(cfg, W, toks) if dtype != "float32" else None
+
+
+def check(got, case, dtype, what="", rows=slice(None)):
+    """Row-wise error against the oracle, relative to the logits' size.  float32 engines are held to 2e-4.  bfloat16
+    engines are held to three times the rounding noise that nine rows in ten of the oracle stay below (no less than 4e-2);
+    one row in ten may pass that bound, up to three times the oracle's noisiest row.  A 16-bit run forms the router's logits
+    from rounded activations, so its prompts are made without close choices of experts (clear_prompt)."""
+    want = case.want[rows]
+    scale = np.sqrt((case.want ** 2).mean())
+    err = np.sqrt(((got - want) ** 2).mean(-1)) / scale
+    assert case.margin.min() > (1e-6 if dtype == "float32" else CLEAR * 0.99), f"{what}: a choice of experts hangs on a margin of {case.margin.min():.2g}"
+    lim = 2e-4 if dtype == "float32" else max(4e-2, 3.0 * float(np.quantile(case.noise, 0.9)))
+    over = err >= lim
+    worst = int(np.argmax(err))
+    if dtype != "float32" and over.any() and len(err) >= 10:
+        assert over.mean() <= 0.1 and (err < 3.0 * float(case.noise.max())).all(), f"{what}: {over.sum()} of {len(err)} rows over {lim:.3g}, row {worst} is {err[worst]:.3g} of the logits' size"
+        return
+    assert not over.any(), f"{what}: row {worst} is {err[worst]:.3g} of the logits' size (limit {lim:.3g})"
+
+
+def prompt(cfg, n, seed=1):
+    return torch.randint(0, cfg["vocab"], (n,), generator=torch.Generator().manual_seed(seed)).tolist()
+
+
+CLEAR = 0.01      # of a choice score
+
+
+def clear_prompt(cfg, W, n, seed=1):
+    """A random prompt in which every choice of experts is decided by a margin that rounding to 16 bits does not reach:
+    tokens whose choice is close are drawn again until none is left."""
+    g = torch.Generator().manual_seed(seed)
+    toks = torch.randint(0, cfg["vocab"], (n,), generator=g).tolist()
+    for _ in range(60):
+        mg = []
+        ok.forward(cfg, W, toks, margins=mg)
+        if not mg:
+            return toks
+        close = torch.nonzero(torch.stack(mg).min(0).values < CLEAR).flatten().tolist()
+        if not close:
+            return toks
+        # the first few close ones only: a new token also moves the rows after it
+        for t in close[:max(1, len(close) // 2)]:
+            toks[t] = int(torch.randint(0, cfg["vocab"], (1,), generator=g))
+    raise AssertionError("no prompt without close choices found")
+
+
+MOE, SCAN, PAR = ok.moe_mlp, ok.mamba_layer, ok.parallel_layer
+
+
+def only(W, side, layer=0):
+    """The other side of a parallel mixer contributes nothing: what is left is one mechanism alone."""
+    other = f"l{layer}.mix.{'right' if side == 'left' else 'left'}.out"
+    return dict(W, **{other: torch.zeros_like(W[other])})
+
+
+ALONE = {      # name: (layers, the side of a parallel mixer that counts)
+    "scan": ([SCAN(mlp=None)], None),
+    "scan-no-conv": ([SCAN(conv=1, mlp=None)], None),
+    "scan-two-taps": ([SCAN(conv=2, inner=16, state=16, mlp=None)], None),
+    "scan-five-taps": ([SCAN(conv=5, mlp=None)], None),
+    "scan-one-state-rank-one": ([SCAN(state=1, dt_rank=1, mlp=None)], None),
+    "scan-odd": ([SCAN(inner=21, state=7, dt_rank=5, conv=3, mlp=None)], None),
+    "attention": ([PAR(mlp=None)], "left"),
+    "attention-window-of-one": ([PAR(size=1, mlp=None)], "left"),
+    "attention-window-beyond-prompt": ([PAR(size=1000, mlp=None)], "left"),
+    "attention-every-head-its-own": ([PAR(heads=3, kv_heads=3, dim=5, vdim=9, dims=4, mlp=None)], "left"),
+    "attention-one-kv-head": ([PAR(heads=3, kv_heads=1, dims=2, mlp=None)], "left"),
+    "attention-no-turn": ([PAR(dims=0, mlp=None)], "left"),
+    "attention-no-scaling": ([PAR(mlp=None)], "left"),
+    "recurrence": ([PAR(mlp=None)], "right"),
+    "recurrence-no-conv": ([PAR(conv=1, mlp=None)], "right"),
+    "recurrence-four-taps": ([PAR(conv=4, r_vdim=8, state=8, mlp=None)], "right"),
+    "recurrence-one-group": ([PAR(groups=1, norm_groups=1, mlp=None)], "right"),
+    "recurrence-every-head-its-own": ([PAR(r_heads=3, groups=3, norm_groups=5, mlp=None)], "right"),
+    "recurrence-norm-groups-beside-heads": ([PAR(r_heads=3, groups=1, r_vdim=4, norm_groups=6, mlp=None)], "right"),
+    "parallel": ([PAR(mlp=None)], None),
+    "dense": ([SCAN(mlp=ok.dense_mlp())], None),
+    "moe": ([SCAN()], None),
+    "moe-no-groups": ([SCAN(mlp=MOE(groups=1, keep=1))], None),
+    "moe-all-groups-kept": ([SCAN(mlp=MOE(groups=3, keep=3, top=4))], None),
+    "moe-groups-of-one": ([SCAN(mlp=MOE(groups=6, keep=4, top=2))], None),
+    "moe-whole-group": ([SCAN(mlp=MOE(top=3, groups=2, keep=1))], None),
+    "moe-top-one": ([SCAN(mlp=MOE(top=1, scale=1.0))], None),
+    "moe-no-shared": ([SCAN(mlp=MOE(shared_ff=0))], None),
+    "moe-tight-limits": ([SCAN(mlp=MOE(limit=0.2, shared_limit=0.1))], None),
+}
+
+
+@pytest.mark.parametrize("mech", sorted(ALONE))
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_mechanism_alone(kge, tmp_path, mech, dtype):
+    layers, side = ALONE[mech]
+    cfg = ok.make_config(copy.deepcopy(layers))
+    if mech == "attention-no-scaling":
+        cfg["layers"][0]["mixer"]["left"]["rot"].pop("scaling")
+    W = ok.make_weights(cfg, seed=3)
+    if side:
+        W = only(W, side)
+    c = Case(cfg, W, clear_prompt(cfg, W, 45), dtype)
+    llm = make_engine(kge, tmp_path, cfg, W, dtype)
+    check(run_pieces(llm, 0, c.toks, [45]), c, dtype, mech)
+    check(run_pieces(llm, 1, c.toks, [21, 1, 1, 2, 20]), c, dtype, mech + ", in pieces")
+    llm.close()
+
+
+def full(**kw):
+    """Both kinds of layer with different windows, heads, taps and feed-forwards, one layer without a feed-forward."""
+    layers = [SCAN(mlp=ok.dense_mlp(28)), PAR(), SCAN(inner=36, state=9, dt_rank=2, conv=2, mlp=None),
+              PAR(heads=2, kv_heads=1, dim=6, vdim=10, size=11, scale=0.5, base=30.0, dims=4, original=12, r_heads=6, r_vdim=4, state=10, groups=3, norm_groups=1, conv=4,
+                  mlp=MOE(ff=16, experts=9, top=2, groups=3, keep=2, limit=0.8, scale=0.9)),
+              SCAN(inner=24, state=16, dt_rank=6, conv=3)]
+    return ok.make_config(layers, **dict(dict(width=96), **kw))
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_prefill_decode_and_pieces_agree_with_the_oracle(kge, tmp_path, dtype):
+    cfg = full()
+    W = ok.make_weights(cfg, seed=5)
+    c = Case(cfg, W, clear_prompt(cfg, W, 75), dtype)
+    llm = make_engine(kge, tmp_path, cfg, W, dtype)
+    for rid, pieces in enumerate([[75], [30] + [1] * 45, [1] * 75, [2, 3, 17, 2, 31, 5, 2, 2, 9, 2], [23, 2, 24, 26], [47, 2, 1, 1, 24]]):
+        got = run_pieces(llm, rid, c.toks, pieces)
+        llm.trace_end(rid)
+        check(got, c, dtype, f"pieces {pieces[:6]}")
+    llm.close()
+
+
+def test_layer_outputs_match(kge, tmp_path):
+    """The residual stream after every layer."""
+    cfg = full()
+    W = ok.make_weights(cfg, seed=6)
+    toks = prompt(cfg, 33)
+    _, layers = ok.forward(cfg, W, toks, return_layers=True)
+    llm = make_engine(kge, tmp_path, cfg, W, "float32")
+    L = len(layers)
+    buf = np.zeros((L, 33, cfg["width"]), dtype=np.float32)
+    llm.set_layer_dump(buf)
+    run_pieces(llm, 0, toks, [20, 13])
+    last = buf.reshape(-1)[:L * 13 * cfg["width"]].reshape(L, 13, cfg["width"]).copy()      # the dump is packed per step: [layer, row of the step, width]
+    llm.set_layer_dump(None)
+    llm.close()
+    for i, x in enumerate(layers):      # the dump holds the last step's rows: positions 20 .. 32
+        assert np.abs(last[i] - x.numpy()[20:]).max() < 2e-4 * float(x.abs().max()), f"layer {i}"
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_mixed_batches_of_unequal_requests(kge, tmp_path, dtype):
+    cfg = full()
+    W = ok.make_weights(cfg, seed=7)
+    P = {r: clear_prompt(cfg, W, n, 10 + r) for r, n in enumerate([61, 9, 40, 1])}
+    C = {r: Case(cfg, W, t, dtype) for r, t in P.items()}
+    # each step: (request, number of tokens); prompt pieces beside single tokens, requests pausing and resuming
+    steps = [[(0, 19), (1, 1), (3, 1)], [(1, 1), (2, 2), (0, 2)], [(0, 20), (1, 1)], [(2, 18), (1, 1), (0, 1)], [(1, 5), (2, 1)],
+             [(0, 1), (2, 1)], [(0, 18), (2, 18)]]
+    llm = make_engine(kge, tmp_path, cfg, W, dtype)
+    at = {r: 0 for r in P}
+    got = {r: [] for r in P}
+    for st in steps:
+        entries = []
+        for r, n in st:
+            llm.trace_add(r, P[r][at[r]:at[r] + n])
+            entries.append((r, n, list(range(n))))
+        lg = llm.trace_step(entries)
+        k = 0
+        for r, n in st:
+            got[r].append(lg[k:k + n])
+            k += n
+            at[r] += n
+    llm.close()
+    for r in P:
+        assert at[r] == len(P[r])
+        check(np.concatenate(got[r]), C[r], dtype, f"request {r}")
+
+
+def test_pages_and_slots_are_used_again(kge, tmp_path):
+    """Two state slots and a pool of 96 tokens: five requests pass through, each in pages and a slot that an earlier
+    request filled; each must come out as if it had run alone (a slot's old states or convolution rows, or a page's old keys,
+    must not leak)."""
+    cfg = full()
+    W = ok.make_weights(cfg, seed=8)
+    llm = make_engine(kge, tmp_path, cfg, W, "float32", tokens=96, bs=16, seqs=2)
+    P = {r: prompt(cfg, n, 20 + r) for r, n in enumerate([40, 33, 47, 18, 30])}
+    got = {}
+    got[0] = run_pieces(llm, 0, P[0], [40])
+    llm.trace_add(1, P[1][:20])
+    a = llm.trace_step([(1, 20, list(range(20)))])
+    llm.trace_end(0)
+    llm.trace_add(2, P[2])
+    llm.trace_add(1, P[1][20:])
+    b = llm.trace_step([(2, 30, list(range(30))), (1, 13, list(range(13)))])
+    got[1] = np.concatenate([a, b[30:]])
+    c = llm.trace_step([(2, 17, list(range(17)))])
+    got[2] = np.concatenate([b[:30], c])
+    llm.trace_end(1)
+    got[3] = run_pieces(llm, 3, P[3], [1, 1, 16])
+    llm.trace_end(2)
+    llm.trace_end(3)
+    got[4] = run_pieces(llm, 4, P[4], [29, 1])
+    llm.close()
+    for r in P:
+        check(got[r], Case(cfg, W, P[r], "float32"), "float32", f"request {r}")
+
+
+EDGES = [      # heads, kv heads, dim, vdim, window, page: per-row kernel; mma.sync (equal and unequal sizes); the tcgen05 prompt kernel
+    (4, 2, 6, 5, 21, 16), (4, 1, 16, 8, 37, 16), (6, 2, 48, 80, 64, 32), (6, 3, 64, 128, 45, 64), (4, 2, 64, 64, 70, 64), (6, 2, 128, 128, 33, 16), (8, 8, 64, 64, 66, 64)]
+
+
+@pytest.mark.parametrize("case", EDGES)
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_window_edges_with_peaked_scores(kge, tmp_path, dtype, case):
+    """The attention side alone with a large score scale, so that single keys carry most of a row's weight: a window that is
+    one token off moves the logits far beyond rounding."""
+    heads, kv, dim, vdim, size, bs = case
+    cfg = ok.make_config([PAR(heads=heads, kv_heads=kv, dim=dim, vdim=vdim, size=size, scale=2.5 / dim ** 0.5, base=300.0, original=64, mlp=None)], width=40)
+    W = only(ok.make_weights(cfg, seed=9), "left")
+    c = Case(cfg, W, prompt(cfg, 200, 30), dtype)
+    scale = float(np.sqrt((c.want ** 2).mean()))
+    for delta in (1, -1):
+        other = copy.deepcopy(cfg)
+        other["layers"][0]["mixer"]["left"]["mask"]["size"] += delta
+        diff = np.sqrt(((ok.forward(other, W, c.toks).numpy() - c.want) ** 2).mean(-1))[size + 2:] / scale
+        assert float((diff > 0.02).mean()) > 0.05 and float(diff.max()) > 0.1, f"a window of {delta:+d} does not show"
+    llm = make_engine(kge, tmp_path, cfg, W, dtype, bs=bs)
+    check(run_pieces(llm, 0, c.toks, [200]), c, dtype, "whole")
+    llm.trace_end(0)
+    check(run_pieces(llm, 1, c.toks[:100], [15, 1, 1, 1, 14, 2, 30, 1, 1, 34]), c, dtype, "pieces and single tokens across page borders", slice(0, 100))
+    llm.trace_end(1)
+    check(run_pieces(llm, 2, c.toks, [size - 2] + [1] * (200 - size + 2)), c, dtype, "decoding while the window comes into play")
+    llm.close()
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_one_standing_key_until_it_leaves_the_window(kge, tmp_path, dtype):
+    """A token at a page's last row that moves every row that sees it, far back in the window, and none after that (the layer
+    below it is left out, so only the attention carries anything over)."""
+    cfg = ok.make_config([PAR(heads=3, kv_heads=1, dim=32, vdim=32, size=90, scale=0.35, original=64, mlp=None)], width=40)
+    W = only(ok.make_weights(cfg, seed=16), "left")
+    c = Case(cfg, W, prompt(cfg, 170, 33), dtype)
+    moved = ok.forward(cfg, W, c.toks[:63] + [(c.toks[63] + 1) % cfg["vocab"]] + c.toks[64:]).numpy()
+    assert float(np.abs(moved - c.want)[120:153].max()) > 0.02 and float(np.abs(moved - c.want)[63 + 90:].max()) < 1e-9
+    llm = make_engine(kge, tmp_path, cfg, W, dtype, bs=64)
+    check(run_pieces(llm, 0, c.toks, [170]), c, dtype, "whole")
+    llm.trace_end(0)
+    check(run_pieces(llm, 1, c.toks, [63, 1, 2, 60, 3] + [1] * 41), c, dtype, "pieces, then decoding")
+    llm.close()
+
+
+def test_rotary_frequencies_in_every_band(kge, tmp_path):
+    """Wavelengths below, between and above the two bounds, factors below and above 1, and a turn of part of the head, at
+    positions where a wrong frequency shows."""
+    for kw in (dict(dim=24, dims=24, base=5000.0, original=200, factor=8.0, low=1.0, high=4.0), dict(dim=16, dims=10, base=900.0, original=60, factor=0.5, low=2.0, high=9.0),
+               dict(dim=12, dims=12, base=100.0, original=30, factor=3.0, low=1.5, high=2.5)):
+        cfg = ok.make_config([PAR(heads=2, kv_heads=2, vdim=8, size=64, scale=1.0 / kw["dim"] ** 0.5, mlp=None, **kw)], width=32)
+        rot = cfg["layers"][0]["mixer"]["left"]["rot"]
+        plain = [kw["base"] ** (-2.0 * i / kw["dims"]) for i in range(kw["dims"] // 2)]
+        ratio = [f / p for f, p in zip(ok.frequencies(rot), plain)]
+        lo, hi = min(1.0, 1.0 / kw["factor"]), max(1.0, 1.0 / kw["factor"])
+        assert any(r == 1.0 for r in ratio) and any(abs(r * kw["factor"] - 1.0) < 1e-12 for r in ratio) and any(lo + 1e-3 < r < hi - 1e-3 for r in ratio)
+        W = only(ok.make_weights(cfg, seed=18), "left")
+        c = Case(cfg, W, prompt(cfg, 150, 34), "float32")
+        llm = make_engine(kge, tmp_path, cfg, W, "float32", name=f"m{kw['dim']}")
+        check(run_pieces(llm, 0, c.toks, [149, 1]), c, "float32", str(kw))
+        llm.close()
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("mixer", ["scan", "recurrence", "recurrence-chunks"])
+def test_states_that_decay_slowly(kge, tmp_path, dtype, mixer):
+    """Decays close to 1 beside fast ones: the state remembers the first tokens for hundreds of positions, so a state that is
+    lost, reset or carried over at the cut of a prompt shows at the end."""
+    if mixer == "scan":
+        cfg = ok.make_config([SCAN(inner=24, state=16, dt_rank=4, conv=3, mlp=None)], width=32)
+        W = ok.make_weights(cfg, seed=10)
+        W["l0.mix.A_log"] = torch.where(torch.arange(16) % 5 == 0, 0.5, -6.0).expand(24, 16).to(ok.DT).clone()
+        W["l0.mix.o"] = W["l0.mix.o"] * 0.03125      # the state grows: keep the stream where Dynamic Tanh still bends
+    else:
+        z = dict(r_heads=3, r_vdim=8, state=16, groups=1, norm_groups=1) if mixer == "recurrence-chunks" else dict(r_heads=3, r_vdim=5, state=7, groups=1, norm_groups=1)
+        cfg = ok.make_config([PAR(mlp=None, **z)], width=32)
+        W = only(ok.make_weights(cfg, seed=10), "right")
+        W["l0.mix.right.A_log"] = torch.tensor([-6.5, 1.0, -6.0], dtype=ok.DT)
+    toks = [3] * 8 + [5, 9, 11, 2] * 63
+    c = Case(cfg, W, toks, dtype)
+    other = ok.forward(cfg, W, [20, 41, 33, 60, 17, 8, 29, 71] + toks[8:]).numpy()
+    assert float(np.abs(other[-20:] - c.want[-20:]).max()) > 0.02      # the first tokens still matter 250 positions later
+    llm = make_engine(kge, tmp_path, cfg, W, dtype)
+    check(run_pieces(llm, 0, toks, [260]), c, dtype, "whole")
+    llm.trace_end(0)
+    check(run_pieces(llm, 1, toks, [63, 2, 1, 64, 2, 97, 1, 30]), c, dtype, "pieces")
+    llm.trace_end(1)
+    check(run_pieces(llm, 2, toks, [200] + [1] * 60), c, dtype, "decoding")
+    llm.close()
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_steps_of_very_different_sizes(kge, tmp_path, dtype):
+    """Step sizes from nearly 0 to dozens side by side: log decays of a chunk add up to thousands while neighbours differ by
+    little, and nothing may overflow or drown."""
+    cfg = ok.make_config([PAR(r_heads=4, r_vdim=16, state=16, groups=2, norm_groups=2, mlp=None), SCAN(inner=32, state=16, dt_rank=8, mlp=None)], width=48)
+    W = only(ok.make_weights(cfg, seed=19), "right")
+    W["l0.mix.right.in"][-4:] *= 16.0
+    W["l0.mix.right.A_log"] = torch.tensor([1.5, -3.0, 3.0, 0.0], dtype=ok.DT)
+    W["l1.mix.dt"] = W["l1.mix.dt"] * 8.0
+    c = Case(cfg, W, prompt(cfg, 150, 41), dtype)
+    P = ok.sub(W, "l0.mix.right.")
+    h = ok.dyt(W["embed"][torch.tensor(c.toks)] * 3.0, W, "l0.norm1")
+    la = torch.exp(P["A_log"]) * ok.softplus(h @ P["in"][-4:].T + P["dt_bias"])
+    assert float(la[:64].sum(0).max()) > 1000.0 and float(la.min()) < 1e-3
+    llm = make_engine(kge, tmp_path, cfg, W, dtype)
+    check(run_pieces(llm, 0, c.toks, [150]), c, dtype, "whole")
+    check(run_pieces(llm, 1, c.toks, [66, 2, 1, 1, 63, 17]), c, dtype, "pieces")
+    llm.close()
+
+
+def test_convolution_rows_cross_every_cut(kge, tmp_path):
+    """The projected rows before a step's first one come from the slot, also when the steps before brought one or two tokens
+    only, in steps with and without other requests."""
+    cfg = ok.make_config([SCAN(conv=4, mlp=None), PAR(conv=5, mlp=None), SCAN(conv=2, inner=28, mlp=None)])
+    W = ok.make_weights(cfg, seed=22)
+    c = Case(cfg, W, prompt(cfg, 40, 36), "float32")
+    llm = make_engine(kge, tmp_path, cfg, W, "float32")
+    for rid, pieces in enumerate([[1, 1, 2, 1, 3, 2, 30], [2, 1, 1, 1, 1, 34], [5, 1, 2, 32]]):
+        check(run_pieces(llm, rid, c.toks, pieces), c, "float32", f"pieces {pieces}")
+        llm.trace_end(rid)
+    # two requests side by side: one decodes while the other brings pieces
+    d = Case(cfg, W, prompt(cfg, 20, 37), "float32")
+    got, at = [], 0
+    for n, k in [(1, 3), (1, 1), (2, 1), (1, 5), (15, 1)]:
+        llm.trace_add(7, d.toks[at:at + n])
+        llm.trace_add(8, c.toks[:k])
+        got.append(llm.trace_step([(8, k, []), (7, n, list(range(n)))]))
+        at += n
+    llm.close()
+    check(np.concatenate(got), d, "float32", "beside another request")
+
+
+def test_router_choices_with_corrections_of_both_signs(kge, tmp_path):
+    """Corrections large enough to change most choices, some rows with only negative choice scores, group counts that are
+    no powers of two, more router outputs than lanes in a warp, and groups whose best expert is not in the best group."""
+    for experts, groups, keep, top in [(45, 9, 3, 7), (9, 3, 2, 4), (4, 1, 1, 2), (64, 4, 2, 11), (10, 5, 2, 3)]:
+        cfg = ok.make_config([SCAN(mlp=MOE(ff=5, experts=experts, top=top, groups=groups, keep=keep))], width=20)
+        W = ok.make_weights(cfg, seed=31)
+        W["l0.mlp.correction"] = (torch.randn(experts, generator=torch.Generator().manual_seed(1)) * 0.7 - 0.9).to(torch.bfloat16).to(ok.DT)
+        c = Case(cfg, W, prompt(cfg, 50, 38), "float32")
+        plain = dict(W, **{"l0.mlp.correction": torch.zeros(experts, dtype=ok.DT)})
+        assert float(np.abs(ok.forward(cfg, plain, c.toks).numpy() - c.want).max()) > 0.05
+        if 1 < keep < groups:      # judged by the best expert alone, other groups would stay
+            two = ok.group_scores
+            ok.group_scores = lambda s, G: s.reshape(s.shape[0], G, -1).max(-1).values
+            try:
+                assert float(np.abs(ok.forward(cfg, W, c.toks).numpy() - c.want).max()) > 0.05
+            finally:
+                ok.group_scores = two
+        llm = make_engine(kge, tmp_path, cfg, W, "float32", name=f"m{experts}")
+        check(run_pieces(llm, 0, c.toks, [30, 1, 19]), c, "float32", f"{experts} router outputs")
+        llm.close()
+
+
+def test_dynamic_tanh_bends_and_shifts(kge, tmp_path):
+    """Scalars from nearly linear to saturated (also negative), large shifts, and a stream scale that makes them matter."""
+    cfg = ok.make_config([SCAN(mlp=ok.dense_mlp()), PAR()], scale=7.5)
+    W = ok.make_weights(cfg, seed=33)
+    for name, a in (("l0.norm1", 0.02), ("l0.norm2", 3.0), ("l1.norm1", -0.75), ("l1.norm2", 0.125), ("final.norm", 1.5)):
+        W[name + ".alpha"] = torch.tensor(a, dtype=torch.float32).to(torch.bfloat16).to(ok.DT)
+        W[name + ".b"] = W[name + ".b"] * 4.0
+    c = Case(cfg, W, prompt(cfg, 40, 42), "float32")
+    llm = make_engine(kge, tmp_path, cfg, W, "float32")
+    check(run_pieces(llm, 0, c.toks, [30, 1, 9]), c, "float32")
+    llm.close()
+
+
+def big():
+    """Sizes the tensor-core paths take: 16-byte rows everywhere, 64- and 128-wide heads (the tcgen05 prompt kernel) or
+    unequal ones (mma.sync), recurrent heads for the chunked products, experts for the grouped GEMMs."""
+    moe = MOE(ff=64, experts=8, top=3, groups=2, keep=1, shared_ff=64)
+    return [PAR(heads=4, kv_heads=2, dim=64, vdim=64, size=70, scale=0.13, base=1000.0, original=256, r_heads=4, r_vdim=64, state=128, groups=2, norm_groups=4, conv=4, mlp=moe),
+            SCAN(inner=160, state=16, dt_rank=16, conv=4, mlp=moe),
+            PAR(heads=2, kv_heads=1, dim=128, vdim=128, size=129, scale=0.1, base=1000.0, original=256, r_heads=6, r_vdim=40, state=64, groups=1, norm_groups=1, conv=3, mlp=ok.dense_mlp(96)),
+            SCAN(inner=96, state=32, dt_rank=8, conv=2, mlp=None)]
+
+
+def run_mixed(kge, tmp_path, cfg, W, n=290, tokens=1024, bs=64):
+    """Whole, pieces then decoding, two decode rows of unequal contexts, a single token beside a prompt piece."""
+    c = Case(cfg, W, clear_prompt(cfg, W, n, 32))
+    llm = make_engine(kge, tmp_path, cfg, W, "bfloat16", bs=bs, tokens=tokens)
+    check(run_pieces(llm, 0, c.toks, [n]), c, "bfloat16", "whole")
+    llm.trace_end(0)
+    check(run_pieces(llm, 1, c.toks, [150, 3, 45, 2, n - 230] + [1] * 30), c, "bfloat16", "pieces, then decoding")
+    llm.trace_end(1)
+    a, b = Case(cfg, W, clear_prompt(cfg, W, 150, 35)), Case(cfg, W, clear_prompt(cfg, W, 9, 36))
+    llm.trace_add(2, a.toks[:140])
+    llm.trace_add(3, b.toks[:3])
+    llm.trace_step([(2, 140, []), (3, 3, [])])
+    ga, gb = [], []
+    for i in range(6):
+        llm.trace_add(2, a.toks[140 + i:141 + i])
+        llm.trace_add(3, b.toks[3 + i:4 + i])
+        lg = llm.trace_step([(2, 1, [0]), (3, 1, [0])])
+        ga.append(lg[0])
+        gb.append(lg[1])
+    d = Case(cfg, W, clear_prompt(cfg, W, 200, 37))
+    llm.trace_end(3)
+    llm.trace_add(4, d.toks[:131])
+    llm.trace_step([(4, 131, [])])
+    llm.trace_add(2, a.toks[146:147])
+    llm.trace_add(4, d.toks[131:])
+    lg = llm.trace_step([(2, 1, [0]), (4, 69, list(range(69)))])
+    llm.trace_add(2, a.toks[147:148])
+    llm.trace_add(5, b.toks)
+    l2 = llm.trace_step([(5, 9, list(range(9))), (2, 1, [0])])      # the single token after the piece
+    llm.close()
+    check(np.stack(ga), a, "bfloat16", "long request of a decode batch", slice(140, 146))
+    check(np.stack(gb), b, "bfloat16", "short request of a decode batch", slice(3, 9))
+    check(lg[:1], a, "bfloat16", "a single token beside a prompt piece", slice(146, 147))
+    check(lg[1:], d, "bfloat16", "a prompt piece that starts inside a page beside a single token", slice(131, 200))
+    check(l2[:9], b, "bfloat16", "a short prompt before a single token")
+    check(l2[9:], a, "bfloat16", "a single token after a prompt", slice(147, 148))
+
+
+def test_tensor_core_sizes(kge, tmp_path):
+    cfg = ok.make_config(big(), width=64, vocab=96)
+    W = ok.make_weights(cfg, seed=15)
+    run_mixed(kge, tmp_path, cfg, W)
+
+
+SSD_SIZES = [      # heads, groups, vdim, state, taps: the chunked products (padded states and columns, several column tiles, states of up to 128), the plain kernel
+    (4, 1, 64, 128, 4), (3, 1, 40, 16, 3), (2, 2, 128, 64, 2), (4, 2, 72, 104, 4), (2, 1, 200, 8, 1), (6, 3, 24, 48, 3), (5, 1, 7, 9, 4), (2, 1, 16, 160, 3), (2, 2, 12, 256, 2), (3, 3, 8, 33, 5), (1, 1, 8, 1, 2)]
+
+
+@pytest.mark.parametrize("shape", SSD_SIZES)
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_recurrent_head_sizes(kge, tmp_path, dtype, shape):
+    heads, groups, vdim, state, conv = shape
+    cfg = ok.make_config([PAR(heads=1, kv_heads=1, r_heads=heads, groups=groups, r_vdim=vdim, state=state, norm_groups=heads, conv=conv, mlp=None)], width=48)
+    W = only(ok.make_weights(cfg, seed=25), "right")
+    c = Case(cfg, W, prompt(cfg, 210, 39), dtype)
+    llm = make_engine(kge, tmp_path, cfg, W, dtype)
+    check(run_pieces(llm, 0, c.toks, [210]), c, dtype, "whole")
+    llm.trace_end(0)
+    check(run_pieces(llm, 1, c.toks, [64, 2, 62, 1, 1, 65, 1, 14]), c, dtype, "pieces")
+    llm.trace_end(1)
+    # two pieces and a single token in one step
+    a, b = Case(cfg, W, prompt(cfg, 100, 43), dtype), Case(cfg, W, prompt(cfg, 9, 44), dtype)
+    llm.trace_add(2, b.toks[:8])
+    llm.trace_step([(2, 8, [])])
+    llm.trace_add(2, b.toks[8:])
+    llm.trace_add(3, a.toks)
+    llm.trace_add(4, c.toks[:70])
+    lg = llm.trace_step([(2, 1, [0]), (3, 100, list(range(100))), (4, 70, list(range(70)))])
+    llm.close()
+    check(lg[:1], b, dtype, "a single token beside pieces", slice(8, 9))
+    check(lg[1:101], a, dtype, "a piece beside others")
+    check(lg[101:], c, dtype, "another piece", slice(0, 70))
+
+
+SCAN_SIZES = [(40, 16, 8, 4), (33, 24, 12, 3), (64, 4, 1, 2), (17, 48, 3, 4), (32, 64, 16, 4), (20, 100, 4, 3), (24, 128, 8, 2), (9, 200, 2, 1), (12, 256, 5, 3), (48, 8, 24, 5)]      # channels, state, rank, taps
+
+
+@pytest.mark.parametrize("shape", SCAN_SIZES)
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_scan_sizes(kge, tmp_path, dtype, shape):
+    inner, state, rank, conv = shape
+    cfg = ok.make_config([SCAN(inner=inner, state=state, dt_rank=rank, conv=conv, mlp=None)], width=48)
+    W = ok.make_weights(cfg, seed=27)
+    c = Case(cfg, W, prompt(cfg, 70, 45), dtype)
+    llm = make_engine(kge, tmp_path, cfg, W, dtype, seqs=20, tokens=2048)
+    check(run_pieces(llm, 0, c.toks, [70]), c, dtype, "whole")
+    check(run_pieces(llm, 1, c.toks, [7, 2, 1, 8, 9, 16, 1, 1, 25]), c, dtype, "pieces")
+    # many requests that decode side by side, at different positions
+    for r in range(2, 19):
+        llm.trace_add(r, c.toks[:r])
+    llm.trace_step([(r, r, []) for r in range(2, 19)])
+    for r in range(2, 19):
+        llm.trace_add(r, c.toks[r:r + 1])
+    lg = llm.trace_step([(r, 1, [0]) for r in range(2, 19)])
+    llm.close()
+    check(lg, c, dtype, "decoding side by side", slice(2, 19))
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("tokens", [40, 300])
+@pytest.mark.parametrize("shared", [0, 64])
+def test_experts_of_few_and_many_rows(kge, tmp_path, dtype, tokens, shared):
+    """Routed rows below and above what the grouped tensor-core GEMMs and the router's matrix product take, decode rows after them."""
+    cfg = ok.make_config([SCAN(mlp=MOE(ff=128, experts=12, top=4, groups=3, keep=2, shared_ff=shared))], width=128)
+    W = ok.make_weights(cfg, seed=26)
+    c = Case(cfg, W, clear_prompt(cfg, W, tokens, 40), dtype)
+    llm = make_engine(kge, tmp_path, cfg, W, dtype, bs=64)
+    check(run_pieces(llm, 0, c.toks, [tokens]), c, dtype, "whole")
+    llm.trace_end(0)
+    check(run_pieces(llm, 1, c.toks, [tokens - 4, 1, 1, 2]), c, dtype, "pieces")
+    llm.close()
+
+
+def test_first_tokens(kge, tmp_path):
+    cfg = full()
+    W = ok.make_weights(cfg, seed=11)
+    llm = make_engine(kge, tmp_path, cfg, W, "float32")
+    for rid, n in enumerate([1, 2, 3, 5]):
+        c = Case(cfg, W, prompt(cfg, n, 40 + n), "float32")
+        got = run_pieces(llm, rid, c.toks, [n])
+        llm.trace_end(rid)
+        check(got, c, "float32", f"{n} tokens")
+    llm.close()
+
+
+def test_long_decoding(kge, tmp_path):
+    cfg = full()
+    W = ok.make_weights(cfg, seed=12)
+    c = Case(cfg, W, prompt(cfg, 200, 50), "float32")
+    llm = make_engine(kge, tmp_path, cfg, W, "float32")
+    got = run_pieces(llm, 0, c.toks, [4] + [1] * 196)
+    llm.close()
+    check(got, c, "float32")
+
+
+OTHER = [
+    # nothing is 16-byte aligned; only parallel layers
+    dict(layers=[PAR(heads=3, kv_heads=1, dim=5, vdim=7, dims=2, size=6, r_heads=3, r_vdim=3, state=5, groups=1, norm_groups=9, conv=3, mlp=MOE(ff=7, experts=5, top=2, groups=5, keep=3)),
+                 PAR(heads=1, kv_heads=1, dim=11, vdim=3, dims=10, size=17, r_heads=1, r_vdim=1, state=1, groups=1, norm_groups=1, conv=1, mlp=None)], vocab=53, width=22, eps=1e-3, scale=1.0),
+    # only scans; five taps; one channel more than a block holds
+    dict(layers=[SCAN(inner=17, state=3, dt_rank=7, conv=5, mlp=MOE(ff=9, experts=4, top=1, groups=2, keep=2)), SCAN(inner=10, state=10, dt_rank=10, conv=1, mlp=ok.dense_mlp(5))], vocab=67, width=42, scale=0.5),
+    # equal sizes everywhere
+    dict(layers=[PAR(heads=8, kv_heads=8, dim=8, vdim=8, size=8, r_heads=8, r_vdim=8, state=8, groups=8, norm_groups=8, conv=8, mlp=MOE(ff=8, experts=8, top=8, groups=8, keep=8, shared_ff=8)),
+                 SCAN(inner=8, state=8, dt_rank=8, conv=8, mlp=ok.dense_mlp(8))], vocab=80, width=8),
+    # wide values, a channel count far from the width
+    dict(layers=[PAR(heads=2, kv_heads=2, dim=16, vdim=136, size=12, r_heads=2, r_vdim=136, state=12, groups=2, norm_groups=4, conv=2, mlp=MOE(ff=32, groups=1, keep=1)),
+                 SCAN(inner=200, state=2, dt_rank=1, mlp=MOE(ff=32, experts=16, groups=4, keep=2, top=5))], vocab=90, width=48),
+]
+
+
+@pytest.mark.parametrize("sizes", OTHER)
+def test_other_sizes(kge, tmp_path, sizes):
+    cfg = ok.make_config(**copy.deepcopy(sizes))
+    W = ok.make_weights(cfg, seed=13)
+    c = Case(cfg, W, clear_prompt(cfg, W, 50, 60))
+    for dtype in ("float32", "bfloat16"):        # the same sizes through the 16-bit kernels and their fallbacks
+        llm = make_engine(kge, tmp_path, cfg, W, dtype, name=dtype)
+        check(run_pieces(llm, 0, c.toks, [50]), c, dtype, "whole, " + dtype)
+        check(run_pieces(llm, 1, c.toks, [13, 2, 1, 1, 1, 32]), c, dtype, "pieces, " + dtype)
+        llm.close()
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("model", ["small", "big"])
+def test_greedy_generation_through_the_scheduler(kge, tmp_path, dtype, model):
+    """LLM.generate: the continuous-batching scheduler cuts the prompts into 16-token steps, admits the third request
+    when a slot frees up, samples greedily, and replays its decode steps as a CUDA graph while windows pass over the
+    decoded tokens."""
+    cfg = full() if model == "small" else ok.make_config(big(), width=64, vocab=96)
+    W = ok.make_weights(cfg, seed=14)
+    prompts = [clear_prompt(cfg, W, n, 70 + n) for n in (37, 5, 21)]
+    llm = make_engine(kge, tmp_path, cfg, W, dtype, seqs=2, batched=16)
+    outs = llm.generate(prompts, kge.SamplingParams(max_tokens=14, temperature=0.0, ignore_eos=True))
+    assert llm.kernel_launches > 0
+    llm.close()
+    compared = 0
+    for p, o in zip(prompts, outs):
+        got = o.outputs[0].token_ids
+        assert len(got) == 14
+        mg = []
+        lg = ok.forward(cfg, W, list(p) + list(got), margins=mg)[len(p) - 1:-1]      # teacher-forced: a different choice must be a near-tie of the oracle
+        close = torch.stack(mg).min(0).values[len(p) - 1:-1] < CLEAR
+        for k, g in enumerate(got):
+            if dtype != "float32" and bool(close[k]):      # from here on another expert may have been chosen
+                break
+            compared += 1
+            best = int(torch.argmax(lg[k]))
+            if g != best:      # the samplers read 16-bit logits rows: two logits within their spacing tie
+                gap = float(lg[k][best] - lg[k][g])
+                assert gap < (2.0 ** -7 * max(1.0, float(lg[k][best].abs())) if dtype == "float32" else 0.15), f"token {k}: chose {g}, oracle {best} leads by {gap}"
+    assert compared >= (42 if dtype == "float32" else 6)
+
+
+def test_trace_runner_command_line(kge, tmp_path):
+    """bin/trace_run end to end on this design: pieces of two requests side by side, a request that ends and one that
+    takes its pages and slot, both number formats."""
+    import json
+    import os
+    import subprocess
+    import sys
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    cfg = full()
+    W = ok.make_weights(cfg, seed=17)
+    d = str(tmp_path / "m")
+    ok.save_model_dir(d, cfg, W)
+    P = {"a": clear_prompt(cfg, W, 50, 80), "b": clear_prompt(cfg, W, 31, 81), "c": clear_prompt(cfg, W, 40, 82)}
+    C = {k: Case(cfg, W, v) for k, v in P.items()}
+    steps = [
+        {"step": 0, "entries": [{"id": "a", "tokens": P["a"][:30], "want": [0, 29]}, {"id": "b", "tokens": P["b"][:2], "want": []}], "end": []},
+        {"step": 1, "entries": [{"id": "b", "tokens": P["b"][2:], "want": [0, 28]}, {"id": "a", "tokens": P["a"][30:31], "want": [0]}], "end": ["b"]},
+        {"step": 2, "entries": [{"id": "a", "tokens": P["a"][31:], "want": [18]}, {"id": "c", "tokens": P["c"], "want": [39, 5]}], "end": ["a", "c"]},
+    ]
+    rows = {0: [("a", 0), ("a", 29)], 1: [("b", 2), ("b", 30), ("a", 30)], 2: [("a", 49), ("c", 39), ("c", 5)]}
+    for dtype in ("float32", "bfloat16"):
+        out = str(tmp_path / ("out_" + dtype))
+        r = subprocess.run([sys.executable, os.path.join(root, "bin", "trace_run"), "--model", d, "--dtype", dtype, "--out", out, "--max-tokens", "128"],
+                           input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True, timeout=600)
+        assert r.returncode == 0, r.stderr[-2000:]
+        assert [l for l in r.stdout.splitlines() if l.startswith("done")] == ["done 0", "done 1", "done 2"]
+        for st, rr in rows.items():
+            got = np.fromfile(os.path.join(out, f"{st}.f32"), dtype="<f4").reshape(len(rr), cfg["vocab"])
+            for g, (k, i) in zip(got, rr):
+                check(g[None], C[k], dtype, f"step {st}, request {k}", slice(i, i + 1))
+
+
+def test_server_command_line_and_sampling(kge, tmp_path):
+    """`vllm serve DIR` picks the design from config.json: greedy completions over HTTP (token-id prompts) equal the
+    in-process engine's, in bfloat16 and with --dtype float32; sampling with a temperature and a seed is reproducible and
+    stays inside the vocabulary."""
+    import json
+    import os
+    import socket
+    import subprocess
+    import time
+    import urllib.request
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    binary = os.path.join(root, "kubernetes-gpu-cluster_b200", "bin", "vllm")
+    assert os.path.exists(binary), "build the server: make -C kubernetes-gpu-cluster_b200"
+    cfg = full()
+    W = ok.make_weights(cfg, seed=19)
+    d = str(tmp_path / "m")
+    ok.save_model_dir(d, cfg, W)
+    prompts = [prompt(cfg, n, 100 + n) for n in (23, 4, 40)]
+    for dtype in ("bfloat16", "float32"):
+        llm = kge.LLM(d, dtype=dtype, max_model_len=128, max_num_seqs=4, max_num_batched_tokens=32, num_gpu_blocks_override=16, enable_prefix_caching=False)
+        ref = [o.outputs[0].token_ids for o in llm.generate(prompts, kge.SamplingParams(max_tokens=8, temperature=0.0, ignore_eos=True))]
+        warm = [o.outputs[0].token_ids for o in llm.generate(prompts[:1], kge.SamplingParams(max_tokens=8, temperature=0.8, top_k=20, seed=7, ignore_eos=True))]
+        again = [o.outputs[0].token_ids for o in llm.generate(prompts[:1], kge.SamplingParams(max_tokens=8, temperature=0.8, top_k=20, seed=7, ignore_eos=True))]
+        llm.close()
+        assert warm == again and all(0 <= t < cfg["vocab"] for t in warm[0])
+        s = socket.socket()
+        s.bind(("127.0.0.1", 0))
+        port = s.getsockname()[1]
+        s.close()
+        proc = subprocess.Popen([binary, "serve", d, "--host", "127.0.0.1", "--port", str(port), "--dtype", dtype, "--max-model-len", "128", "--max-num-seqs", "4",
+                                 "--max-num-batched-tokens", "32", "--num-gpu-blocks-override", "16", "--served-model-name", "z", "--trust-remote-code"],
+                                stdout=subprocess.PIPE, stderr=subprocess.PIPE, text=True)
+        try:
+            t0 = time.time()
+            while True:
+                try:
+                    with urllib.request.urlopen(f"http://127.0.0.1:{port}/health", timeout=2) as r:
+                        if r.status == 200:
+                            break
+                except Exception:
+                    pass
+                assert proc.poll() is None, proc.stderr.read()[-2000:]
+                assert time.time() - t0 < 120, "server did not come up"
+                time.sleep(0.2)
+            req = urllib.request.Request(f"http://127.0.0.1:{port}/v1/completions", headers={"Content-Type": "application/json"},
+                                         data=json.dumps({"model": "z", "prompt": prompts, "max_tokens": 8, "temperature": 0, "ignore_eos": True}).encode())
+            with urllib.request.urlopen(req, timeout=60) as r:
+                body = json.loads(r.read().decode())
+            assert [c["token_ids"] for c in body["choices"]] == ref, dtype
+        finally:
+            proc.terminate()
+            try:
+                proc.wait(timeout=20)
+            except subprocess.TimeoutExpired:
+                proc.kill()
