@@ -10,6 +10,7 @@
 //     stage's "full" barrier, read the swizzled tile with ldmatrix and release the stage with one arrive per warp.
 //     (The cp.async version spent 42 % of its issue slots, mostly on per-16-byte address generation, and reached
 //     84 % of HBM peak; profiles/r01_ncu_summary.md.)
+//   - A sliding window cuts the range of tiles at its lower end (masking what lies before it in the first one).
 //   - The split-KV partials of a (request, kv head) are merged by whichever of its CTAs finishes LAST (arrival counter
 //     after __threadfence), in split order - the same sums as attn_merge_kernel, without a second launch.
 // Keys past the end of a sequence: the producer always fetches whole tiles; block-table entries past the table are read
@@ -108,7 +109,7 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
                        bf16* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml,
                        const bf16* __restrict__ q, int q_stride, const int32_t* __restrict__ block_table, int max_blocks,
                        const int32_t* __restrict__ seq_lens, const int32_t* __restrict__ qsl, int H, int KV, int bs_shift,
-                       float scale_log2, float cap_in2, float cap_log2, const float* __restrict__ sinks) {
+                       float scale_log2, float cap_in2, float cap_log2, const float* __restrict__ sinks, int window) {
   constexpr int CH = HD / 8;
   constexpr uint32_t TILE = BN * HD * 2;                  // one K or V tile
   constexpr uint32_t Q_BYTES = 16 * HD * 2;
@@ -139,9 +140,11 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
   pdl_launch_dependents();
   pdl_wait();                                   // q, the KV rows of this step and the metadata come from earlier kernels
   const int kv_len = seq_lens[b];
+  // a sliding window (> 0) leaves the request's last `window` keys: the splits share the tiles from the one that holds the first of them
+  const int k_lo = window > 0 ? max(kv_len - window, 0) : 0, tile0 = k_lo / BN;
   const int ntiles_all = (kv_len + BN - 1) / BN;
-  const int tps = (ntiles_all + nsplit - 1) / nsplit;
-  const int t_begin = split * tps, t_end = min(ntiles_all, t_begin + tps);
+  const int tps = (ntiles_all - tile0 + nsplit - 1) / nsplit;
+  const int t_begin = tile0 + split * tps, t_end = min(ntiles_all, t_begin + tps);
   const int qrow = qsl[b];
   if (warp < 4) {
     // the Q tile arrives while the producer warp already has the first K/V tiles in flight
@@ -224,10 +227,10 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_co
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         const int k0 = key_base + j * 8;
-        s[j][0] = (k0 < kv_len) ? score_log2(s[j][0], scale_log2, cap_in2, cap_log2) : -INFINITY;
-        s[j][1] = (k0 + 1 < kv_len) ? score_log2(s[j][1], scale_log2, cap_in2, cap_log2) : -INFINITY;
-        s[j][2] = (k0 < kv_len) ? score_log2(s[j][2], scale_log2, cap_in2, cap_log2) : -INFINITY;
-        s[j][3] = (k0 + 1 < kv_len) ? score_log2(s[j][3], scale_log2, cap_in2, cap_log2) : -INFINITY;
+        s[j][0] = (k0 < kv_len && k0 >= k_lo) ? score_log2(s[j][0], scale_log2, cap_in2, cap_log2) : -INFINITY;
+        s[j][1] = (k0 + 1 < kv_len && k0 + 1 >= k_lo) ? score_log2(s[j][1], scale_log2, cap_in2, cap_log2) : -INFINITY;
+        s[j][2] = (k0 < kv_len && k0 >= k_lo) ? score_log2(s[j][2], scale_log2, cap_in2, cap_log2) : -INFINITY;
+        s[j][3] = (k0 + 1 < kv_len && k0 + 1 >= k_lo) ? score_log2(s[j][3], scale_log2, cap_in2, cap_log2) : -INFINITY;
         mx0 = fmaxf(mx0, fmaxf(s[j][0], s[j][1]));
         mx1 = fmaxf(mx1, fmaxf(s[j][2], s[j][3]));
       }
@@ -699,7 +702,7 @@ template <int HD>
 static int launch_decode_tma(bf16* out, const bf16* q, int q_stride, const bf16* kc, const bf16* vc, const int32_t* bt, int max_blocks,
                              const int32_t* sl, const int32_t* qsl, int B, int H, int KV, int bs, int ns, float scale_log2,
                              float* part_o, float* part_ml, void* ws, int64_t ws_bytes, int max_seq_len, float cap_in2, float cap_log2,
-                             const float* sinks, cudaStream_t st) {
+                             const float* sinks, cudaStream_t st, int window = 0) {
   int bs_shift = 0;
   while ((1 << bs_shift) < bs) ++bs_shift;
   CUtensorMap tk, tv;
@@ -709,7 +712,7 @@ static int launch_decode_tma(bf16* out, const bf16* q, int q_stride, const bf16*
   if (int rc = make_tmap(&tk, kc, rows, HD, box_rows)) return rc;
   if (int rc = make_tmap(&tv, vc, rows, HD, box_rows)) return rc;
   // persistent variant (knob attn_persistent): needs partial slots for the segments of a group in the caller's workspace
-  if (tunable(TUN_ATTN_PERSISTENT) && ws && B <= 192) {
+  if (tunable(TUN_ATTN_PERSISTENT) && ws && B <= 192 && window == 0) {
     int64_t slots = ws_bytes / ((int64_t)B * H * (HD + 2) * 4);
     if (slots > 32) slots = 32;
     if (slots >= 3) {
@@ -741,7 +744,7 @@ static int launch_decode_tma(bf16* out, const bf16* q, int q_stride, const bf16*
   auto kern = adt::attn_decode_tma_kernel<HD>;
   KGE_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, adt::smem_bytes<HD>()));
   KGE_CUDA_OK(launch_pdl(kern, dim3(ns, KV, B), dim3(160), adt::smem_bytes<HD>(), st, tk, tv, out, part_o, part_ml, q, q_stride, bt,
-                         max_blocks, sl, qsl, H, KV, bs_shift, scale_log2, cap_in2, cap_log2, sinks));
+                         max_blocks, sl, qsl, H, KV, bs_shift, scale_log2, cap_in2, cap_log2, sinks, window));
   return 0;
 }
 
@@ -756,6 +759,26 @@ int paged_attn_decode_tma(bf16* out, const bf16* q, int q_stride, const bf16* kc
                                   max_seq_len, cap_in2, cap_log2, sinks, st);
   return launch_decode_tma<64>(out, q, q_stride, kc, vc, bt, max_blocks, sl, qsl, B, H, KV, bs, ns, scale_log2, part_o, part_ml, ws, ws_bytes,
                                max_seq_len, cap_in2, cap_log2, sinks, st);
+}
+
+int attn_decode_splits(int B, int KV, int max_seq_len);      // attn.cu
+
+// One token per request under a sliding window: the request's last `window` keys.  Sizes: paged_attn_extras_decode_ok; ws holds
+// kge_attn_workspace_bytes.  max_seq_len bounds the contexts that a captured launch may grow to.
+int paged_attn_window_decode(void* out, const void* q, int q_stride, const void* kc, const void* vc, const int32_t* bt, int max_blocks, const int32_t* sl, const int32_t* qsl,
+                             int B, int H, int KV, int hd, int bs, float scale, int window, int max_seq_len, void* ws, int64_t ws_bytes, cudaStream_t st) {
+  KGE_REQUIRE(window > 0 && (hd == 64 || hd == 128) && q_stride % 8 == 0, "paged_attn_window_decode: window %d, heads of %d", window, hd);
+  int ns = attn_decode_splits(B, KV, window < max_seq_len ? window : max_seq_len);
+  const int64_t per = (int64_t)B * H * (hd + 2) * 4;
+  if (!ws || per * ns > ws_bytes) ns = 1;
+  float* po = (float*)ws;
+  float* pml = po + (int64_t)B * H * ns * hd;
+  const float sc = scale * 1.4426950408889634f;
+  if (hd == 128)
+    return launch_decode_tma<128>((bf16*)out, (const bf16*)q, q_stride, (const bf16*)kc, (const bf16*)vc, bt, max_blocks, sl, qsl, B, H, KV, bs, ns, sc, po, pml, nullptr, 0, max_seq_len, 0.f, 0.f,
+                                  nullptr, st, window);
+  return launch_decode_tma<64>((bf16*)out, (const bf16*)q, q_stride, (const bf16*)kc, (const bf16*)vc, bt, max_blocks, sl, qsl, B, H, KV, bs, ns, sc, po, pml, nullptr, 0, max_seq_len, 0.f, 0.f,
+                               nullptr, st, window);
 }
 
 }  // namespace KGE_ELT_NS

@@ -34,6 +34,9 @@ bool paged_attn_window_tc_ok(int H, int KV, int hd, int vd, int bs, int pool, in
 int paged_attn_window_tc(void* out, const void* q, int q_stride, const void* kc, const void* vc, const void* pkc, const void* pvc, const int32_t* bt,
                          int max_blocks, const int32_t* sl, const int32_t* qsl, int B, int max_q_len, int H, int KV, int hd, int bs, float scale,
                          int window, int keep_first, int pool, int pool_slots, const float* sinks, cudaStream_t st);
+// attn_decode_tma.cu: one token per request under a sliding window, keys and values staged by TMA (sizes: paged_attn_extras_decode_ok)
+int paged_attn_window_decode(void* out, const void* q, int q_stride, const void* kc, const void* vc, const int32_t* bt, int max_blocks, const int32_t* sl, const int32_t* qsl,
+                             int B, int H, int KV, int hd, int bs, float scale, int window, int max_seq_len, void* ws, int64_t ws_bytes, cudaStream_t st);
 // gemm_tc.cu: one tcgen05 launch over row groups padded to 256 (the experts of a prompt step)
 int gemm_grouped(void* y, const void* x, const void* w, int T, int N, int K, int groups, const int32_t* tile_group, int glu, float glu_alpha,
                  float glu_limit, cudaStream_t st);
@@ -673,7 +676,7 @@ int hybrid_engine_build(kge_engine* e, const ModelDir& md, int64_t dummy_seed, s
     // split-KV scratch of the TMA-staged decode attention, for attention mixers whose heads it takes
     int64_t need = 0;
     for (auto& h : s.hybrid)
-      if ((h.mixer == HybridLayerSpec::ATTENTION || (h.mixer == HybridLayerSpec::LATENT && !h.latent_cache)) && !e->f32 && (h.dim == 64 || h.dim == 128) && h.vdim == h.dim)
+      if ((h.mixer == HybridLayerSpec::ATTENTION || h.mixer == HybridLayerSpec::WINDOW_SSD || (h.mixer == HybridLayerSpec::LATENT && !h.latent_cache)) && !e->f32 && (h.dim == 64 || h.dim == 128) && h.vdim == h.dim)
         need = std::max<int64_t>(need, kge_attn_workspace_bytes(Rm, h.heads, h.dim, e->cfg.max_model_len));
     if (need > 0) {
       e->ws_attn_bytes = need;
@@ -1209,11 +1212,15 @@ int hybrid_forward(kge_engine* e, int T, int B, int R, int max_blocks, const Ste
       while (aa.num_decode < B && hm.qsl[aa.num_decode + 1] - hm.qsl[aa.num_decode] == 1) ++aa.num_decode;
       double keys = 0;                                   // visible keys over all rows
       for (int t = 0; t < T; ++t) keys += std::min(hm.pos[t] + 1, h.window);
-      // steps with prompt pieces, 64- / 128-wide heads, bfloat16: the tcgen05 kernel; decode steps and everything else: the mma.sync / per-row kernels
+      // steps with prompt pieces, 64- / 128-wide heads, bfloat16: the tcgen05 kernel; decode steps of such heads: the TMA-staged split-KV kernel;
+      // everything else: the mma.sync / per-row kernels
       const bool tc = !e->f32 && !decode_only && ldp % 8 == 0 && ((uintptr_t)e->pbuf & 15) == 0 && paged_attn_window_tc_ok(h.heads, h.kv_heads, h.dim, h.vdim, bs, 0, 0);
+      const bool dec_tc = !e->f32 && decode_only && e->ws_attn && h.vdim == h.dim && ldp % 8 == 0 && ((uintptr_t)e->pbuf & 15) == 0 && paged_attn_extras_decode_ok(B, h.heads, h.kv_heads, h.dim, bs);
       HFWD(decode_only ? C_ATT_DEC : C_ATT_GEN, (decode_only ? keys : (double)T) * h.kv_heads * (h.dim + h.vdim) * es + (double)T * h.heads * (h.dim + h.vdim) * es,
            2.0 * keys * h.heads * (h.dim + h.vdim),
-           tc ? paged_attn_window_tc(e->mixbuf, e->pbuf, ldp, L.kc, L.vc, nullptr, nullptr, m.btab, max_blocks, m.seq_lens, m.qsl, B, aa.max_q, h.heads, h.kv_heads, h.dim, bs,
+           dec_tc ? paged_attn_window_decode(e->mixbuf, e->pbuf, ldp, L.kc, L.vc, m.btab, max_blocks, m.seq_lens, m.qsl, B, h.heads, h.kv_heads, h.dim, bs, h.scale, h.window,
+                                             max_blocks * bs, e->ws_attn, e->ws_attn_bytes, st)
+           : tc ? paged_attn_window_tc(e->mixbuf, e->pbuf, ldp, L.kc, L.vc, nullptr, nullptr, m.btab, max_blocks, m.seq_lens, m.qsl, B, aa.max_q, h.heads, h.kv_heads, h.dim, bs,
                                      h.scale, h.window, 0, 0, 0, nullptr, st)
               : attn_bias_chunk(aa, st));
       HFWD(C_ACT, (double)T * ka * 3 * es, 0, sigmoid_gate_mul(e->mixbuf, ka, at(e->pbuf, L.off_mg), ldp, T, ka, elt, st));

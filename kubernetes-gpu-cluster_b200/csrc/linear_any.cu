@@ -366,10 +366,92 @@ __global__ void __launch_bounds__(256) linear_stream_kernel(LinearArgs a) {
     }
 }
 
+// Many rows, a short sum, fp32 output (the second half of a low-rank pair): the output is the traffic.  128 x 128 tiles whose operands
+// are staged whole (K <= 256) with cp.async; eight warps of 64 rows x 32 outputs, fragments by ldmatrix, the same order of summation
+// as above, two outputs per store.
+constexpr int WBM = 128, WBN = 128, WMAXK = 256;
+
+__device__ __forceinline__ void la_ldsm4(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)));
+}
+
+template <int ACT>
+__global__ void __launch_bounds__(256) linear_short_kernel(LinearArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  typedef __nv_bfloat16 E;
+  extern __shared__ __align__(16) unsigned char lw_raw[];
+  const int pitch = a.K + MPAD, pieces = a.K / 8;
+  E* xs = reinterpret_cast<E*>(lw_raw);                       // [WBM][pitch]
+  E* ws = xs + WBM * pitch;                                   // [WBN][pitch]
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, m0 = blockIdx.y * WBM, n0 = blockIdx.x * WBN;
+  for (int i = tid; i < (WBM + WBN) * pieces; i += 256) {
+    const int r = i / pieces, k = i % pieces * 8;
+    const bool isx = r < WBM;
+    const int g = isx ? m0 + r : n0 + r - WBM;
+    const bool ok = isx ? g < a.T : g < a.N;
+    const E* src = isx ? (const E*)a.x + (ok ? (int64_t)g * a.ldx + k : 0) : (const E*)a.w + (ok ? (int64_t)g * a.K + k : 0);
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(xs + r * pitch + k)), "l"(src), "r"(ok ? 16 : 0));
+  }
+  asm volatile("cp.async.commit_group;");
+  const int wm = (warp >> 2) * 64, wn = (warp & 3) * 32, lr = lane & 7, lm = lane >> 3;
+  float2 bias[4];
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const int n = n0 + wn + j * 8 + (lane & 3) * 2;
+    bias[j] = make_float2(a.bias && n < a.N ? ldf((const E*)a.bias + n) : 0.f, a.bias && n + 1 < a.N ? ldf((const E*)a.bias + n + 1) : 0.f);
+  }
+  float acc[4][4][4] = {};
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
+  for (int k = 0; k < a.K; k += 16) {
+    uint32_t bf[2][4];
+#pragma unroll
+    for (int j = 0; j < 2; ++j) la_ldsm4(bf[j], ws + (wn + j * 16 + (lm >> 1) * 8 + lr) * pitch + k + (lm & 1) * 8);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      uint32_t af[4];
+      la_ldsm4(af, xs + (wm + i * 16 + (lm & 1) * 8 + lr) * pitch + k + (lm >> 1) * 8);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) mma_bf16_16816(acc[i][j], af, bf[j >> 1][(j & 1) * 2], bf[j >> 1][(j & 1) * 2 + 1]);
+    }
+  }
+  float* y = (float*)a.y;
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int hh = 0; hh < 2; ++hh) {
+      const int r = m0 + wm + i * 16 + (lane >> 2) + hh * 8;
+      if (r >= a.T) continue;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int n = n0 + wn + j * 8 + (lane & 3) * 2;
+        if (n >= a.N) continue;                               // N is even: a pair is inside or outside
+        float u = acc[i][j][hh * 2] + bias[j].x, v = acc[i][j][hh * 2 + 1] + bias[j].y;
+        if (ACT == ACT_EXP_DECAY) { u = exp_decay(a.act_coef[n], u); v = exp_decay(a.act_coef[n + 1], v); }
+        else { u = act_apply(ACT, u); v = act_apply(ACT, v); }
+        *reinterpret_cast<float2*>(y + (int64_t)r * a.ldy + n) = make_float2(u * a.alpha, v * a.alpha);
+      }
+    }
+}
+
+static bool linear_short_ok(const LinearArgs& a) {
+  return a.elt == KGE_ELT_BF16 && a.out_f32 && !a.w2 && !a.group_off && !a.xrows && !a.yrows && !a.row_scale && !a.accumulate && a.nz == 1 && a.T > 256 && a.K % 16 == 0 && a.K <= WMAXK &&
+         a.N % 2 == 0 && a.ldy % 2 == 0 && a.ldx % 8 == 0 && (a.T + WBM - 1) / WBM <= 65535 && (a.act == ACT_NONE || a.act == ACT_SOFTPLUS || a.act == ACT_EXP_DECAY) &&
+         ((reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.w)) & 15) == 0 && (reinterpret_cast<uintptr_t>(a.y) & 7) == 0;
+}
+
 int linear_any(const LinearArgs& a, cudaStream_t st) {
   KGE_REQUIRE(a.x && a.w && a.y && a.N > 0 && a.K > 0 && a.nz > 0, "linear_any: bad arguments");
   KGE_REQUIRE(a.act != ACT_EXP_DECAY || (a.act_coef && !a.w2), "linear_any: the decay needs its coefficients");
   if (a.T <= 0) return 0;
+  if (linear_short_ok(a)) {
+    const size_t smem = (size_t)(WBM + WBN) * (a.K + MPAD) * 2;
+    auto kern = a.act == ACT_SOFTPLUS ? linear_short_kernel<ACT_SOFTPLUS> : a.act == ACT_EXP_DECAY ? linear_short_kernel<ACT_EXP_DECAY> : linear_short_kernel<ACT_NONE>;
+    KGE_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    KGE_CUDA_OK(launch_pdl(kern, dim3((a.N + WBN - 1) / WBN, (a.T + WBM - 1) / WBM), dim3(256), smem, st, a));
+    return 0;
+  }
   const int rows = a.group_off ? (a.max_rows > 0 ? a.max_rows : a.T) : a.T;
   dim3 grid((a.N + LBN - 1) / LBN, (rows + LBM - 1) / LBM, a.nz), block(256);
   KGE_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "linear_any: too many row tiles (%u) or slices (%u)", grid.y, grid.z);

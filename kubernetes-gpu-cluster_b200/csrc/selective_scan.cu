@@ -134,6 +134,123 @@ __global__ void __launch_bounds__(SS_THREADS) selective_scan_kernel(SelectiveSca
   }
 }
 
+// The same walk for bfloat16 rows in whole 16-byte pieces (channels, states, strides and offsets multiples of 8): a thread requests the
+// next stage's pieces as they are and converts B and C once, on their way to shared memory.
+template <int KQ, int NPT, int CT>
+__global__ void __launch_bounds__(SS_THREADS) selective_scan_vec_kernel(SelectiveScanArgs a) {
+  pdl_launch_dependents();
+  typedef __nv_bfloat16 E;
+  constexpr int CH = SS_THREADS / KQ, NW = KQ * NPT, NP = NPT / 2;
+  constexpr int NBC = 2 * CT * NW / 8, NX = CT * CH / 8, ND = CT * CH / 4;      // 16-byte pieces of a stage: B and C rows, x (and z) rows, dt rows
+  constexpr int PB = NBC / SS_THREADS, PX = (2 * NX + SS_THREADS - 1) / SS_THREADS, PD = (ND + SS_THREADS - 1) / SS_THREADS;
+  static_assert(NBC % SS_THREADS == 0 && CH % 8 == 0, "pieces");
+  __shared__ __align__(16) float BCs[CT][2 * NW], ds[CT][CH];
+  __shared__ __align__(16) E xz[2][CT][CH];
+  const int tid = threadIdx.x, kq = tid % KQ, ch = tid / KQ, c0 = blockIdx.x * CH, c = c0 + ch, b = blockIdx.y, N = a.N, C = a.C;
+  const bool on = c < C;
+  f2 A2[NP];
+#pragma unroll
+  for (int i = 0; i < NP; ++i) {
+    const int n = kq * NPT + 2 * i;
+    A2[i] = pk(on && n < N ? a.A[(int64_t)c * N + n] * LOG2E : 0.f, on && n + 1 < N ? a.A[(int64_t)c * N + n + 1] * LOG2E : 0.f);
+  }
+  const float D = on ? a.D[c] : 0.f;
+  pdl_wait();
+  const int r0 = a.qsl[b], r1 = a.qsl[b + 1];
+  if (r0 >= r1) return;
+  const bool fresh = a.positions[r0] == 0;
+  float* Sg = a.state + (int64_t)a.slots[b] * a.slot_stride + (int64_t)c * N + kq * NPT;
+  f2 S[NP];
+#pragma unroll
+  for (int i = 0; i < NP; ++i) {
+    const int n = kq * NPT + 2 * i;
+    S[i] = pk(on && !fresh && n < N ? Sg[2 * i] : 0.f, on && !fresh && n + 1 < N ? Sg[2 * i + 1] : 0.f);
+  }
+  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+  uint4 pb[PB], px[PX], pd[PD];
+  auto fetch = [&](int t0) {
+#pragma unroll
+    for (int i = 0; i < PB; ++i) {
+      const int e = i * SS_THREADS + tid, t = t0 + e / (NW / 4), q = e % (NW / 4), n = q % (NW / 8) * 8;
+      const E* src = (const E*)(q < NW / 8 ? a.b : a.c) + (int64_t)t * a.ldbc + n;
+      pb[i] = t < r1 && n < N ? *reinterpret_cast<const uint4*>(src) : zero;
+    }
+#pragma unroll
+    for (int i = 0; i < PX; ++i) {
+      const int e = i * SS_THREADS + tid, z = e / NX, f = e % NX, t = t0 + f / (CH / 8), k = c0 + f % (CH / 8) * 8;
+      px[i] = e < 2 * NX && t < r1 && k < C ? *reinterpret_cast<const uint4*>(z ? (const E*)a.z + (int64_t)t * a.ldz + k : (const E*)a.x + (int64_t)t * a.ldx + k) : zero;
+    }
+#pragma unroll
+    for (int i = 0; i < PD; ++i) {
+      const int e = i * SS_THREADS + tid, t = t0 + e / (CH / 4), k = c0 + e % (CH / 4) * 4;
+      pd[i] = e < ND && t < r1 && k < C ? *reinterpret_cast<const uint4*>(a.dt + (int64_t)t * a.lddt + k) : zero;      // a row beyond the request leaves the state as it is
+    }
+  };
+  fetch(r0);
+  for (int t0 = r0; t0 < r1; t0 += CT) {
+    __syncthreads();                                 // the previous stage's readers are done
+#pragma unroll
+    for (int i = 0; i < PB; ++i) {
+      const int e = i * SS_THREADS + tid;
+      float* dst = &BCs[e / (NW / 4)][e % (NW / 4) * 8];
+      *reinterpret_cast<float4*>(dst) = make_float4(__uint_as_float(pb[i].x << 16), __uint_as_float(pb[i].x & 0xffff0000u), __uint_as_float(pb[i].y << 16), __uint_as_float(pb[i].y & 0xffff0000u));
+      *reinterpret_cast<float4*>(dst + 4) = make_float4(__uint_as_float(pb[i].z << 16), __uint_as_float(pb[i].z & 0xffff0000u), __uint_as_float(pb[i].w << 16), __uint_as_float(pb[i].w & 0xffff0000u));
+    }
+#pragma unroll
+    for (int i = 0; i < PX; ++i) {
+      const int e = i * SS_THREADS + tid;
+      if (e < 2 * NX) reinterpret_cast<uint4*>(&xz[0][0][0])[e] = px[i];
+    }
+#pragma unroll
+    for (int i = 0; i < PD; ++i) {
+      const int e = i * SS_THREADS + tid;
+      if (e < ND) reinterpret_cast<uint4*>(&ds[0][0])[e] = pd[i];
+    }
+    __syncthreads();
+    if (t0 + CT < r1) fetch(t0 + CT);
+    const int n = min(CT, r1 - t0);
+#pragma unroll 2
+    for (int q = 0; q < n; q += 4) {
+      float y[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const float dt = ds[q + u][ch], dx = dt * __bfloat162float(xz[0][q + u][ch]);
+        const f2 dt2 = pk(dt, dt), dx2 = pk(dx, dx);
+        f2 acc = 0ull;
+#pragma unroll
+        for (int i = 0; i < NP; i += 2) {
+          const ulonglong2 B2 = *reinterpret_cast<const ulonglong2*>(&BCs[q + u][kq * NPT + 2 * i]), C2 = *reinterpret_cast<const ulonglong2*>(&BCs[q + u][NW + kq * NPT + 2 * i]);
+          float e0, e1, e2, e3;
+          upk(mul2(dt2, A2[i]), e0, e1);
+          upk(mul2(dt2, A2[i + 1]), e2, e3);
+          S[i] = fma2(pk(ex2(e0), ex2(e1)), S[i], mul2(dx2, B2.x));
+          S[i + 1] = fma2(pk(ex2(e2), ex2(e3)), S[i + 1], mul2(dx2, B2.y));
+          acc = fma2(S[i], C2.x, acc);
+          acc = fma2(S[i + 1], C2.y, acc);
+        }
+        y[u] = sum2(acc);
+      }
+      const bool o0 = kq & 1, o1 = kq & 2;           // sums over the KQ lanes as above
+      const float s0 = (o0 ? y[1] : y[0]) + __shfl_xor_sync(0xffffffffu, o0 ? y[0] : y[1], 1);
+      const float s1 = (o0 ? y[3] : y[2]) + __shfl_xor_sync(0xffffffffu, o0 ? y[2] : y[3], 1);
+      float s = (o1 ? s1 : s0) + __shfl_xor_sync(0xffffffffu, o1 ? s0 : s1, 2);
+#pragma unroll
+      for (int off = 4; off < KQ; off <<= 1) s += __shfl_xor_sync(0xffffffffu, s, off);
+      const int u = q + (kq & 3);
+      if (on && kq < 4 && u < n)
+        ((E*)a.out)[(int64_t)(t0 + u) * a.ldo + c] = __float2bfloat16_rn(fmaf(D, __bfloat162float(xz[0][u][ch]), s) * silu_f<E>(__bfloat162float(xz[1][u][ch])));
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < NP; ++i) {
+    const int n = kq * NPT + 2 * i;
+    float x, y;
+    upk(S[i], x, y);
+    if (on && n < N) Sg[2 * i] = x;
+    if (on && n + 1 < N) Sg[2 * i + 1] = y;
+  }
+}
+
 // one row per request (row b belongs to request b): NQ = N / 4 neighbouring lanes hold a channel, RPT requests per thread
 template <typename E, int RPT>
 __global__ void __launch_bounds__(256) selective_step_kernel(SelectiveScanArgs a, int NQ) {
@@ -180,6 +297,12 @@ cudaError_t launch_scan(const SelectiveScanArgs& a, cudaStream_t st) {
   return launch_pdl(selective_scan_kernel<E, KQ, NPT, CT>, dim3((a.C + CH - 1) / CH, a.B), dim3(SS_THREADS), 0, st, a);
 }
 
+template <int KQ, int NPT, int CT>
+cudaError_t launch_scan_vec(const SelectiveScanArgs& a, cudaStream_t st) {
+  constexpr int CH = SS_THREADS / KQ;
+  return launch_pdl(selective_scan_vec_kernel<KQ, NPT, CT>, dim3((a.C + CH - 1) / CH, a.B), dim3(SS_THREADS), 0, st, a);
+}
+
 template <typename E>
 cudaError_t dispatch(const SelectiveScanArgs& a, cudaStream_t st) {
   const int NQ = a.N / 4;
@@ -190,6 +313,10 @@ cudaError_t dispatch(const SelectiveScanArgs& a, cudaStream_t st) {
     return a.B >= 16 ? launch_pdl(selective_step_kernel<E, 4>, dim3(gx, (a.B + 3) / 4), dim3(256), 0, st, a, NQ)
                      : launch_pdl(selective_step_kernel<E, 1>, dim3(gx, a.B), dim3(256), 0, st, a, NQ);
   }
+  auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  if (std::is_same<E, __nv_bfloat16>::value && a.N % 8 == 0 && a.N <= 64 && a.C % 8 == 0 && a.ldx % 8 == 0 && a.ldz % 8 == 0 && a.ldbc % 8 == 0 && a.lddt % 4 == 0 && al16(a.x) && al16(a.z) &&
+      al16(a.b) && al16(a.c) && al16(a.dt))
+    return a.N <= 16 ? launch_scan_vec<4, 4, 32>(a, st) : a.N <= 32 ? launch_scan_vec<4, 8, 16>(a, st) : launch_scan_vec<8, 8, 16>(a, st);
   if (a.N <= 16) return launch_scan<E, 4, 4, 16>(a, st);
   if (a.N <= 32) return launch_scan<E, 4, 8, 16>(a, st);
   if (a.N <= 64) return launch_scan<E, 8, 8, 8>(a, st);

@@ -224,27 +224,31 @@ __global__ void __launch_bounds__(256, 2) ssd_chunk_kernel(SsdArgs a, int ptiles
   auto dt_raw = [&](int t) { return t < r1 ? ldf((const E*)a.dt_pre + (int64_t)t * a.lddt + h) : 0.f; };
   float raw0 = 0.f, raw1 = 0.f;                       // warp 0: the logits of two tokens per lane, a chunk ahead
   if (warp == 0) { raw0 = dt_raw(r0 + lane * 2); raw1 = dt_raw(r0 + lane * 2 + 1); }
-  const int rt = warp & 3, ct = (warp >> 2) * 32;     // read-out: 16 rows x 32 columns per warp
+  // read-out: 16 rows x 32 columns per warp; a row tile has more keys the later it lies, so the two halves run through them in opposite order
+  const int rt = warp < 4 ? warp : 7 - warp, ct = (warp >> 2) * 32;
   const int lr = lane & 7, lm = lane >> 3;            // ldmatrix: row within a matrix, matrix
+  // running sums, steps and weights of the chunk that starts at t0, into half s of their buffers (warp 0, two tokens per lane); the
+  // logits of the chunk after it are requested
+  auto scalars = [&](int t0, int s) {
+    const int t = t0 + lane * 2;
+    const float d0 = t < r1 ? softplus_f(raw0 + bias) : 0.f, d1 = t + 1 < r1 ? softplus_f(raw1 + bias) : 0.f;      // rows beyond the request: no step, no decay
+    raw0 = dt_raw(t + CL); raw1 = dt_raw(t + CL + 1);
+    const double l0 = (double)(-coef * d0) * 1.4426950408889634, l1 = (double)(-coef * d1) * 1.4426950408889634;
+    double run = l0 + l1;
+#pragma unroll
+    for (int off = 1; off < 32; off <<= 1) { const double o = __shfl_up_sync(0xffffffffu, run, off); if (lane >= off) run += o; }
+    const double c1 = run, c0 = run - l1, tot = __shfl_sync(0xffffffffu, run, 31);
+    const float h0 = (float)c0, h1 = (float)c1;
+    sm.hi[s][lane * 2] = h0; sm.hi[s][lane * 2 + 1] = h1;
+    sm.lo[s][lane * 2] = (float)(c0 - (double)h0); sm.lo[s][lane * 2 + 1] = (float)(c1 - (double)h1);
+    sm.dt[s][lane * 2] = d0; sm.dt[s][lane * 2 + 1] = d1;
+    sm.w[s][lane * 2] = exp2f((float)(tot - c0)) * d0; sm.w[s][lane * 2 + 1] = exp2f((float)(tot - c1)) * d1;
+    sm.er[s][lane * 2] = exp2f(h0); sm.er[s][lane * 2 + 1] = exp2f(h1);
+    if (lane == 0) sm.etot[s] = exp2f((float)tot);
+  };
+  if (warp == 0) scalars(r0, 0);
   int s = 0;
   for (int t0 = r0; t0 < r1; t0 += CL, s ^= 1) {
-    if (warp == 0) {
-      const int t = t0 + lane * 2;
-      const float d0 = t < r1 ? softplus_f(raw0 + bias) : 0.f, d1 = t + 1 < r1 ? softplus_f(raw1 + bias) : 0.f;      // rows beyond the request: no step, no decay
-      raw0 = dt_raw(t + CL); raw1 = dt_raw(t + CL + 1);
-      const double l0 = (double)(-coef * d0) * 1.4426950408889634, l1 = (double)(-coef * d1) * 1.4426950408889634;
-      double run = l0 + l1;
-#pragma unroll
-      for (int off = 1; off < 32; off <<= 1) { const double o = __shfl_up_sync(0xffffffffu, run, off); if (lane >= off) run += o; }
-      const double c1 = run, c0 = run - l1, tot = __shfl_sync(0xffffffffu, run, 31);
-      const float h0 = (float)c0, h1 = (float)c1;
-      sm.hi[s][lane * 2] = h0; sm.hi[s][lane * 2 + 1] = h1;
-      sm.lo[s][lane * 2] = (float)(c0 - (double)h0); sm.lo[s][lane * 2 + 1] = (float)(c1 - (double)h1);
-      sm.dt[s][lane * 2] = d0; sm.dt[s][lane * 2 + 1] = d1;
-      sm.w[s][lane * 2] = exp2f((float)(tot - c0)) * d0; sm.w[s][lane * 2 + 1] = exp2f((float)(tot - c1)) * d1;
-      sm.er[s][lane * 2] = exp2f(h0); sm.er[s][lane * 2 + 1] = exp2f(h1);
-      if (lane == 0) sm.etot[s] = exp2f((float)tot);
-    }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
     const int n = min(CL, r1 - t0);
@@ -313,8 +317,9 @@ __global__ void __launch_bounds__(256, 2) ssd_chunk_kernel(SsdArgs a, int ptiles
           }
         }
     }
-    __syncthreads();                                  // C and the split state have been read
     const bool more = t0 + CL < r1;
+    if (warp == 0 && more) scalars(t0 + CL, s ^ 1);   // the warp with the shortest read-out
+    __syncthreads();                                  // C and the split state have been read
     if (more) load_rows(&sm.C[0][0], BP, cg, t0 + CL, NPC, N / 8);
     {
       const float et = sm.etot[s];

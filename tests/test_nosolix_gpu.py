@@ -246,8 +246,8 @@ def test_pages_and_slots_are_used_again(kge, tmp_path):
         check(got[r], Case(cfg, W, P[r], "float32"), "float32", f"request {r}")
 
 
-EDGES = [      # heads, kv heads, dim, vdim, window, page: per-row kernel; mma.sync (equal and unequal sizes); the tcgen05 prompt kernel
-    (4, 2, 6, 5, 21, 16), (4, 1, 16, 8, 37, 16), (6, 2, 48, 80, 64, 32), (6, 3, 64, 128, 45, 64), (4, 2, 64, 64, 70, 64), (6, 2, 128, 128, 33, 16), (8, 8, 64, 64, 66, 64)]
+EDGES = [      # heads, kv heads, dim, vdim, window, page: per-row kernel; mma.sync (equal and unequal sizes); the tcgen05 prompt kernel, alone and with the TMA-staged decode kernel
+    (4, 2, 6, 5, 21, 16), (4, 1, 16, 8, 37, 16), (6, 2, 48, 80, 64, 32), (6, 3, 64, 128, 45, 64), (4, 2, 64, 64, 70, 64), (6, 2, 128, 128, 33, 16), (4, 2, 128, 128, 39, 128), (8, 8, 64, 64, 66, 64)]
 
 
 @pytest.mark.parametrize("case", EDGES)
@@ -272,6 +272,29 @@ def test_window_edges_with_peaked_scores(kge, tmp_path, dtype, case):
     llm.trace_end(1)
     check(run_pieces(llm, 2, c.toks, [size - 2] + [1] * (200 - size + 2)), c, dtype, "decoding while the window comes into play")
     llm.close()
+
+
+@pytest.mark.parametrize("dim", [64, 128])
+def test_decoding_under_a_long_window(kge, tmp_path, dim):
+    """A window of many key tiles, split over several CTAs when few requests decode: contexts shorter and longer than the window in
+    one batch, its lower edge inside a tile."""
+    cfg = ok.make_config([PAR(heads=4, kv_heads=2, dim=dim, vdim=dim, size=523, scale=2.0 / dim ** 0.5, base=300.0, original=64, mlp=None)], width=40)
+    W = only(ok.make_weights(cfg, seed=28), "left")
+    a, b = Case(cfg, W, prompt(cfg, 650, 46)), Case(cfg, W, prompt(cfg, 30, 47))
+    llm = make_engine(kge, tmp_path, cfg, W, "bfloat16", bs=64, tokens=1024)
+    llm.trace_add(0, a.toks[:630])
+    llm.trace_add(1, b.toks[:10])
+    llm.trace_step([(0, 630, []), (1, 10, [])])
+    ga, gb = [], []
+    for i in range(20):
+        llm.trace_add(0, a.toks[630 + i:631 + i])
+        llm.trace_add(1, b.toks[10 + i:11 + i])
+        lg = llm.trace_step([(0, 1, [0]), (1, 1, [0])])
+        ga.append(lg[0])
+        gb.append(lg[1])
+    llm.close()
+    check(np.stack(ga), a, "bfloat16", "long request", slice(630, 650))
+    check(np.stack(gb), b, "bfloat16", "short request", slice(10, 30))
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
@@ -497,7 +520,7 @@ def test_recurrent_head_sizes(kge, tmp_path, dtype, shape):
     check(lg[101:], c, dtype, "another piece", slice(0, 70))
 
 
-SCAN_SIZES = [(40, 16, 8, 4), (33, 24, 12, 3), (64, 4, 1, 2), (17, 48, 3, 4), (32, 64, 16, 4), (20, 100, 4, 3), (24, 128, 8, 2), (9, 200, 2, 1), (12, 256, 5, 3), (48, 8, 24, 5)]      # channels, state, rank, taps
+SCAN_SIZES = [(40, 16, 8, 4), (40, 24, 8, 3), (33, 24, 12, 3), (64, 4, 1, 2), (17, 48, 3, 4), (32, 64, 16, 4), (20, 100, 4, 3), (24, 128, 8, 2), (9, 200, 2, 1), (12, 256, 5, 3), (48, 8, 24, 5)]      # channels, state, rank, taps
 
 
 @pytest.mark.parametrize("shape", SCAN_SIZES)
