@@ -10,7 +10,7 @@ namespace kge {
 // Thread-local error text behind kge_last_error() (api.cc).
 void set_error(const char* fmt, ...);
 // Process-wide switch for programmatic dependent launch (api.cc).  On by default; turned off by
-// KGE_DISABLE_PDL and by tensor-parallel engines (see DESIGN.md "known issues").
+// KGE_DISABLE_PDL and by tensor-parallel engines.
 bool pdl_enabled();
 void pdl_set_enabled(bool on);
 // pdl_break_next(): the next launch from this thread is an ordinary stream-ordered launch (it neither starts early nor
